@@ -50,6 +50,7 @@ extern "C" {
 #define RD_EPI_BIAS_SILU_RES 3 /* C = R[m,n] + silu(acc + bias[n]) */
 #define RD_EPI_RES 4           /* C = R[m,n] + acc (R may alias C) */
 #define RD_EPI_SWIGLU 5        /* C[m,i] = silu(acc[m,2i]) * acc[m,2i+1]; C has N/2 columns */
+#define RD_EPI_XIELU 9         /* C = xIELU(acc); through rd_gemm_xielu / rd_gemm_bf16_tc_xielu, which take its coefficients */
 
 /* Attention visibility of the new tokens among themselves. */
 #define RD_ATTN_CAUSAL 0 /* new token i sees new tokens 0..i */
@@ -161,8 +162,8 @@ RD_API int rd_drafter_dense_log_probs(int B, int W, int Lb, int V, const float* 
  * (LM head, modeling_llama.py:272).  bias [N] in `dtype`; R [M, ldr] in out_dtype.
  *
  * rd_gemm is the exact-fp32 / generic path (CUDA cores).  rd_gemm_bf16_tc is the tensor-core
- * path (tcgen05 + TMEM accumulators, operands staged by TMA); it needs bf16 operands, K a
- * multiple of 64, 16-byte aligned A, W and C/R rows; `tensor_maps` is a host pointer returned
+ * path (tcgen05 + TMEM accumulators, operands staged by TMA); it needs bf16 operands, K >= 64 and a
+ * multiple of 8, 16-byte aligned A, W and C/R rows; `tensor_maps` is a host pointer returned
  * by rd_gemm_plan_create for these exact (A, W) buffers. */
 RD_API int rd_gemm(int dtype, int out_dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
             const void* bias, const void* R, int64_t ldr, int m_max, const int32_t* m_dev, int N, int K,
@@ -174,6 +175,18 @@ RD_API void* rd_gemm_plan_create(const void* A, int64_t lda, int m_max, const vo
 RD_API void rd_gemm_plan_destroy(void* plan);
 RD_API int rd_gemm_bf16_tc(const void* plan, int out_dtype, void* C, int64_t ldc, const void* bias, const void* R,
                     int64_t ldr, const int32_t* m_dev, int epilogue, int32_t* status, void* stream);
+
+/* C = xIELU(A W^T): pos z^2 + z/2 for z > 0, neg (e^z - 1 - z) + z/2 otherwise (pos = softplus(p),
+ * neg = 1/2 + softplus(q) of the activation's two parameters).  No counterpart in the reference. */
+RD_API int rd_gemm_xielu(int dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int m_max,
+                  const int32_t* m_dev, int N, int K, float pos, float neg, void* stream);
+RD_API int rd_gemm_bf16_tc_xielu(const void* plan, void* C, int64_t ldc, const int32_t* m_dev, float pos, float neg,
+                          int32_t* status, void* stream);
+
+/* A W^T whose output features [0, n_split) go to C as bf16 and [n_split, N) to C_hi as fp32 (column n - n_split):
+ * projections some of whose outputs must not be rounded, such as the gates of a recurrence.  n_split a multiple of 32. */
+RD_API int rd_gemm_bf16_tc_split(const void* plan, void* C, int64_t ldc, float* C_hi, int64_t ld_hi, int n_split,
+                          const int32_t* m_dev, int32_t* status, void* stream);
 
 /* The QKV projection (modeling_llama.py:141-143) with apply_rotary_pos_emb (:104-110) and the cache
  * append (:157-159) done in its epilogue: `plan` holds (normed activations, packed [q;k;v] weight
@@ -383,6 +396,58 @@ RD_API int rd_cache_unpack(int dtype, void* cache, int NL, int B, int nkv, int m
 #define RD_STATIC_SCRATCH_BYTES (16u << 20)
 RD_API int rd_cache_unpack_static(int dtype, void* cache, int NL, int B, int nkv, int max_len, int hd, int S,
                                   const int64_t* unpacker, int n_flat, void* stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Decoders with a 32-bit residual stream, sliding-window attention and matrix-memory layers.  No
+ * counterpart in the reference. */
+
+/* One row of the residual stream and its norm: x[t] = embed_scale * table[ids[t]] (table given), or
+ * sum_j coeff[j] * hist[j * hist_stride + t * H ..] over n_hist stored fp32 rows (coeff NULL: n_hist is 1 and
+ * the row is taken as it is); x_out (optional) receives x; y[t] = weight * x / sqrt(mean over each of `groups`
+ * equal consecutive parts of x^2 + eps), rounded once.  table, weight, y in `dtype`; coeff on the device. */
+RD_API int rd_stream_norm(int dtype, const void* table, const int64_t* ids, float embed_scale, const float* hist,
+                   int64_t hist_stride, const float* coeff, int n_hist, float* x_out, const void* weight, void* y, int m_max,
+                   const int32_t* m_dev, int H, int groups, float eps, void* stream);
+
+/* Rotary embedding of the first rot_dims features of every q and k head (feature i paired with i + rot_dims/2;
+ * cos/sin tables [n_pos, rot_dims/2]) and the cache append.  proj row: q [nh*dim] | k [nkv*dim] | v [nkv*vdim] | anything;
+ * q is rotated in place, k and v go to k_cache [B, nkv, max_len, dim] / v_cache [B, nkv, max_len, vdim]. */
+RD_API int rd_rotary_append(int dtype, void* proj, int64_t ld, void* k_cache, void* v_cache, const int32_t* tok_row,
+                     const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos,
+                     int m_max, const int32_t* m_dev, int nh, int nkv, int dim, int vdim, int rot_dims, int max_len,
+                     void* stream);
+
+/* Attention of the new tokens of every row over the row's cached keys and the new tokens themselves, where a query at
+ * position p sees a key at position s <= p iff p - s < window or s < keep_first.  Cached key j sits at position j, a
+ * causal new token i of a row at base_len + i; in mode RD_ATTN_TREE new tokens see each other through tree_mask and sit
+ * at tok_pos [m].  q: head h of token t at q + t*ldq + h*dim; gate (optional): head h's output is multiplied by
+ * sigmoid(gate[t*ld_gate + h]); out [m, nh*vdim].  vdim <= 512. */
+RD_API int rd_attention_window(int dtype, const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const void* gate,
+                        int64_t ld_gate, void* out, const int32_t* row_start, const int32_t* kv_begin, const int32_t* base_len,
+                        int B, int nh, int nkv, int dim, int vdim, int max_len, int max_new, int mode, const int32_t* tok_pos,
+                        const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first, void* stream);
+
+/* Matrix-memory recurrence with exponential gates over the new tokens of every row, token after token, continuing and
+ * updating the row's fp32 state S [B, nh, dim, vdim], n [B, nh, dim], m [B, nh] (a row whose base_len is 0 starts from
+ * zero): see csrc/mlstm.cu for the equations.  proj row: q [nh*dim] | k [nh*dim] | v [nh*vdim] | g [nh*vdim] in `dtype`;
+ * gates row: input [nh] | forget [nh] pre-activations, fp32, bias_* fp32 [nh].  out [m, nh*vdim]: normalised per head,
+ * times norm_weight, times sigmoid(g); NULL updates the state only.  With path given row b runs the tokens
+ * row_start[b] + path[(b*W + seq[b])*Lb + j], j = 0 .. count[b], instead of all of its own (commit of an accepted draft). */
+RD_API int rd_mlstm_scan(int dtype, const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
+                  const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S, float* n,
+                  float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int max_new,
+                  const int32_t* path, int W, int Lb, const int32_t* seq, const int32_t* count, void* stream);
+
+/* K or V rows of an accepted draft path: slot base_len[b] + unpacker[b, seq, j] moves to base_len[b] + j for j = 0 ..
+ * n_accepted[b] (cache [B, nkv, max_len, dim], one call per plane). */
+RD_API int rd_cache_commit(int dtype, void* cache, int B, int nkv, int max_len, int dim, const int32_t* kv_begin,
+                    const int32_t* base_len, const int32_t* unpacker, int W, int Lb, const int32_t* n_accepted,
+                    const int32_t* seq_in_beam, void* stream);
+
+/* Bookkeeping between two one-token decode steps: next_tok[b] goes to token_buf (optional) at column buf_begin[b] +
+ * kv_len[b]; slot[b] = begin[b] + kv_len[b] (at most limit - 1), base_len[b] = kv_len[b], kv_len[b] += 1. */
+RD_API int rd_decode_advance(const int64_t* next_tok, int64_t* token_buf, int64_t buf_ld, const int32_t* buf_begin,
+                      const int32_t* begin, int32_t* kv_len, int32_t* base_len, int32_t* slot, int limit, int B, void* stream);
 
 #ifdef __cplusplus
 }

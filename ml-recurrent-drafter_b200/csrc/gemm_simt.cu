@@ -22,7 +22,8 @@ template <typename T, typename OutT, int EPI>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A, int64_t lda, const T* __restrict__ W,
                                                         int64_t ldw, OutT* C, int64_t ldc, const T* __restrict__ bias,
                                                         const OutT* R, int64_t ldr, int m_max,
-                                                        const int32_t* __restrict__ m_dev, int N, int K) {
+                                                        const int32_t* __restrict__ m_dev, int N, int K, float act0,
+                                                        float act1) {
   const int M = rd::live_rows(m_dev, m_max);
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   if (m0 >= M) return;
@@ -73,6 +74,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
         float v = acc[i][j];
         if (EPI == RD_EPI_BIAS || EPI == RD_EPI_BIAS_SILU || EPI == RD_EPI_BIAS_SILU_RES) v += rd::Num<T>::to_f(bias[n]);
         if (EPI == RD_EPI_BIAS_SILU || EPI == RD_EPI_BIAS_SILU_RES) v = rd::silu_exact(v);
+        if (EPI == RD_EPI_XIELU) v = rd::xielu_exact(v, act0, act1);
         if (EPI == RD_EPI_BIAS_SILU_RES || EPI == RD_EPI_RES) v += rd::Num<OutT>::to_f(R[(int64_t)m * ldr + n]);
         store_out<OutT>(C + (int64_t)m * ldc + n, v);
       }
@@ -82,12 +84,12 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
 
 template <typename T, typename OutT>
 int launch(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, const void* bias, const void* R,
-           int64_t ldr, int m_max, const int32_t* m_dev, int N, int K, int epilogue, cudaStream_t s) {
+           int64_t ldr, int m_max, const int32_t* m_dev, int N, int K, int epilogue, float act0, float act1, cudaStream_t s) {
   dim3 grid((N + BN - 1) / BN, (m_max + BM - 1) / BM);
 #define RD_LAUNCH_EPI(E)                                                                                              \
   case E:                                                                                                             \
     gemm_simt_kernel<T, OutT, E><<<grid, 256, 0, s>>>((const T*)A, lda, (const T*)W, ldw, (OutT*)C, ldc, (const T*)bias, \
-                                                      (const OutT*)R, ldr, m_max, m_dev, N, K);                       \
+                                                      (const OutT*)R, ldr, m_max, m_dev, N, K, act0, act1);           \
     break;
   switch (epilogue) {
     RD_LAUNCH_EPI(RD_EPI_NONE)
@@ -96,6 +98,7 @@ int launch(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int6
     RD_LAUNCH_EPI(RD_EPI_BIAS_SILU_RES)
     RD_LAUNCH_EPI(RD_EPI_RES)
     RD_LAUNCH_EPI(RD_EPI_SWIGLU)
+    RD_LAUNCH_EPI(RD_EPI_XIELU)
     default:
       return RD_ERR_ARG;
   }
@@ -106,9 +109,9 @@ int launch(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int6
 
 }  // namespace
 
-extern "C" int rd_gemm(int dtype, int out_dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C,
-                       int64_t ldc, const void* bias, const void* R, int64_t ldr, int m_max, const int32_t* m_dev, int N,
-                       int K, int epilogue, void* stream) {
+static int gemm_checked(int dtype, int out_dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+                        const void* bias, const void* R, int64_t ldr, int m_max, const int32_t* m_dev, int N, int K,
+                        int epilogue, float act0, float act1, void* stream) {
   RD_REQUIRE(A && W && C, RD_ERR_ARG);
   RD_REQUIRE(m_max >= 1 && N >= 1 && K >= 1 && lda >= K && ldw >= K, RD_ERR_SIZE);
   const bool need_bias = epilogue == RD_EPI_BIAS || epilogue == RD_EPI_BIAS_SILU || epilogue == RD_EPI_BIAS_SILU_RES;
@@ -119,10 +122,23 @@ extern "C" int rd_gemm(int dtype, int out_dtype, const void* A, int64_t lda, con
   RD_REQUIRE(ldc >= (epilogue == RD_EPI_SWIGLU ? N / 2 : N), RD_ERR_SIZE);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == RD_F32 && out_dtype == RD_F32)
-    return launch<float, float>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, s);
+    return launch<float, float>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, act0, act1, s);
   if (dtype == RD_BF16 && out_dtype == RD_BF16)
-    return launch<__nv_bfloat16, __nv_bfloat16>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, s);
+    return launch<__nv_bfloat16, __nv_bfloat16>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, act0, act1, s);
   if (dtype == RD_BF16 && out_dtype == RD_F32)
-    return launch<__nv_bfloat16, float>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, s);
+    return launch<__nv_bfloat16, float>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, act0, act1, s);
   return RD_ERR_DTYPE;
+}
+
+extern "C" int rd_gemm(int dtype, int out_dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+                       const void* bias, const void* R, int64_t ldr, int m_max, const int32_t* m_dev, int N,
+                       int K, int epilogue, void* stream) {
+  RD_REQUIRE(epilogue != RD_EPI_XIELU, RD_ERR_ARG);  // it has parameters: rd_gemm_xielu
+  return gemm_checked(dtype, out_dtype, A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, 0.f, 0.f, stream);
+}
+
+extern "C" int rd_gemm_xielu(int dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int m_max,
+                             const int32_t* m_dev, int N, int K, float pos, float neg, void* stream) {
+  return gemm_checked(dtype, dtype, A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, m_max, m_dev, N, K, RD_EPI_XIELU, pos, neg,
+                      stream);
 }

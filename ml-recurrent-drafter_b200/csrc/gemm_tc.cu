@@ -258,6 +258,12 @@ struct EpiArgs {
   int64_t ss_in_ld;
   int ss_slices;
   float norm_dim, norm_eps;
+  // RD_EPI_XIELU only: the activation's two coefficients
+  float act0, act1;
+  // kEpiSplit only: output features >= n_split go to C_hi in fp32
+  float* C_hi;
+  int64_t ld_hi;
+  int n_split;
   // kEpiArgmax / kEpiSliceMax only: per (32-feature slice, token) partial results, laid out [slice][part_ld]
   float* part_val;               // kEpiSliceMax: largest stored value
   unsigned long long* part_key;  // kEpiArgmax: (order-preserving key of the largest logit) << 32 | ~(first id holding it)
@@ -272,6 +278,10 @@ constexpr int kEpiArgmax = 7;
 // that follows find its threshold from the slice maxima and read only the slices that can hold kept entries
 constexpr int kEpiSliceMax = 8;
 
+// projection whose last output features are needed unrounded: features [0, n_split) are stored as usual, features
+// [n_split, N) as fp32 in a second matrix; n_split is a multiple of 32, so a warp has one kind only
+constexpr int kEpiSplit = 10;
+
 constexpr int kScrLd = 36;  // floats per scratch row: 16-byte aligned rows, conflict-free float4 reads
 
 // Element-wise part of the epilogue in accumulator layout (lane = output feature n, i = token).
@@ -284,6 +294,10 @@ __device__ __forceinline__ void epilogue_math(float* v, const EpiArgs& e, int n,
   if (EPI == RD_EPI_BIAS_SILU || EPI == RD_EPI_BIAS_SILU_RES) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = rd::silu_f(v[i]);
+  }
+  if (EPI == RD_EPI_XIELU) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = rd::xielu_f(v[i], e.act0, e.act1);
   }
   if (EPI == RD_EPI_SWIGLU && swiglu_here) {
     // feature-per-lane stores only (the vector path forms the product after the transpose):
@@ -524,6 +538,17 @@ __device__ __forceinline__ void epilogue_block(float* v, const EpiArgs& e, float
             ((ss_red_block[tl] + ss_red_block[32 + tl]) + ss_red_block[64 + tl]) + ss_red_block[96 + tl];
     }
   }
+}
+
+// kEpiSplit: one 32-token block of the fp32 features.  Lane = feature, so every token's row piece is one
+// coalesced 128-byte store as it stands.
+__device__ __forceinline__ void epilogue_hi_block(const float* v, const EpiArgs& e, int lane, int n_warp0, int tok0, int tok_limit,
+                                                  int N) {
+  if (n_warp0 + lane >= N) return;
+  float* dst = e.C_hi + (int64_t)tok0 * e.ld_hi + (n_warp0 - e.n_split) + lane;
+#pragma unroll
+  for (int i = 0; i < 32; ++i)
+    if (tok0 + i < tok_limit) dst[(int64_t)i * e.ld_hi] = v[i];
 }
 
 // kEpiArgmax: one 32-token block of a tile.  v: accumulator values (lane = vocabulary id n_warp0 + lane,
@@ -771,7 +796,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int w_tiles = (N + BM - 1) / BM;
   const Chunking ch = make_chunking(M, w_tiles, gridDim.x);
   const int total_tiles = M > 0 ? w_tiles * ch.n_chunks : 0;
-  const int k_blocks = K / BK;
+  const int k_blocks = (K + BK - 1) / BK;  // past K the operand tiles read as zeros
 
   if (warp == 0) {
     // ---------------- TMA producer ----------------
@@ -920,6 +945,8 @@ __global__ void __launch_bounds__(kThreads, 1)
                               norm_in ? s_scale + c : nullptr);
         } else if (EPI == kEpiArgmax) {
           epilogue_argmax_block(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N);
+        } else if (EPI == kEpiSplit && n_warp0 >= epi.n_split) {
+          epilogue_hi_block(v, epi, lane, n_warp0, tok_base + c, tok_limit, N);
         } else {
           epilogue_math<EPI>(v, epi, n_warp0 + lane, N, !vec_ok, bias);
           epilogue_block<EPI, OUT_F32>(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N, vec_ok, res_cur,
@@ -1079,7 +1106,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int w_pairs = (N + 2 * BM - 1) / (2 * BM);
   const Chunking ch = make_chunking(M, w_pairs, n_pairs);
   const int all_tiles = M > 0 ? w_pairs * ch.n_chunks : 0;
-  const int k_blocks = K / BK;
+  const int k_blocks = (K + BK - 1) / BK;  // past K the operand tiles read as zeros
   // The launch lasts rounds = ceil(tiles / pairs) tile times however the tiles are dealt, so only as many
   // pairs take part as fill those rounds evenly (258 tiles on 74 pairs: 4 rounds, 65 pairs); the others
   // leave at once, and the SMs they free lower the power the busy ones share (c2 step 12.99 -> 12.97 ms).
@@ -1242,6 +1269,8 @@ __global__ void __launch_bounds__(kThreads, 1)
                               norm_in ? s_scale + c : nullptr);
         } else if (EPI == kEpiArgmax) {
           epilogue_argmax_block(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N);
+        } else if (EPI == kEpiSplit && n_warp0 >= epi.n_split) {
+          epilogue_hi_block(v, epi, lane, n_warp0, tok_base + c, tok_limit, N);
         } else {
           epilogue_math<EPI>(v, epi, n_warp0 + lane, N, !vec_ok, bias);
           epilogue_block<EPI, OUT_F32>(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N, vec_ok, res_cur,
@@ -1410,6 +1439,8 @@ int launch_epi(const GemmPlan* p, int out_dtype, const EpiArgs& e, const int32_t
     case RD_EPI_BIAS_SILU_RES: return launch_out<RD_EPI_BIAS_SILU_RES>(p, out_dtype, e, m_dev, status, s);
     case RD_EPI_RES: return launch_out<RD_EPI_RES>(p, out_dtype, e, m_dev, status, s);
     case RD_EPI_SWIGLU: return launch_out<RD_EPI_SWIGLU>(p, out_dtype, e, m_dev, status, s);
+    case RD_EPI_XIELU: return launch_out<RD_EPI_XIELU>(p, out_dtype, e, m_dev, status, s);
+    case kEpiSplit: return launch_out<kEpiSplit>(p, RD_BF16, e, m_dev, status, s);
     case kEpiQkvRope: return launch_out<kEpiQkvRope>(p, out_dtype, e, m_dev, status, s);
     case kEpiArgmax: return launch_out<kEpiArgmax>(p, out_dtype, e, m_dev, status, s);
     case kEpiSliceMax: return launch_out<kEpiSliceMax>(p, out_dtype, e, m_dev, status, s);
@@ -1420,7 +1451,7 @@ int launch_epi(const GemmPlan* p, int out_dtype, const EpiArgs& e, const int32_t
 }  // namespace
 
 extern "C" void* rd_gemm_plan_create(const void* A, int64_t lda, int m_max, const void* W, int64_t ldw, int N, int K) {
-  if (!A || !W || m_max < 1 || N < 1 || K < BK || K % BK != 0 || lda < K || ldw < K) return nullptr;
+  if (!A || !W || m_max < 1 || N < 1 || K < BK || K % 8 != 0 || lda < K || ldw < K) return nullptr;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15) || (lda * 2) % 16 || (ldw * 2) % 16) return nullptr;
   GemmPlan* p = new GemmPlan();
   p->m_max = m_max;
@@ -1455,6 +1486,31 @@ extern "C" int rd_gemm_bf16_tc(const void* plan, int out_dtype, void* C, int64_t
   e.ldr = ldr;
   cudaStream_t s = (cudaStream_t)stream;
   return launch_epi(p, out_dtype, e, m_dev, epilogue, status, s);
+}
+
+extern "C" int rd_gemm_bf16_tc_xielu(const void* plan, void* C, int64_t ldc, const int32_t* m_dev, float pos, float neg,
+                                     int32_t* status, void* stream) {
+  RD_REQUIRE(plan && C, RD_ERR_ARG);
+  EpiArgs e{};
+  e.C = C;
+  e.ldc = ldc;
+  e.act0 = pos;
+  e.act1 = neg;
+  return launch_epi(static_cast<const GemmPlan*>(plan), RD_BF16, e, m_dev, RD_EPI_XIELU, status, (cudaStream_t)stream);
+}
+
+extern "C" int rd_gemm_bf16_tc_split(const void* plan, void* C, int64_t ldc, float* C_hi, int64_t ld_hi, int n_split,
+                                     const int32_t* m_dev, int32_t* status, void* stream) {
+  RD_REQUIRE(plan && C && C_hi, RD_ERR_ARG);
+  const GemmPlan* p = static_cast<const GemmPlan*>(plan);
+  RD_REQUIRE(n_split >= 32 && n_split % 32 == 0 && n_split < p->N && ldc >= n_split && ld_hi >= p->N - n_split, RD_ERR_SIZE);
+  EpiArgs e{};
+  e.C = C;
+  e.ldc = ldc;
+  e.C_hi = C_hi;
+  e.ld_hi = ld_hi;
+  e.n_split = n_split;
+  return launch_epi(p, RD_BF16, e, m_dev, kEpiSplit, status, (cudaStream_t)stream);
 }
 
 static bool norm_in_ok(const GemmPlan* p, const float* ss_in, int64_t ss_ld, int ss_slices, int norm_dim, float eps) {

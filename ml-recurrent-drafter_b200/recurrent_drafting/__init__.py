@@ -6,13 +6,17 @@ through the C ABI of libredrafter_b200.so; there is no CPU path."""
 from . import (  # noqa: F401
     attention,
     autoregressive,
+    configuration_dilavik,
     configuration_drafter,
     kv_cache,
+    modeling_dilavik,
     modeling_drafter,
     modeling_llama,
     recurrent_drafting,
+    registry,
     replicas,
     rng,
+    session,
     stats,
     tree_attention,
 )

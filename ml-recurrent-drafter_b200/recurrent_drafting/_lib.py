@@ -35,6 +35,9 @@ SIGNATURES = {
     "rd_beam_select": (_I, [_I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P]),
     "rd_drafter_dense_log_probs": (_I, [_I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
     "rd_gemm": (_I, [_I, _I, _P, _L, _P, _L, _P, _L, _P, _P, _L, _I, _P, _I, _I, _I, _P]),
+    "rd_gemm_xielu": (_I, [_I, _P, _L, _P, _L, _P, _L, _I, _P, _I, _I, _F, _F, _P]),
+    "rd_gemm_bf16_tc_xielu": (_I, [_P, _P, _L, _P, _F, _F, _P, _P]),
+    "rd_gemm_bf16_tc_split": (_I, [_P, _P, _L, _P, _L, _I, _P, _P, _P]),
     "rd_gemm_plan_create": (_P, [_P, _L, _I, _P, _L, _I, _I]),
     "rd_gemm_plan_destroy": (None, [_P]),
     "rd_gemm_bf16_tc": (_I, [_P, _I, _P, _L, _P, _P, _L, _P, _I, _P, _P]),
@@ -66,6 +69,12 @@ SIGNATURES = {
     "rd_sample_from_sparse": (_I, [_P, _P, _P, _I, _P, _P, _P]),
     "rd_emit_tokens": (_I, [_P, _I, _P, _P, _P, _L, _I, _I, _P, _P]),
     "rd_cache_unpack": (_I, [_I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P, _P]),
+    "rd_stream_norm": (_I, [_I, _P, _P, _F, _P, _L, _P, _I, _P, _P, _P, _I, _P, _I, _I, _F, _P]),
+    "rd_rotary_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
+    "rd_attention_window": (_I, [_I, _P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _I, _P]),
+    "rd_mlstm_scan": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P]),
+    "rd_cache_commit": (_I, [_I, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _P]),
+    "rd_decode_advance": (_I, [_P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _P]),
     "rd_cache_unpack_static": (_I, [_I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P]),
 }
 

@@ -1,55 +1,59 @@
-"""Greedy one-token-per-step decoding over the same model, cache and kernels
+"""One-token-per-step decoding over the same models, caches and kernels
 (recurrent_drafting/autoregressive.py:13-53).  The comparator of the speculative loop: with greedy
 search both must produce the same tokens.
 
-As in the reference, positions are the tokens' column indices in the left-padded input (the
-reference passes arange(past, cur) without subtracting the padding, autoregressive.py:37-39)."""
-from typing import Generator
+As in the reference, a Llama token's position is its column index in the left-padded input (the
+reference passes arange(past, cur) without subtracting the padding, autoregressive.py:37-39); models
+whose positions count from each sequence's first token (positions_are_columns = False) store their
+rows without the padding."""
+from typing import Generator, Optional
 
 import torch
 
-from . import _lib, kv_cache
-from .recurrent_drafting import RecurrentDrafting, SpecialTokens, _count_left_paddings
+from . import _lib
+from .recurrent_drafting import SamplingArgs, SpecialTokens, _count_left_paddings
+from .session import DecodeGraphs, Session, graphs_enabled
 
 
 @torch.inference_mode()
-def generate(model: RecurrentDrafting, input_ids: torch.Tensor, max_length: int,
-             special_tokens: SpecialTokens) -> Generator[torch.Tensor, None, None]:
-    llm = model.llm
+def generate(model, input_ids: torch.Tensor, max_length: int, special_tokens: SpecialTokens,
+             sampling_args: SamplingArgs = SamplingArgs(1.0, True),
+             cuda_graphs: Optional[bool] = None) -> Generator[torch.Tensor, None, None]:
+    """Yields the (batch, length) token matrix after every step.  model: a RecurrentDrafting, or a base model of the
+    registry.  Steps after the second are replayed from CUDA graphs where the model allows it."""
+    llm = getattr(model, "llm", model)
     B, Lp = input_ids.shape
     dev = input_ids.device
-    cache = kv_cache.Cache(B, max_length, llm.n_layers, model.llm_n_kv_heads(), llm.head_dim, llm.dtype, dev)
-    i32 = dict(dtype=torch.int32, device=dev)
+    if not input_ids.is_cuda:
+        raise _lib.RedrafterError("input_ids must live on a CUDA device: this package has no CPU path")
     pads = _count_left_paddings(input_ids, special_tokens.pad)
-    n_new = Lp - pads
-    cols = torch.arange(Lp, device=dev)[None, :].expand(B, Lp)
-    live = cols >= pads[:, None]
+    live = torch.arange(Lp, device=dev)[None, :] >= pads[:, None]
+    first = pads.tolist()
+    assert max(first) < Lp, "a prompt row holds only padding"
+    session = Session(llm, B, max_length, begin=first if llm.positions_are_columns else None)
     tok_ids = input_ids[live].contiguous()
-    M = tok_ids.numel()
-    tok_row = torch.arange(B, device=dev)[:, None].expand(B, Lp)[live].to(torch.int32)
-    tok_slot = cols[live].to(torch.int32)
-    row_start = torch.zeros(B + 1, **i32)
-    row_start[1:] = torch.cumsum(n_new, 0).to(torch.int32)
-    kv_begin = pads.to(torch.int32)
-    kv_len = torch.zeros(B, **i32)
-    n_pos = max_length + 1
-    ws = llm.workspace(M, B)
-    hidden = llm.backbone(ws, cache._cache, M, None, tok_ids, tok_row, tok_slot, tok_slot, row_start, kv_begin, kv_len, B,
-                          Lp, Lp, _lib.ATTN_CAUSAL, n_pos=n_pos)
-    last_hidden = hidden[(row_start[1:] - 1).long()].contiguous()
-    kv_len = n_new.to(torch.int32)
+    counts = [Lp - p for p in first]
+    hidden = session.extend(tok_ids, counts)
+    ends = torch.cumsum(torch.tensor(counts), 0).sub_(1).to(dev)
+    session.last_hidden.copy_(hidden[ends])
     tokens = torch.full((B, max_length), special_tokens.pad, dtype=torch.int64, device=dev)
     tokens[:, :Lp] = input_ids
-    nxt = torch.empty(B, dtype=torch.int64, device=dev)
-    one_row = torch.arange(B, **i32)
-    step_rows = torch.arange(B + 1, **i32)
-    ws1 = llm.workspace(B, B)
+    columns = pads.to(torch.int32)
+    use_graphs = graphs_enabled(llm, cuda_graphs)
+    graphs: Optional[DecodeGraphs] = None
     length = Lp
-    V = llm.config.vocab_size
+    steps = 0
     while length < max_length:
-        logits = llm.lm_logits(last_hidden, ws1["logits"])
-        _lib.call("rd_argmax_rows", _lib.ptr(logits), logits.stride(0), B, None, V, None, _lib.ptr(nxt), _lib.stream())
-        tokens[:, length] = nxt
+        if use_graphs and graphs is None and steps == 2:
+            graphs = DecodeGraphs(session, sampling_args, tokens, columns)
+        steps += 1
+        if not sampling_args.greedy:
+            session.draw_uniforms()
+        if graphs is not None:
+            graphs.pick.replay()
+            _lib.count_replay(graphs.n_pick)
+        else:
+            session.pick(sampling_args, tokens, columns)
         length += 1
         out = tokens[:, :length].clone()
         yield out
@@ -57,7 +61,9 @@ def generate(model: RecurrentDrafting, input_ids: torch.Tensor, max_length: int,
             break
         if length >= max_length:
             break
-        slot = (kv_begin + kv_len).contiguous()
-        last_hidden = llm.backbone(ws1, cache._cache, B, None, nxt, one_row, slot, slot, step_rows, kv_begin, kv_len, B, 1,
-                                   length, _lib.ATTN_CAUSAL, n_pos=n_pos)
-        kv_len = kv_len + 1
+        if graphs is not None:
+            graphs.forward.replay()
+            _lib.count_replay(graphs.n_forward)
+        else:
+            session.forward(session.max_length if use_graphs else length)
+    session.check()

@@ -6,7 +6,8 @@ it and only grows: row b occupies slots [kv_begin[b], kv_begin[b] + kv_len[b]). 
 are device int32 vectors owned by the decode loop; the View/Cache surface below keeps the
 reference's scalar `length` semantics for callers that use the cache the reference's way.
 """
-from typing import Tuple
+from dataclasses import dataclass
+from typing import List, Sequence, Tuple, Union
 
 import torch
 
@@ -53,6 +54,19 @@ class Cache:
         self._cache = torch.zeros([n_layers, 2, batch_size, n_heads, max_length, head_dim], dtype=dtype, device=device)
         self.sliced = tuple((View(self._cache, layer, 0), View(self._cache, layer, 1)) for layer in range(n_layers))
 
+    @property
+    def storage(self) -> torch.Tensor:
+        """What the model's backbone() takes."""
+        return self._cache
+
+    @property
+    def max_length(self) -> int:
+        return self._cache.shape[4]
+
+    def set_length(self, length: int) -> None:
+        for k, v in self.sliced:
+            k.length = v.length = length
+
     def unpack(self, prompt_length: int, tree_attn_index: torch.Tensor) -> None:
         """Replicates the packed-tree K/V into per-beam layout (kv_cache.py:58-98).  The decode loop
         of this package does not need it (its commit reads the packed slots directly)."""
@@ -88,3 +102,77 @@ class Cache:
                   n_heads, max_length, head_dim, prompt_length, _lib.ptr(idx), n_flat, _lib.stream())
         for k, v in self.sliced:
             k.length = v.length = prompt_length + n_flat
+
+
+@dataclass(frozen=True)
+class KeyValueSpec:
+    """A layer that keeps keys and values of every token."""
+
+    heads: int
+    dim: int
+    vdim: int
+
+
+@dataclass(frozen=True)
+class MatrixStateSpec:
+    """A layer that keeps a matrix state of fixed size: S [heads, dim, vdim], n [heads, dim], m [heads], fp32."""
+
+    heads: int
+    dim: int
+    vdim: int
+
+
+LayerSpec = Union[KeyValueSpec, MatrixStateSpec]
+
+
+class LayerKeyValues:
+    def __init__(self, spec: KeyValueSpec, batch: int, max_length: int, dtype: torch.dtype, device):
+        self.keys = torch.zeros(batch, spec.heads, max_length, spec.dim, dtype=dtype, device=device)
+        self.values = torch.zeros(batch, spec.heads, max_length, spec.vdim, dtype=dtype, device=device)
+
+
+class LayerMatrixState:
+    def __init__(self, spec: MatrixStateSpec, batch: int, draft_tokens: int, dtype: torch.dtype, device):
+        f32 = dict(dtype=torch.float32, device=device)
+        self.S = torch.zeros(batch, spec.heads, spec.dim, spec.vdim, **f32)
+        self.n = torch.zeros(batch, spec.heads, spec.dim, **f32)
+        self.m = torch.zeros(batch, spec.heads, **f32)
+        # Projections and gates of the packed draft tokens: a verify step leaves the state alone, and the commit runs the
+        # accepted path through the recurrence from here.
+        width = 2 * spec.heads * (spec.dim + spec.vdim)
+        self.draft_proj = torch.empty(draft_tokens, (width + 7) // 8 * 8, dtype=dtype, device=device) if draft_tokens else None
+        self.draft_gates = torch.empty(draft_tokens, 2 * spec.heads, **f32) if draft_tokens else None
+
+
+class HybridCache:
+    """State of a decoder whose layers differ in what they carry from token to token.  Attention layers keep keys
+    [batch, heads, max_length, dim] and values [batch, heads, max_length, vdim], slot = position in the row; recurrent
+    layers keep their state.  Rows are independent; a row whose length is 0 starts afresh whatever its memory holds (the
+    recurrent kernels take the zero state then, and no key beyond a row's length is ever read), so giving a row back is
+    setting its length to 0."""
+
+    def __init__(self, layers: Sequence[LayerSpec], batch_size: int, max_length: int, dtype: torch.dtype, device,
+                 draft_tokens: int = 0) -> None:
+        self.max_length = max_length
+        self.batch_size = batch_size
+        self.length = 0
+        self.layers: List[Union[LayerKeyValues, LayerMatrixState]] = []
+        for spec in layers:
+            if isinstance(spec, KeyValueSpec):
+                self.layers.append(LayerKeyValues(spec, batch_size, max_length, dtype, device))
+            elif isinstance(spec, MatrixStateSpec):
+                self.layers.append(LayerMatrixState(spec, batch_size, draft_tokens, dtype, device))
+            else:
+                raise TypeError(f"unknown layer spec {spec!r}")
+
+    @property
+    def storage(self) -> "HybridCache":
+        return self
+
+    def set_length(self, length: int) -> None:
+        self.length = length
+
+    def bytes_per_token(self) -> int:
+        """Memory that grows with the sequence."""
+        return sum((l.keys[0, :, 0].numel() + l.values[0, :, 0].numel()) * l.keys.element_size()
+                   for l in self.layers if isinstance(l, LayerKeyValues))

@@ -150,7 +150,7 @@ class RecurrentDrafting(torch.nn.Module):
     def llm_n_kv_heads(self) -> int:
         if isinstance(self.llm, modeling_llama.LlamaForCausalLM):
             return self.llm.n_kv_heads
-        raise TypeError(f"Unsupported base model type {type(self.llm)}")
+        raise TypeError(f"the layers of a {type(self.llm).__name__} have no common number of key/value heads")
 
     def generate(self, ledger: stats.Ledger, input_ids: torch.Tensor, max_length: int,
                  beam_shape: modeling_drafter.BeamShape = modeling_drafter.BeamShape(10, -1),
@@ -184,8 +184,8 @@ class RecurrentDrafting(torch.nn.Module):
         st.kv_begin.zero_()
         base_len = torch.zeros(B, dtype=torch.int32, device=dev)
         ws = llm.workspace(M, B)
-        hidden = llm.backbone(ws, cache._cache, M, None, tok_ids, tok_row, tok_pos, tok_slot, row_start, st.kv_begin,
-                              base_len, B, Lp, Lp, _lib.ATTN_CAUSAL, n_pos=cache._cache.shape[4] + 1)
+        hidden = llm.backbone(ws, cache.storage, M, None, tok_ids, tok_row, tok_pos, tok_slot, row_start, st.kv_begin,
+                              base_len, B, Lp, Lp, _lib.ATTN_CAUSAL, n_pos=cache.max_length + 1)
         last = (row_start[1:] - 1).long()
         st.ctx.copy_(hidden[last])
         logits = llm.lm_logits(st.ctx, ws["logits"])
@@ -201,8 +201,7 @@ class RecurrentDrafting(torch.nn.Module):
         st.kv_len.copy_(n_new.to(torch.int32))
         # the same compaction for the token ids: column c of row b holds input_ids[b, pads[b] + c]
         st.token_buf[:, :Lp] = torch.gather(input_ids, 1, (cols + pads[:, None]).clamp_(max=Lp - 1))
-        for k, v in cache.sliced:
-            k.length = v.length = Lp
+        cache.set_length(Lp)
         return int(n_new.max().item())
 
     # One decode step = three phases that enqueue kernels and never synchronise with the host
@@ -216,8 +215,7 @@ class RecurrentDrafting(torch.nn.Module):
         llm = self.llm
         B = st.kv_begin.shape[0]
         W, Lb = beam_shape.width, beam_shape.length
-        cache_t = cache._cache
-        max_len = cache_t.shape[4]
+        max_len = cache.max_length
         fp = tree_attention.pack_flat(draft.beams, st.kv_begin, st.kv_len, out=st.fp)
         m_max = B * W * Lb
         ws = llm.workspace(m_max, m_max)
@@ -225,9 +223,8 @@ class RecurrentDrafting(torch.nn.Module):
             # On the tensor-core path the bound on the keys only decides the key-range split of the attention; it is
             # taken from the cache's capacity there, so that every step of a request launches the same kernels.
             # The CUDA-core attention sizes its shared memory by it and gets the tight bound.
-            tc_path = llm.dtype == torch.bfloat16 and llm.head_dim == 128
-            max_kv = max_len if tc_path else s_max + W * Lb
-            hidden = llm.backbone(ws, cache_t, m_max, fp.m_dev, fp.tokens, fp.tok_row, fp.tok_pos, fp.tok_slot,
+            max_kv = max_len if llm.graph_capturable else s_max + W * Lb
+            hidden = llm.backbone(ws, cache.storage, m_max, fp.m_dev, fp.tokens, fp.tok_row, fp.tok_pos, fp.tok_slot,
                                   fp.row_start, st.kv_begin, fp.base_len, B, W * Lb, max_kv, _lib.ATTN_TREE,
                                   tree_mask=fp.tree_mask, mask_words=fp.mask_words, n_pos=max_len + 1)
             fused_head = llm.fused_head_ok()
@@ -251,8 +248,12 @@ class RecurrentDrafting(torch.nn.Module):
         W, Lb = beam_shape.width, beam_shape.length
         code = _lib.dtype_code(llm.dtype)
         sm = _lib.stream()
-        cache_t = cache._cache
-        NL, _, _, nkv, max_len, hd = cache_t.shape
+        max_len = cache.max_length
+        # one tensor of equal layers: the acceptance kernel moves the accepted rows itself.  Otherwise it decides, and the
+        # model's layers commit what they keep (commit_draft below).
+        uniform = isinstance(cache, kv_cache.Cache)
+        cache_t = cache.storage if uniform else None
+        NL, nkv, hd = (cache_t.shape[0], cache_t.shape[3], cache_t.shape[5]) if uniform else (0, 0, 0)
         H = llm.config.hidden_size
         m_max = B * W * Lb
         V = logits.shape[1]
@@ -278,6 +279,7 @@ class RecurrentDrafting(torch.nn.Module):
                       _lib.ptr(st.kv_begin), _lib.ptr(fp.base_len), _lib.ptr(st.kv_len), _lib.ptr(st.token_buf),
                       _lib.ptr(st.n_accepted), _lib.ptr(st.seq_in_beam), _lib.ptr(st.init_tok), _lib.ptr(st.ctx),
                       None, sm)
+        llm.commit_draft(cache, fp, st.n_accepted, st.seq_in_beam, beam_shape, kv_begin=st.kv_begin)
 
     def _step(self, st: _DecodeState, cache: kv_cache.Cache, beam_shape, sampling_args: SamplingArgs, s_max: int,
               rec: stats.TextGeneration.Step, graphs: Optional["_StepGraphs"] = None) -> None:
@@ -304,7 +306,7 @@ class RecurrentDrafting(torch.nn.Module):
         """CUDA graphs are used on the tensor-core path when enabled (the uniforms of a sampling step are drawn
         outside the graphs, from torch's generator as without them)."""
         llm = self.llm
-        return bool(self.cuda_graphs and llm.dtype == torch.bfloat16 and llm.head_dim == 128 and llm.fused_head_ok())
+        return bool(self.cuda_graphs and llm.graph_capturable)
 
     def _generate(self, text_generation: stats.TextGeneration, input_ids: torch.Tensor, max_length: int,
                   beam_shape: modeling_drafter.BeamShape, sampling_args: SamplingArgs,
@@ -317,20 +319,12 @@ class RecurrentDrafting(torch.nn.Module):
         init_seq_len = seq_len
         W, Lb = beam_shape.width, beam_shape.length
         dev = input_ids.device
-        cache = kv_cache.Cache(
-            batch_size=B,
-            max_length=max_length + Lb * W,
-            n_layers=llm.n_layers,
-            n_heads=self.llm_n_kv_heads(),
-            head_dim=llm.head_dim,
-            dtype=llm.dtype,
-            device=dev,
-        )
+        cache = llm.new_cache(B, max_length + Lb * W, draft_tokens=B * W * Lb, device=dev)
         st = _DecodeState(llm, B, W, Lb, max_length + Lb * W, dev)
         llm.gemm_status = st.status
         self.last_state = st
         self.last_cache = cache
-        assert max_length + Lb * W <= st.token_buf.shape[1] == cache._cache.shape[4]
+        assert max_length + Lb * W <= st.token_buf.shape[1] == cache.max_length
         s_max = self._comprehend_prompt(st, cache, input_ids, sampling_args, special_tokens.pad)
         ref_len = seq_len  # the reference's padded sequence length S before the step
         graphs = _StepGraphs() if self._graphs_apply(sampling_args) else None
@@ -356,8 +350,7 @@ class RecurrentDrafting(torch.nn.Module):
                           _lib.stream())
                 self.last_ref_lengths = (ref_len, s_max)
                 ref_len = s_max
-                for k, v in cache.sliced:
-                    k.length = v.length = s_max
+                cache.set_length(s_max)
                 seq_len = out.shape[1]
                 rec.set({"input_id_length": seq_len, "avg_num_accepted": int(st.small_host[1].sum()) / B})
                 yield out[:, :max_length] if seq_len > max_length else out
