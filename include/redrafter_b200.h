@@ -421,11 +421,12 @@ RD_API int rd_rotary_append(int dtype, void* proj, int64_t ld, void* k_cache, vo
  * position p sees a key at position s <= p iff p - s < window or s < keep_first.  Cached key j sits at position j, a
  * causal new token i of a row at base_len + i; in mode RD_ATTN_TREE new tokens see each other through tree_mask and sit
  * at tok_pos [m].  q: head h of token t at q + t*ldq + h*dim; gate (optional): head h's output is multiplied by
- * sigmoid(gate[t*ld_gate + h]); out [m, nh*vdim].  vdim <= 512. */
+ * sigmoid(gate[t*ld_gate + h]); out [m, nh*vdim].  vdim <= 512.  max_kv: upper bound of base_len + new tokens; it only
+ * decides how many CTAs share a row's keys. */
 RD_API int rd_attention_window(int dtype, const void* q, int64_t ldq, const void* k_cache, const void* v_cache, const void* gate,
                         int64_t ld_gate, void* out, const int32_t* row_start, const int32_t* kv_begin, const int32_t* base_len,
                         int B, int nh, int nkv, int dim, int vdim, int max_len, int max_new, int mode, const int32_t* tok_pos,
-                        const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first, void* stream);
+                        const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first, int max_kv, void* stream);
 
 /* Matrix-memory recurrence with exponential gates over the new tokens of every row, token after token, continuing and
  * updating the row's fp32 state S [B, nh, dim, vdim], n [B, nh, dim], m [B, nh] (a row whose base_len is 0 starts from
@@ -437,6 +438,23 @@ RD_API int rd_mlstm_scan(int dtype, const void* proj, int64_t ld, const float* g
                   const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S, float* n,
                   float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int max_new,
                   const int32_t* path, int W, int Lb, const int32_t* seq, const int32_t* count, void* stream);
+
+/* The same recurrence over prompts, in chunks of 64 tokens on the tensor cores (bf16; dim <= 256, dim and vdim multiples
+ * of 8, 16-byte aligned buffers, ld a multiple of 8).  workspace: rd_mlstm_chunk_workspace_bytes() of device memory. */
+RD_API int64_t rd_mlstm_chunk_workspace_bytes(int m_max, int B, int nh, int dim, int vdim);
+RD_API int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
+                   const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S, float* n,
+                   float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int m_max,
+                   void* workspace, int64_t workspace_bytes, void* stream);
+
+/* The same recurrence over packed draft trees: every new token continues its row's state along its own ancestors
+ * (tree_mask, at most RD_MAX_BEAM_LENGTH of them, itself included); the state is left as it was.  workspace:
+ * m_max*nh*vdim floats. */
+RD_API int rd_mlstm_tree(int dtype, const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
+                  const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, const float* S,
+                  const float* n, const float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim,
+                  int vdim, int m_max, const uint32_t* tree_mask, int mask_words, float* workspace, int64_t workspace_bytes,
+                  void* stream);
 
 /* K or V rows of an accepted draft path: slot base_len[b] + unpacker[b, seq, j] moves to base_len[b] + j for j = 0 ..
  * n_accepted[b] (cache [B, nkv, max_len, dim], one call per plane). */

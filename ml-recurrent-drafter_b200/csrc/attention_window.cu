@@ -3,7 +3,9 @@
 //
 //   attention_window_rowwise_kernel  any dtype and size: one warp per (query, head), online softmax over 32 keys
 //                                    at a time, exact expf.  fp32 models and odd sizes.
-#include "attention_window.cuh"
+//   attention_window_prefill_kernel,  bf16 on warp-level tensor cores (attention_window_tc.cuh): head sizes up to 128
+//   attention_window_decode_kernel    in multiples of 8 (decode: values up to 256).
+#include "attention_window_tc.cuh"
 
 namespace {
 
@@ -93,7 +95,7 @@ extern "C" int rd_attention_window(int dtype, const void* q, int64_t ldq, const 
                                    const void* gate, int64_t ld_gate, void* out, const int32_t* row_start,
                                    const int32_t* kv_begin, const int32_t* base_len, int B, int nh, int nkv, int dim, int vdim,
                                    int max_len, int max_new, int mode, const int32_t* tok_pos, const uint32_t* tree_mask,
-                                   int mask_words, float scale, int window, int keep_first, void* stream) {
+                                   int mask_words, float scale, int window, int keep_first, int max_kv, void* stream) {
   RD_REQUIRE(q && k_cache && v_cache && out && row_start && kv_begin && base_len, RD_ERR_ARG);
   RD_REQUIRE(mode == RD_ATTN_CAUSAL || (mode == RD_ATTN_TREE && tree_mask && tok_pos && mask_words >= 1), RD_ERR_ARG);
   RD_REQUIRE(dtype == RD_F32 || dtype == RD_BF16, RD_ERR_DTYPE);
@@ -104,5 +106,19 @@ extern "C" int rd_attention_window(int dtype, const void* q, int64_t ldq, const 
                  tree_mask, mask_words, nh,   nkv, dim, vdim, max_len, mode, scale, window, keep_first};
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == RD_F32) return launch_rowwise<float>(a, B, max_new, s);
+  const uintptr_t bits = (uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out;
+  if (dim % 8 == 0 && vdim % 8 == 0 && ldq % 8 == 0 && bits % 16 == 0 && dim <= 256 && vdim <= 256) {
+    // two row tiles of queries per key/value head are still cheaper to read K and V for than one 128-query tile per head
+    const bool decode = (nh / nkv) * max_new <= 2 * rd_win::kRows;
+    if (decode) {
+      if (dim <= 64 && vdim <= 64) return rd_win::launch_decode<64, 64>(a, B, max_new, max_kv, s);
+      if (dim <= 128 && vdim <= 128) return rd_win::launch_decode<128, 128>(a, B, max_new, max_kv, s);
+      return rd_win::launch_decode<256, 256>(a, B, max_new, max_kv, s);
+    }
+    if (dim <= 64 && vdim <= 64) return rd_win::launch_prefill<64, 64>(a, B, max_new, s);
+    if (dim <= 64 && vdim <= 128) return rd_win::launch_prefill<64, 128>(a, B, max_new, s);
+    if (dim <= 128 && vdim <= 64) return rd_win::launch_prefill<128, 64>(a, B, max_new, s);
+    if (dim <= 128 && vdim <= 128) return rd_win::launch_prefill<128, 128>(a, B, max_new, s);
+  }
   return launch_rowwise<__nv_bfloat16>(a, B, max_new, s);
 }

@@ -6,13 +6,13 @@
 // followed by the RMS norm of every head's o, the norm weight and the output gate sigmoid(g).
 #include <cooperative_groups.h>
 
-#include "rd_common.cuh"
+#include "mlstm_common.cuh"
 
 namespace cg = cooperative_groups;
 
 namespace {
 
-constexpr float kDenEps = 1e-6f;
+using namespace rd_mlstm;
 
 struct MlstmArgs {
   const void* proj;     // [m, ld]: q [nh*dim] | k [nh*dim] | v [nh*vdim] | g [nh*vdim]
@@ -38,9 +38,6 @@ struct MlstmArgs {
   const int32_t* count;
   int nh, dim, vdim, slice;  // slice: value columns per CTA
 };
-
-__device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
-__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
 constexpr int kScanThreads = 256;
 
@@ -252,7 +249,157 @@ int launch_scan(const MlstmArgs& a0, int B, int max_new, cudaStream_t s) {
   return RD_OK;
 }
 
+// Packed draft trees: every new token continues the row's state along its own path of ancestors (tree_mask, itself
+// included; ascending packed index is root to leaf), and the state is left as it was.  With the path's tokens 1 .. k,
+//   num = e^(sum f + m - m_k) S^T q + sum_j e^(f_(j+1) + .. + f_k + i_j - m_k) (q . k_j) v_j
+// and the denominator likewise.  A CTA holds 64 value columns of the state in shared memory; a warp takes four tokens
+// at a time.  Writes o in fp32; launch_norm_gate() follows.
+constexpr int kTreeCols = 64;
+constexpr int kTreeTok = 4;
+constexpr int kTreeWarps = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kTreeWarps * 32) mlstm_tree_kernel(const MlstmArgs a, const uint32_t* __restrict__ tree_mask,
+                                                                    int mask_words, float* __restrict__ o_out) {
+  extern __shared__ __align__(16) float smem[];
+  rd::pdl_launch_dependents();
+  rd::pdl_wait();
+  const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * kTreeCols;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rs = a.row_start[b], n_tok = a.row_start[b + 1] - rs;
+  if (n_tok <= 0) return;
+  const int dim = a.dim, vdim = a.vdim;
+  float* S_s = smem;                                      // [dim][kTreeCols]
+  float* q_s = S_s + dim * kTreeCols + warp * dim * kTreeTok;  // [dim][kTreeTok]
+  const bool fresh = a.base_len[b] == 0;
+  const float* S_g = a.S + ((int64_t)b * a.nh + h) * dim * vdim;
+  const float* n_g = a.n + ((int64_t)b * a.nh + h) * dim;
+  for (int i = tid; i < dim * kTreeCols; i += kTreeWarps * 32) {
+    const int d = i / kTreeCols, c = c0 + i % kTreeCols;
+    S_s[i] = (c < vdim && !fresh) ? S_g[(int64_t)d * vdim + c] : 0.f;
+  }
+  __syncthreads();
+  const float m0 = fresh ? 0.f : a.m[(int64_t)b * a.nh + h];
+  const float qscale = rsqrtf((float)dim);
+  const float bi = a.bias_i[h], bf = a.bias_f[h];
+  const int ca = c0 + lane * 2;  // this lane's two value columns
+  for (int i0 = warp * kTreeTok; i0 < n_tok; i0 += kTreeWarps * kTreeTok) {
+    float nq[kTreeTok];
+#pragma unroll
+    for (int u = 0; u < kTreeTok; ++u) {
+      const T* qp = (const T*)a.proj + (int64_t)(rs + min(i0 + u, n_tok - 1)) * a.ld + (int64_t)h * dim;
+      float acc = 0.f;
+      for (int d = lane; d < dim; d += 32) {
+        const float qv = rd::Num<T>::to_f(qp[d]) * qscale;
+        q_s[d * kTreeTok + u] = qv;
+        acc = fmaf(qv, fresh ? 0.f : n_g[d], acc);
+      }
+      nq[u] = rd::warp_sum(acc);
+    }
+    __syncwarp();
+    float x[kTreeTok][2];
+#pragma unroll
+    for (int u = 0; u < kTreeTok; ++u) x[u][0] = x[u][1] = 0.f;
+    for (int d = 0; d < dim; ++d) {
+      const float2 s2 = *reinterpret_cast<const float2*>(S_s + d * kTreeCols + lane * 2);
+      const float4 q4 = *reinterpret_cast<const float4*>(q_s + d * kTreeTok);
+      const float qv[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+      for (int u = 0; u < kTreeTok; ++u) {
+        x[u][0] = fmaf(s2.x, qv[u], x[u][0]);
+        x[u][1] = fmaf(s2.y, qv[u], x[u][1]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < kTreeTok; ++u) {
+      const int i = i0 + u;
+      if (i >= n_tok) break;
+      const uint32_t* mask = tree_mask + (int64_t)(rs + i) * mask_words;
+      int anc[RD_MAX_BEAM_LENGTH];
+      float fg[RD_MAX_BEAM_LENGTH], ig[RD_MAX_BEAM_LENGTH];
+      int depth = 0;
+      float m = m0, sum_f = 0.f;
+      for (int wd = 0; wd < mask_words; ++wd) {
+        uint32_t bits = mask[wd];
+        while (bits != 0u && depth < RD_MAX_BEAM_LENGTH) {
+          const int jn = wd * 32 + __ffs(bits) - 1;
+          bits &= bits - 1u;
+          const float* gp = a.gates + (int64_t)(rs + jn) * a.ld_gates + h;
+          const float ii = soft_cap(gp[0] + bi, a.cap), ff = log_sigmoid(soft_cap(gp[a.nh] + bf, a.cap));
+          m = fmaxf(ff + m, ii);
+          sum_f += ff;
+#pragma unroll
+          for (int e = 0; e < RD_MAX_BEAM_LENGTH; ++e)
+            if (e == depth) {
+              anc[e] = jn;
+              fg[e] = ff;
+              ig[e] = ii;
+            }
+          ++depth;
+        }
+      }
+      const float inter = expf(sum_f + m0 - m);
+      float y0 = x[u][0] * inter, y1 = x[u][1] * inter, den = nq[u] * inter;
+      float tail = 0.f;  // sum of the log forget gates after token e of the path
+#pragma unroll
+      for (int e = RD_MAX_BEAM_LENGTH - 1; e >= 0; --e) {
+        if (e >= depth) continue;
+        const T* row = (const T*)a.proj + (int64_t)(rs + anc[e]) * a.ld;
+        const T* kp = row + (int64_t)(a.nh + h) * dim;
+        float dot = 0.f;
+        for (int d = lane; d < dim; d += 32) dot = fmaf(q_s[d * kTreeTok + u], rd::Num<T>::to_f(kp[d]), dot);
+        const float p = rd::warp_sum(dot) * expf(tail + ig[e] - m);
+        tail += fg[e];
+        den += p;
+        const T* vp = row + (int64_t)2 * a.nh * dim + (int64_t)h * vdim;
+        if (ca < vdim) y0 = fmaf(p, rd::Num<T>::to_f(vp[ca]), y0);
+        if (ca + 1 < vdim) y1 = fmaf(p, rd::Num<T>::to_f(vp[ca + 1]), y1);
+      }
+      const float inv = 1.0f / (fmaxf(fabsf(den), expf(-m)) + kDenEps);
+      float* dst = o_out + ((int64_t)(rs + i) * a.nh + h) * vdim;
+      if (ca < vdim) dst[ca] = y0 * inv;
+      if (ca + 1 < vdim) dst[ca + 1] = y1 * inv;
+    }
+    __syncwarp();
+  }
+}
+
+template <typename T>
+int launch_tree(const MlstmArgs& a, int B, int m_max, const uint32_t* tree_mask, int mask_words, float* o, cudaStream_t s) {
+  const size_t smem = (size_t)a.dim * (kTreeCols + kTreeWarps * kTreeTok) * sizeof(float);
+  RD_REQUIRE(smem <= 200 * 1024, RD_ERR_SIZE);
+  auto kern = mlstm_tree_kernel<T>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    RD_CHECK_CHAINED(e);
+  }
+  cudaError_t err = rd::launch_chained(kern, dim3((a.vdim + kTreeCols - 1) / kTreeCols, a.nh, B), dim3(kTreeWarps * 32), smem, s, 1, a,
+                                       tree_mask, mask_words, o);
+  RD_CHECK_CHAINED(err);
+  const T* gp = (const T*)a.proj + (int64_t)2 * a.nh * a.dim + (int64_t)a.nh * a.vdim;
+  return launch_norm_gate<T>(o, gp, a.ld, a.norm_w, a.out, a.eps, m_max, a.row_start, B, a.nh, a.dim, a.vdim, nullptr, nullptr,
+                             nullptr, s);
+}
+
 }  // namespace
+
+extern "C" int rd_mlstm_tree(int dtype, const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
+                             const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, const float* S,
+                             const float* n, const float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh,
+                             int dim, int vdim, int m_max, const uint32_t* tree_mask, int mask_words, float* workspace,
+                             int64_t workspace_bytes, void* stream) {
+  RD_REQUIRE(proj && gates && bias_i && bias_f && S && n && m && row_start && base_len && norm_weight && out && tree_mask && workspace,
+             RD_ERR_ARG);
+  RD_REQUIRE(B >= 1 && B <= 65535 && nh >= 1 && nh <= 65535 && dim >= 1 && vdim >= 1 && m_max >= 1 && gate_cap > 0.f &&
+                 mask_words >= 1 && ld >= 2 * (int64_t)nh * (dim + vdim) && ld_gates >= 2 * nh,
+             RD_ERR_SIZE);
+  RD_REQUIRE(workspace_bytes >= (int64_t)m_max * nh * vdim * (int64_t)sizeof(float), RD_ERR_CAPACITY);
+  MlstmArgs a{proj, ld,  gates, ld_gates,  bias_i,   bias_f, gate_cap, norm_weight, eps, out, const_cast<float*>(S), const_cast<float*>(n),
+              const_cast<float*>(m), row_start, base_len, nullptr, 0, 0, nullptr, nullptr, nh, dim, vdim, 0};
+  if (dtype == RD_F32) return launch_tree<float>(a, B, m_max, tree_mask, mask_words, workspace, (cudaStream_t)stream);
+  if (dtype == RD_BF16) return launch_tree<__nv_bfloat16>(a, B, m_max, tree_mask, mask_words, workspace, (cudaStream_t)stream);
+  return RD_ERR_DTYPE;
+}
 
 extern "C" int rd_mlstm_scan(int dtype, const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
                              const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S,

@@ -9,8 +9,9 @@ of tokens per step:" and "Tokens/second" lines).
 Differences that the missing network and datasets impose: prompts are token ids, either read from
 --prompt_token_ids (a text file, one request per line, ids separated by blanks or commas) or drawn
 uniformly at random (--synthetic_prompts N, the stand-in for --eval_mt_bench); --hf_llm and
---hf_drafter are checkpoint directories, or `random:NAME` (NAME in tiny, vicuna-7b, vicuna-13b) for
-random-init weights of that architecture.  A tokenizer directory is optional and only used to print
+--hf_drafter are checkpoint directories, or `random:NAME` (NAME in tiny, vicuna-7b, vicuna-13b, dilavik-tiny) for
+random-init weights of that architecture; the base model's class follows the architecture its config.json
+names (registry.py).  A tokenizer directory is optional and only used to print
 text.  There is no CPU path: --use_gpu must name a CUDA device.
 """
 import argparse
@@ -28,11 +29,24 @@ ARCHITECTURES = {
 }
 
 
+# a decoder with window attention and matrix-memory layers, small enough for a smoke run
+DILAVIK_TINY = {
+    "architecture": "Dilavik", "vocab": 1024, "width": 384, "embedding": {"scale": 1.5}, "norm": {"eps": 1e-6, "groups": 3},
+    "layers": [
+        {"type": "mlstm", "mixer": {"heads": 3, "dim": 64, "vdim": 128, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": 1024}},
+        {"type": "attention", "mixer": {"heads": 6, "kv_heads": 3, "dim": 64, "vdim": 64, "rot": {"dims": 64, "base": 10000.0},
+                                        "scale": 0.125, "mask": {"size": 128, "keep_first": 4}},
+         "mlp": {"kind": "dense", "ff": 1024}},
+    ],
+}
+
+
 def define_flags() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("--hf_tokenizer", default=None, help="Tokenizer directory (optional; only to print text).")
     ap.add_argument("--hf_llm", default="random:tiny", help="Base LLM checkpoint directory, or random:NAME.")
-    ap.add_argument("--hf_drafter", required=True, help="Drafter checkpoint directory, or random:LAYERS (residual blocks).")
+    ap.add_argument("--hf_drafter", default=None,
+                    help="Drafter checkpoint directory, or random:LAYERS (residual blocks); may be left out with --autoregression.")
     ap.add_argument("--eval_mt_bench", action="store_true", help="Accepted for compatibility: synthetic prompts are used.")
     ap.add_argument("--prompt_token_ids", default=None, help="Text file with one request per line (token ids).")
     ap.add_argument("--synthetic_prompts", type=int, default=0, help="Number of random prompts of --max_prompt_length tokens.")
@@ -92,17 +106,23 @@ def left_pad(rows: Sequence[List[int]], pad_id: int) -> torch.Tensor:
 def load_models(args, device):
     from transformers.models.llama.configuration_llama import LlamaConfig
 
-    from .. import configuration_drafter, modeling_drafter, modeling_llama
+    from .. import configuration_dilavik, configuration_drafter, modeling_dilavik, modeling_drafter, modeling_llama, registry
 
     dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}[args.dtype]
-    if args.hf_llm.startswith("random:"):
+    if args.hf_llm == "random:dilavik-tiny":
+        with torch.device(device):
+            llm = modeling_dilavik.DilavikForCausalLM(configuration_dilavik.DilavikConfig.from_dict(DILAVIK_TINY)).to(dtype)
+        llm.init_random(0.02, seed=args.rng_seed)
+    elif args.hf_llm.startswith("random:"):
         cfg = LlamaConfig(rms_norm_eps=1e-6, hidden_act="silu", pad_token_id=args.pad_token_id, **ARCHITECTURES[args.hf_llm.split(":", 1)[1]])
         cfg.rope_theta = 10000.0
         with torch.device(device):
             llm = modeling_llama.LlamaForCausalLM(cfg).to(dtype)
         llm.init_random(0.02, seed=args.rng_seed)
     else:
-        llm = modeling_llama.LlamaForCausalLM.from_pretrained(args.hf_llm, torch_dtype=dtype, device=device)
+        llm = registry.load_model(args.hf_llm, torch_dtype=dtype, device=device)
+    if args.hf_drafter is None:
+        return llm, None
     if args.hf_drafter.startswith("random:"):
         H, V = llm.config.hidden_size, llm.config.vocab_size
         dcfg = configuration_drafter.DrafterConfig(vocab_size=V, hidden_size=H, exit_dim=2 * H,
@@ -119,6 +139,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     from .. import RecurrentDrafting, SamplingArgs, SpecialTokens, autoregressive, modeling_drafter, rng, stats
 
     args = define_flags().parse_args(argv)
+    if args.hf_drafter is None and not args.autoregression:
+        print("--hf_drafter is required unless --autoregression is given", file=sys.stderr)
+        return 2
     rng.seed_pytorch(args.rng_seed)
     if args.use_gpu < 0 or not torch.cuda.is_available():
         print("this implementation has no CPU path: --use_gpu must name a CUDA device", file=sys.stderr)
@@ -126,7 +149,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     device = torch.device(f"cuda:{args.use_gpu}")
     torch.cuda.set_device(device)
     llm, drafter = load_models(args, device)
-    model = RecurrentDrafting(llm, drafter)
+    model = RecurrentDrafting(llm, drafter) if drafter is not None else llm
     special = SpecialTokens(args.pad_token_id, args.eos_token_id if args.eos_token_id >= 0 else None)
     tokenizer = None
     if args.hf_tokenizer:
@@ -146,7 +169,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     for rows in batch(prompts, args.batch_size):
         input_ids = left_pad(rows, args.pad_token_id).to(device)
         if args.autoregression:
-            outputs = autoregressive.generate(model, input_ids, max_length, special)
+            outputs = autoregressive.generate(model, input_ids, max_length, special, SamplingArgs(args.temperature, args.greedy_search))
         else:
             outputs = model.generate(ledger, input_ids, max_length, shape, SamplingArgs(args.temperature, args.greedy_search), special)
         last = None

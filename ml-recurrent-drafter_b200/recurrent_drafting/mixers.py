@@ -27,6 +27,7 @@ class StepContext:
     base_len: torch.Tensor
     batch: int
     max_new: int
+    max_kv: int  # bounds base_len + new tokens of every row; decides nothing but launch shapes
     mode: int
     tree_mask: Optional[torch.Tensor]
     mask_words: int
@@ -47,6 +48,18 @@ def row_stride(width: int) -> int:
 def rows_of(buffer: torch.Tensor, width: int) -> torch.Tensor:
     """The leading part of a workspace buffer as rows of `width` elements."""
     return buffer.view(-1)[: buffer.shape[0] * width].view(-1, width)
+
+
+class Scratch:
+    """Grow-only device memory that the layers of a model share within a launch."""
+
+    def __init__(self):
+        self._buf: Optional[torch.Tensor] = None
+
+    def get(self, nbytes: int, device) -> torch.Tensor:
+        if self._buf is None or self._buf.numel() < nbytes or self._buf.device != device:
+            self._buf = torch.empty((nbytes + 255) // 256 * 256, dtype=torch.uint8, device=device)
+        return self._buf
 
 
 class RotaryTables:
@@ -122,7 +135,7 @@ class WindowAttention(nn.Module):
         _lib.call("rd_attention_window", code, _lib.ptr(proj), ld, _lib.ptr(state.keys), _lib.ptr(state.values), _lib.ptr(gate), ld,
                   _lib.ptr(mixed), _lib.ptr(ctx.row_start), _lib.ptr(ctx.kv_begin), _lib.ptr(ctx.base_len), ctx.batch, c.heads, c.kv_heads,
                   c.dim, c.vdim, max_len, ctx.max_new, ctx.mode, _lib.ptr(ctx.tok_pos), _lib.ptr(ctx.tree_mask), ctx.mask_words,
-                  c.scale, c.window, c.keep_first, st)
+                  c.scale, c.window, c.keep_first, ctx.max_kv, st)
         self.lin[1](mixed, out, _lib.EPI_RES, residual=residual, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
 
     def commit_draft(self, state: kv_cache.LayerKeyValues, kv_begin, fp, n_accepted, seq_in_beam, beam_shape) -> None:
@@ -137,9 +150,9 @@ class WindowAttention(nn.Module):
 class MatrixMemory(nn.Module):
     """mLSTM: a matrix state per head with exponential, soft-capped gates, output normalised per head and gated."""
 
-    def __init__(self, cfg, width: int, eps: float):
+    def __init__(self, cfg, width: int, eps: float, scratch: "Scratch"):
         super().__init__()
-        self.cfg, self.eps = cfg, eps
+        self.cfg, self.eps, self.scratch = cfg, eps, scratch
         c = cfg
         self.sizes = [c.heads * c.dim, c.heads * c.dim, c.heads * c.vdim, c.heads * c.vdim]  # q, k, v, output gate
         main = sum(self.sizes)
@@ -200,17 +213,43 @@ class MatrixMemory(nn.Module):
         mixed = rows_of(ws["mixed"], self.out_width())
         self.lin[0].split(xn, proj, gates, self.n_split, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
         if tree:
-            raise _lib.RedrafterError("packed draft trees are not supported by the matrix-memory layer yet")
-        self._scan(ctx.batch, ctx.row_start, ctx.base_len, ctx.max_new, state, proj, gates, mixed)
+            self._tree(ctx, state, proj, gates, mixed)
+        elif self._chunked(ctx):
+            self._chunk(ctx, state, proj, gates, mixed)
+        else:
+            self._scan(ctx.batch, ctx.row_start, ctx.base_len, ctx.max_new, state, proj, gates, mixed)
         self.lin[1](mixed, out, _lib.EPI_RES, residual=residual, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
+
+    def _chunked(self, ctx: StepContext) -> bool:
+        """Prompts of a bf16 model; a portion shorter than a quarter of a chunk is run token by token."""
+        c = self.cfg
+        return self.w_in.dtype == torch.bfloat16 and ctx.max_new >= 16 and c.dim % 8 == 0 and c.dim <= 256 and c.vdim % 8 == 0
+
+    def _common(self, proj, gates, mixed, state, row_start, base_len):
+        c = self.cfg
+        return (_lib.ptr(proj), proj.stride(0), _lib.ptr(gates), gates.stride(0), _lib.ptr(self.bias[0]), _lib.ptr(self.bias[1]),
+                c.gate_cap, _lib.ptr(self.norm), self.eps, _lib.ptr(mixed), _lib.ptr(state.S), _lib.ptr(state.n), _lib.ptr(state.m),
+                _lib.ptr(row_start), _lib.ptr(base_len))
+
+    def _chunk(self, ctx: StepContext, state, proj, gates, mixed) -> None:
+        c = self.cfg
+        need = _lib.load().rd_mlstm_chunk_workspace_bytes(ctx.m_max, ctx.batch, c.heads, c.dim, c.vdim)
+        buf = self.scratch.get(need, proj.device)
+        _lib.call("rd_mlstm_chunk", *self._common(proj, gates, mixed, state, ctx.row_start, ctx.base_len), ctx.batch, c.heads, c.dim,
+                  c.vdim, ctx.m_max, _lib.ptr(buf), buf.numel(), _lib.stream())
+
+    def _tree(self, ctx: StepContext, state, proj, gates, mixed) -> None:
+        c = self.cfg
+        buf = self.scratch.get(4 * ctx.m_max * c.heads * c.vdim, proj.device)
+        _lib.call("rd_mlstm_tree", _lib.dtype_code(self.w_in.dtype), *self._common(proj, gates, mixed, state, ctx.row_start, ctx.base_len),
+                  ctx.batch, c.heads, c.dim, c.vdim, ctx.m_max, _lib.ptr(ctx.tree_mask), ctx.mask_words, _lib.ptr(buf), buf.numel(),
+                  _lib.stream())
 
     def _scan(self, batch, row_start, base_len, max_new, state, proj, gates, mixed, path=(None, 0, 0, None, None)) -> None:
         c = self.cfg
         p, W, Lb, seq, count = path
-        _lib.call("rd_mlstm_scan", _lib.dtype_code(self.w_in.dtype), _lib.ptr(proj), proj.stride(0), _lib.ptr(gates), gates.stride(0),
-                  _lib.ptr(self.bias[0]), _lib.ptr(self.bias[1]), c.gate_cap, _lib.ptr(self.norm), self.eps, _lib.ptr(mixed),
-                  _lib.ptr(state.S), _lib.ptr(state.n), _lib.ptr(state.m), _lib.ptr(row_start), _lib.ptr(base_len), batch, c.heads, c.dim,
-                  c.vdim, max_new, _lib.ptr(p), W, Lb, _lib.ptr(seq), _lib.ptr(count), _lib.stream())
+        _lib.call("rd_mlstm_scan", _lib.dtype_code(self.w_in.dtype), *self._common(proj, gates, mixed, state, row_start, base_len), batch,
+                  c.heads, c.dim, c.vdim, max_new, _lib.ptr(p), W, Lb, _lib.ptr(seq), _lib.ptr(count), _lib.stream())
 
     def commit_draft(self, state: kv_cache.LayerMatrixState, kv_begin, fp, n_accepted, seq_in_beam, beam_shape) -> None:
         self._scan(fp.base_len.shape[0], fp.row_start, fp.base_len, beam_shape.length, state, state.draft_proj, state.draft_gates,

@@ -16,13 +16,13 @@ from .modeling_common import Linear, LMHead
 class DecoderLayer(nn.Module):
     """norm1 + mixer, optionally norm2 + feed-forward, and the depth-average coefficients of what goes on."""
 
-    def __init__(self, cfg, index: int, model_cfg: DilavikConfig, rotary: mixers.RotaryTables):
+    def __init__(self, cfg, index: int, model_cfg: DilavikConfig, rotary: mixers.RotaryTables, scratch: mixers.Scratch):
         super().__init__()
         H = model_cfg.hidden_size
         if cfg.type == "attention":
             self.mixer = mixers.WindowAttention(cfg.mixer, H, rotary)
         else:
-            self.mixer = mixers.MatrixMemory(cfg.mixer, H, model_cfg.norm_eps)
+            self.mixer = mixers.MatrixMemory(cfg.mixer, H, model_cfg.norm_eps, scratch)
         self.mlp = mixers.DenseFeedForward(H, cfg.ff) if cfg.ff is not None else None
         self.norm1 = mixers.weight(H)
         self.norm2 = mixers.weight(H) if cfg.ff is not None else None
@@ -40,8 +40,8 @@ class DilavikForCausalLM(LMHead, nn.Module):
         self.n_layers = config.num_hidden_layers
         self.embed_tokens = nn.Embedding(config.vocab_size, H)
         self.embed_tokens.weight.requires_grad_(False)
-        self.rotary = mixers.RotaryTables()
-        self.layers = nn.ModuleList([DecoderLayer(c, i, config, self.rotary) for i, c in enumerate(config.layers)])
+        self.rotary, self.scratch = mixers.RotaryTables(), mixers.Scratch()
+        self.layers = nn.ModuleList([DecoderLayer(c, i, config, self.rotary, self.scratch) for i, c in enumerate(config.layers)])
         self.final_norm = mixers.weight(H)
         self.lm_head = nn.Linear(H, config.vocab_size, bias=False)
         self.lm_head.weight.requires_grad_(False)
@@ -237,8 +237,8 @@ class DilavikForCausalLM(LMHead, nn.Module):
         self._prepare()
         code, st = _lib.dtype_code(self.dtype), _lib.stream()
         H, groups, eps = self.config.hidden_size, self.config.norm_groups, self.config.norm_eps
-        ctx = mixers.StepContext(m_max, m_dev, tok_row, tok_pos, tok_slot, row_start, kv_begin, base_len, batch, max_new, mode,
-                                 tree_mask, mask_words, n_pos, self.gemm_status, ws)
+        ctx = mixers.StepContext(m_max, m_dev, tok_row, tok_pos, tok_slot, row_start, kv_begin, base_len, batch, max_new, max_kv,
+                                 mode, tree_mask, mask_words, n_pos, self.gemm_status, ws)
         md = _lib.ptr(m_dev)
         hist, x, mid, xn = ws["hist"], ws["x"], ws["mid"], ws["xn"]
         stride = hist.stride(0)
