@@ -2,6 +2,9 @@
 // RMS norm, depth average (a weighted sum over the results of all earlier layers), rotary embedding on a
 // part of each head with the append to a cache whose keys and values differ in size, the commit of an
 // accepted draft path to such a cache, and the bookkeeping between two decode steps.
+//
+// No pointer to data of an earlier kernel is __restrict__ here: with programmatic dependent launch a kernel is resident
+// before that data exists, and loads the compiler may take for invariant could move above pdl_wait().
 #include "rd_common.cuh"
 
 namespace {
@@ -14,9 +17,9 @@ constexpr int kNormWarps = kNormThreads / 32;
 // features: each group over its own sqrt(mean of squares + eps), the whole times w.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
-    const T* __restrict__ table, const int64_t* __restrict__ ids, float embed_scale, const float* __restrict__ hist,
-    int64_t hist_stride, const float* __restrict__ coeff, int n_hist, float* __restrict__ x_out, const T* __restrict__ w,
-    T* __restrict__ y, int m_max, const int32_t* __restrict__ m_dev, int H, int groups, int parts, float eps) {
+    const T* table, const int64_t* ids, float embed_scale, const float* hist,
+    int64_t hist_stride, const float* coeff, int n_hist, float* x_out, const T* w,
+    T* y, int m_max, const int32_t* m_dev, int H, int groups, int parts, float eps) {
   extern __shared__ float smem[];
   float* row = smem;              // [H]
   float* part_sum = smem + H;     // [groups * parts]
@@ -114,9 +117,9 @@ constexpr int kRotThreads = 256;
 
 template <typename T>
 __global__ void __launch_bounds__(kRotThreads) rotary_append_kernel(
-    T* __restrict__ proj, int64_t ld, T* __restrict__ k_cache, T* __restrict__ v_cache, const int32_t* __restrict__ tok_row,
-    const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_slot, const float* __restrict__ cos_t,
-    const float* __restrict__ sin_t, int n_pos, int m_max, const int32_t* __restrict__ m_dev, int nh, int nkv, int dim,
+    T* proj, int64_t ld, T* k_cache, T* v_cache, const int32_t* tok_row,
+    const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_t,
+    const float* sin_t, int n_pos, int m_max, const int32_t* m_dev, int nh, int nkv, int dim,
     int vdim, int rot, int max_len) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
@@ -156,12 +159,12 @@ __global__ void __launch_bounds__(kRotThreads) rotary_append_kernel(
 // base + j for j < count[b] + 1.  index rises with j and index[b, j] >= j, so ascending order never reads a
 // row it has already overwritten.  Grid (heads, B).
 template <typename T>
-__global__ void __launch_bounds__(128) cache_commit_kernel(T* __restrict__ cache, int nkv, int max_len, int dim,
-                                                           const int32_t* __restrict__ kv_begin,
-                                                           const int32_t* __restrict__ base_len,
-                                                           const int32_t* __restrict__ unpacker, int W, int Lb,
-                                                           const int32_t* __restrict__ n_accepted,
-                                                           const int32_t* __restrict__ seq_in_beam) {
+__global__ void __launch_bounds__(128) cache_commit_kernel(T* cache, int nkv, int max_len, int dim,
+                                                           const int32_t* kv_begin,
+                                                           const int32_t* base_len,
+                                                           const int32_t* unpacker, int W, int Lb,
+                                                           const int32_t* n_accepted,
+                                                           const int32_t* seq_in_beam) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int b = blockIdx.y, h = blockIdx.x;
@@ -178,10 +181,10 @@ __global__ void __launch_bounds__(128) cache_commit_kernel(T* __restrict__ cache
 
 // After the next token of every row has been chosen: it is appended to the row's token buffer and the row's
 // counters move on.
-__global__ void decode_advance_kernel(const int64_t* __restrict__ next_tok, int64_t* __restrict__ token_buf, int64_t buf_ld,
-                                      const int32_t* __restrict__ buf_begin, const int32_t* __restrict__ begin,
-                                      int32_t* __restrict__ kv_len, int32_t* __restrict__ base_len,
-                                      int32_t* __restrict__ slot, int limit, int B) {
+__global__ void decode_advance_kernel(const int64_t* next_tok, int64_t* token_buf, int64_t buf_ld,
+                                      const int32_t* buf_begin, const int32_t* begin,
+                                      int32_t* kv_len, int32_t* base_len,
+                                      int32_t* slot, int limit, int B) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int b = blockIdx.x * blockDim.x + threadIdx.x;

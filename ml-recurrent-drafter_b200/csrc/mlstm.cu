@@ -259,8 +259,8 @@ constexpr int kTreeTok = 4;
 constexpr int kTreeWarps = 8;
 
 template <typename T>
-__global__ void __launch_bounds__(kTreeWarps * 32) mlstm_tree_kernel(const MlstmArgs a, const uint32_t* __restrict__ tree_mask,
-                                                                    int mask_words, float* __restrict__ o_out) {
+__global__ void __launch_bounds__(kTreeWarps * 32) mlstm_tree_kernel(const MlstmArgs a, const uint32_t* tree_mask,
+                                                                    int mask_words, float* o_out) {
   extern __shared__ __align__(16) float smem[];
   rd::pdl_launch_dependents();
   rd::pdl_wait();

@@ -10,8 +10,9 @@
 //
 // A CTA owns VS value columns of one (row, head) and walks the row's chunks.  It keeps S^T [VS x dim] as mma
 // accumulators: warp (mt, ks) holds value columns 16 mt .. +16 and the dim range of share ks.  As accumulators turn
-// directly into A operands, S^T Q^T needs no exchange; the shares' partial outputs meet in shared memory.  What enters
-// the state, e^(...) v_j, is split into two bf16 parts (its rounding error is then about 2^-17 of it).
+// directly into A operands, S^T Q^T needs no exchange; the shares' partial outputs meet in shared memory.  The fp32
+// operands of the products - P, S and what enters the state, e^(...) v_j - are each split into two bf16 parts (their
+// rounding error is then about 2^-17).
 #include "mlstm_common.cuh"
 #include "mma_sync.cuh"
 
@@ -51,13 +52,24 @@ __device__ __forceinline__ int swz(int r, int c) {
     return r * (CH * 16) + ((c ^ ((r >> 1) & 3)) << 4);  // 4 chunks: two rows per 128 bytes
 }
 
+// x as hi + lo, both bf16
+__device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x0, x1);
+  const float2 f = __bfloat1622float2(h);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = pack_bf16(x0 - f.x, x1 - f.y);
+}
+__device__ __forceinline__ void split_store(uint8_t* hi, uint8_t* lo, int off, float x0, float x1) {
+  split2(x0, x1, *reinterpret_cast<uint32_t*>(hi + off), *reinterpret_cast<uint32_t*>(lo + off));
+}
+
 template <int DP, int VS>
 struct Layout {
   static constexpr int kQ = L * DP * 2, kV = L * VS * 2, kP = L * L * 2;
   static constexpr int kStage = 2 * kQ + kV;  // q, k, v
   static constexpr int kRed = 8 * 16 * kRedLd * 4;
   static constexpr int kMisc = (9 * L + DP + 8) * 4;
-  static constexpr int kBytes = 2 * kStage + kP + 2 * kV + kRed + kMisc;
+  static constexpr int kBytes = 2 * kStage + 2 * kP + 2 * kV + kRed + kMisc;
 };
 
 template <int DP, int VS>
@@ -80,7 +92,8 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_chunk_kernel(const ChunkArg
   if (n_tok <= 0) return;
 
   uint8_t* sP = smem + 2 * Y::kStage;
-  uint8_t* sWhi = sP + Y::kP;
+  uint8_t* sPlo = sP + Y::kP;
+  uint8_t* sWhi = sPlo + Y::kP;
   uint8_t* sWlo = sWhi + Y::kV;
   float* red = reinterpret_cast<float*>(sWlo + Y::kV);  // [8 warps][16][kRedLd]
   float* misc = red + 8 * 16 * kRedLd;
@@ -239,7 +252,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_chunk_kernel(const ChunkArg
           const float p0 = j <= t ? s[nt][hh * 2] * qs * expf(Fm + s_iF[j]) : 0.f;
           const float p1 = j + 1 <= t ? s[nt][hh * 2 + 1] * qs * expf(Fm + s_iF[j + 1]) : 0.f;
           sum[hh] += p0 + p1;
-          *reinterpret_cast<uint32_t*>(sP + swz<8>(t, j >> 3) + (j & 7) * 2) = pack_bf16(p0, p1);
+          split_store(sP, sPlo, swz<8>(t, j >> 3) + (j & 7) * 2, p0, p1);
         }
         sum[hh] += __shfl_xor_sync(0xffffffffu, sum[hh], 1);
         sum[hh] += __shfl_xor_sync(0xffffffffu, sum[hh], 2);
@@ -253,10 +266,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_chunk_kernel(const ChunkArg
       const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sV + off));
       const float w = s_w[r];
       const float x0 = v.x * w, x1 = v.y * w;
-      const __nv_bfloat162 hi = __floats2bfloat162_rn(x0, x1);
-      const float2 hf = __bfloat1622float2(hi);
-      *reinterpret_cast<__nv_bfloat162*>(sWhi + off) = hi;
-      *reinterpret_cast<__nv_bfloat162*>(sWlo + off) = __floats2bfloat162_rn(x0 - hf.x, x1 - hf.y);
+      split_store(sWhi, sWlo, off, x0, x1);
     }
     // ---- n_in . q_t: four threads per token
     {
@@ -286,18 +296,20 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_chunk_kernel(const ChunkArg
       for (int nt = 0; nt < 8; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
 #pragma unroll
       for (int kd = 0; kd < DS / 16; ++kd) {
-        uint32_t af[4];
-        af[0] = pack_bf16(S[2 * kd][0], S[2 * kd][1]);
-        af[1] = pack_bf16(S[2 * kd][2], S[2 * kd][3]);
-        af[2] = pack_bf16(S[2 * kd + 1][0], S[2 * kd + 1][1]);
-        af[3] = pack_bf16(S[2 * kd + 1][2], S[2 * kd + 1][3]);
+        uint32_t hi[4], lo[4];
+        split2(S[2 * kd][0], S[2 * kd][1], hi[0], lo[0]);
+        split2(S[2 * kd][2], S[2 * kd][3], hi[1], lo[1]);
+        split2(S[2 * kd + 1][0], S[2 * kd + 1][1], hi[2], lo[2]);
+        split2(S[2 * kd + 1][2], S[2 * kd + 1][3], hi[3], lo[3]);
 #pragma unroll
         for (int nb = 0; nb < 8; nb += 2) {
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4(b0, b1, b2, b3,
                       smem_addr(sQ + swz<CQ>(nb * 8 + ((lane >> 4) << 3) + (lane & 7), (ks * DS) / 8 + kd * 2 + ((lane >> 3) & 1))));
-          mma_bf16(o[nb], af, b0, b1);
-          mma_bf16(o[nb + 1], af, b2, b3);
+          mma_bf16(o[nb], hi, b0, b1);
+          mma_bf16(o[nb + 1], hi, b2, b3);
+          mma_bf16(o[nb], lo, b0, b1);
+          mma_bf16(o[nb + 1], lo, b2, b3);
         }
       }
 #pragma unroll
@@ -317,8 +329,12 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_chunk_kernel(const ChunkArg
                           smem_addr(sV + swz<CV>(j0 + ((lane >> 4) << 3) + (lane & 7), mt * 2 + ((lane >> 3) & 1))));
 #pragma unroll
         for (int nb = 0; nb < 8; nb += 2) {
+          const int off = swz<8>(nb * 8 + ((lane >> 4) << 3) + (lane & 7), (j0 >> 3) + ((lane >> 3) & 1));
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(b0, b1, b2, b3, smem_addr(sP + swz<8>(nb * 8 + ((lane >> 4) << 3) + (lane & 7), (j0 >> 3) + ((lane >> 3) & 1))));
+          ldmatrix_x4(b0, b1, b2, b3, smem_addr(sP + off));
+          mma_bf16(o[nb], af, b0, b1);
+          mma_bf16(o[nb + 1], af, b2, b3);
+          ldmatrix_x4(b0, b1, b2, b3, smem_addr(sPlo + off));
           mma_bf16(o[nb], af, b0, b1);
           mma_bf16(o[nb + 1], af, b2, b3);
         }

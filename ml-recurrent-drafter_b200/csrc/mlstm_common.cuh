@@ -15,9 +15,9 @@ constexpr int kNormThreads = 256;
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kNormThreads) norm_gate_kernel(
-    const float* __restrict__ o, const T* __restrict__ g, int64_t ld, const T* __restrict__ w, T* __restrict__ out, float eps,
-    const int32_t* __restrict__ row_start, int B, int nh, int dim, int vdim, const float* __restrict__ nm, float* __restrict__ n,
-    float* __restrict__ m) {
+    const float* o, const T* g, int64_t ld, const T* w, T* out, float eps,
+    const int32_t* row_start, int B, int nh, int dim, int vdim, const float* nm, float* n,
+    float* m) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;

@@ -102,7 +102,9 @@ __device__ __forceinline__ int live_rows(const int* m_dev, int m_max) {
 // previous kernel of the stream has finished: it must execute pdl_wait() before its first access to
 // global memory (reads of the predecessor's results and writes to anything the predecessor may still
 // read), and it lets its own successor start early with pdl_launch_dependents().  Both are no-ops
-// in a kernel that was launched the ordinary way.
+// in a kernel that was launched the ordinary way.  Data of an earlier kernel must not be read through a const
+// __restrict__ pointer in straight-line code after the wait: the compiler may treat such loads as invariant and
+// hoist them above it (a commit kernel read the previous step's acceptance that way once its launch overlapped).
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 

@@ -140,7 +140,7 @@ class LayerMatrixState:
         # Projections and gates of the packed draft tokens: a verify step leaves the state alone, and the commit runs the
         # accepted path through the recurrence from here.
         width = 2 * spec.heads * (spec.dim + spec.vdim)
-        self.draft_proj = torch.empty(draft_tokens, (width + 7) // 8 * 8, dtype=dtype, device=device) if draft_tokens else None
+        self.draft_proj = torch.empty(draft_tokens, (width + 31) // 32 * 32, dtype=dtype, device=device) if draft_tokens else None
         self.draft_gates = torch.empty(draft_tokens, 2 * spec.heads, **f32) if draft_tokens else None
 
 

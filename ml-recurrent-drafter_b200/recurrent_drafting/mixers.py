@@ -206,7 +206,8 @@ class MatrixMemory(nn.Module):
         if tree:
             # kept until the accepted path is committed
             proj, gates = state.draft_proj, state.draft_gates
-            assert proj is not None and proj.shape[0] >= ctx.m_max, "the cache was made without room for draft tokens"
+            if proj is None or proj.shape[0] < ctx.m_max or proj.shape[1] < self.n_split:
+                raise _lib.RedrafterError("the cache was made without room for these draft tokens")
         else:
             proj = rows_of(ws["proj"], ld)
             gates = rows_of(ws["gates"], 2 * c.heads)

@@ -134,7 +134,7 @@ def test_edges_of_the_window_and_the_first_tokens_move_the_logits(dt, decode):
     from recurrent_drafting.session import Session
 
     keep, size, T = 3, 40, 130
-    cfg = db.config([db.attention(4, 2, 32, 24, 16, 5000.0, 0.6, size, keep, ff=None)], vocab=64)
+    cfg = db.config([db.attention(4, 2, 32, 24, 16, 5000.0, 0.05, size, keep, ff=None)], vocab=64)
     cfg, w, llm = pair(cfg, dt)
     ids = db.tokens(cfg, T, 3)
     q = T - 1
@@ -148,9 +148,10 @@ def test_edges_of_the_window_and_the_first_tokens_move_the_logits(dt, decode):
         moved = np.abs(feed(s, 0, other, sizes)[q] - base).max()
         expect = np.abs(dilavik.forward(w, cfg, other)[q] - dilavik.forward(w, cfg, ids)[q]).max()
         seen = j < keep or q - j < size
-        assert (expect > 1e-6) == seen
+        assert (expect > 1e-9) == seen
+        assert expect == 0 or expect > 0.02
         assert (moved > 0) == seen, (j, moved)
-        assert abs(moved - expect) < (1e-3 if dt == "fp32" else 0.15) * max(expect, 0.1)
+        assert abs(moved - expect) < (1e-3 if dt == "fp32" else 0.5) * expect + 1e-9
 
 
 def test_long_decoding_stays_on_the_plain_recurrence():
@@ -162,7 +163,7 @@ def test_long_decoding_stays_on_the_plain_recurrence():
     assert db.error(got, dilavik.forward(w, cfg, ids)) < 3e-5
     cfg, w, llm = pair("mixed", "bf16")
     got = feed(Session(llm, 1, 700), 0, ids, [100] + [1] * 600)
-    assert db.error(got, dilavik.forward(w, cfg, ids)) < TOL["bf16"]
+    assert db.error(got, dilavik.forward(w, cfg, ids)) < 1.5 * TOL["bf16"]  # the worst of 700 positions
 
 
 # ------------------------------------------------------------------------------------------ generation
@@ -265,7 +266,8 @@ class PlantedDrafter(torch.nn.Module):
             true = (self.rows[b][at : at + L] + [3] * L)[:L]
             assert int(init_tok[b]) == true[0]
             for i in range(W):
-                hit = 1 + (self.steps + b + i) % L if i != 1 else 1 + (self.steps + 2 * b) % L
+                hit = 1 + (self.steps + b) % L  # the longest right prefix of this step, in beam 1; shorter ones elsewhere
+                hit = hit if i == 1 else max(1, hit - 1 - i)
                 beams[b, i] = torch.tensor(true[:hit] + [3 + (7 * i + self.steps + k) % (self.cfg["vocab"] - 3) for k in range(L - hit)])
         self.steps += 1
 
