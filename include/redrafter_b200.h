@@ -199,6 +199,14 @@ RD_API int rd_gemm_bf16_tc_qkv_rope(const void* plan, const int32_t* m_dev, void
                              const float* cos_table, const float* sin_table, int n_pos, int nh, int nkv, int hd,
                              int max_len, int32_t* status, void* stream);
 
+/* The same for models with an output gate per head and rotary embedding on a part of each head: the packed weight has nh
+ * further rows (the gates, written to gate_out [m, ld_gate] as they are), feature i of a head is paired with i + rot_dims/2
+ * for i < rot_dims/2 (rot_dims a multiple of 16), and the tables [n_pos, 128] hold cos 1 / sin 0 past rot_dims. */
+RD_API int rd_gemm_bf16_tc_qkvg_rope(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,
+                              void* gate_out, int64_t ld_gate, const int32_t* tok_row, const int32_t* tok_pos,
+                              const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos, int nh, int nkv,
+                              int hd, int rot_dims, int max_len, int32_t* status, void* stream);
+
 /* LlamaRMSNorm (modeling_llama.py:21-34) folded into the two GEMMs around it, so that the norm between a residual
  * projection and the next projection needs no kernel of its own (bf16, tensor-core path).
  * rd_gemm_bf16_tc_res_norm (producer): C = A W^T + R as RD_EPI_RES; besides, C2[t, n] = bf16(C[t, n]) * gamma[n] and
@@ -286,6 +294,13 @@ RD_API void* rd_attention_plan_create(const void* q, int m_max, const void* k_ca
 RD_API void rd_attention_plan_destroy(void* plan);
 RD_API int rd_attention_tc(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
                            const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
+                           int32_t* status, void* stream);
+
+/* rd_attention_tc with the visibility and the gate of rd_attention_window (see there); scale > 0; in mode RD_ATTN_TREE the
+ * window is at least RD_MAX_BEAM_LENGTH. */
+RD_API int rd_attention_tc_window(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
+                           const int32_t* base_len, int max_new, int mode, const int32_t* tok_pos, const uint32_t* tree_mask,
+                           int mask_words, float scale, int window, int keep_first, const void* gate, int64_t ld_gate,
                            int32_t* status, void* stream);
 
 /* rd_attention_tc with the key range of every (row, head) cut into n_split shares (1..RD_ATTN_MAX_SPLIT), one CTA
@@ -439,13 +454,14 @@ RD_API int rd_mlstm_scan(int dtype, const void* proj, int64_t ld, const float* g
                   float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int max_new,
                   const int32_t* path, int W, int Lb, const int32_t* seq, const int32_t* count, void* stream);
 
-/* The same recurrence over prompts, in chunks of 64 tokens on the tensor cores (bf16; dim <= 256, dim and vdim multiples
- * of 8, 16-byte aligned buffers, ld a multiple of 8).  workspace: rd_mlstm_chunk_workspace_bytes() of device memory. */
+/* The same recurrence over prompts, in chunks of 128 tokens on the tensor cores (bf16; dim <= 256, vdim <= 512, both
+ * multiples of 8, 16-byte aligned buffers, ld a multiple of 8).  max_new bounds the new tokens of a row.  workspace:
+ * rd_mlstm_chunk_workspace_bytes() of device memory, 16-byte aligned. */
 RD_API int64_t rd_mlstm_chunk_workspace_bytes(int m_max, int B, int nh, int dim, int vdim);
 RD_API int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
                    const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S, float* n,
                    float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int m_max,
-                   void* workspace, int64_t workspace_bytes, void* stream);
+                   int max_new, void* workspace, int64_t workspace_bytes, void* stream);
 
 /* The same recurrence over packed draft trees: every new token continues its row's state along its own ancestors
  * (tree_mask, at most RD_MAX_BEAM_LENGTH of them, itself included); the state is left as it was.  workspace:

@@ -182,13 +182,23 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// WIN: sliding window with kept first tokens and an output gate per head.  Only the key tiles that hold a kept token or lie
+// in some query's window are visited.
+struct WindowArgs {
+  int window, keep_first;
+  const __nv_bfloat16* gate;  // optional [m, ld_gate]
+  int64_t ld_gate;
+  const int32_t* tok_pos;     // tree mode: positions of the new tokens
+};
+
+template <bool WIN>
 __global__ void __launch_bounds__(kThreads, 2)
     attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                           const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                           const int32_t* __restrict__ row_start, const int32_t* __restrict__ kv_begin,
                           const int32_t* __restrict__ base_len, int nh, int nkv, int max_len, int mode,
                           const uint32_t* __restrict__ tree_mask, int mask_words, float scale_log2, int32_t* status,
-                          int n_split, float* __restrict__ partial) {
+                          int n_split, float* __restrict__ partial, const WindowArgs win) {
   const int b = blockIdx.z, h = blockIdx.y;
   rd::pdl_launch_dependents();
   if (threadIdx.x == 0) {
@@ -223,7 +233,14 @@ __global__ void __launch_bounds__(kThreads, 2)
   const int base = base_len[b];
   const int hk = h / (nh / nkv);
   const int kv_end = (mode == RD_ATTN_CAUSAL) ? base + min(n_new, q0 + BMQ) : base + n_new;
-  const int all_tiles = (kv_end + BNK - 1) / BNK;
+  int all_tiles = (kv_end + BNK - 1) / BNK;
+  int kept_tiles = 0, first_tile = 0;  // WIN: tiles of the kept tokens, then [first_tile, end)
+  if (WIN) {
+    const int lo = base + (mode == RD_ATTN_CAUSAL ? q0 : 0) - win.window + 1;
+    first_tile = lo > 0 ? lo / BNK : 0;
+    kept_tiles = min((min(win.keep_first, kv_end) + BNK - 1) / BNK, first_tile);
+    all_tiles += kept_tiles - first_tile;
+  }
   const int per_split = (all_tiles + n_split - 1) / n_split;
   const int t_begin = split * per_split;  // first key tile of this CTA
   const int n_tiles = max(0, min(per_split, all_tiles - t_begin));
@@ -237,6 +254,11 @@ __global__ void __launch_bounds__(kThreads, 2)
     }
     return;
   }
+  // key tile of this CTA's step t
+  auto tile_of = [&](int t) {
+    const int u = t_begin + t;
+    return (WIN && u >= kept_tiles) ? u - kept_tiles + first_tile : u;
+  };
   const int kv_row0 = (b * nkv + hk) * max_len + kv_begin[b];  // row of key 0 in the [B*nkv*max_len, 128] view
 
   if (threadIdx.x == 0) {
@@ -258,14 +280,14 @@ __global__ void __launch_bounds__(kThreads, 2)
     tma_load_2d(sQ, &map_q, q_full, h * HD, rs + q0);
     tma_load_2d(sQ + BMQ * 128, &map_q, q_full, h * HD + 64, rs + q0);
     for (int t = 0; t < kStages && t < n_tiles; ++t) {
-      const int row = kv_row0 + (t_begin + t) * BNK;
+      const int row = kv_row0 + tile_of(t) * BNK;
       uint8_t* dk = sKV + t * kKVStage;
       mbar_expect_tx(&k_full[t], 2 * kSubTile);
       tma_load_2d(dk, &map_k, &k_full[t], 0, row);
       tma_load_2d(dk + kSubTile, &map_k, &k_full[t], 64, row);
     }
     for (int t = 0; t < kStages && t < n_tiles; ++t) {
-      const int row = kv_row0 + (t_begin + t) * BNK;
+      const int row = kv_row0 + tile_of(t) * BNK;
       uint8_t* dv = sKV + t * kKVStage + 2 * kSubTile;
       mbar_expect_tx(&v_full[t], 2 * kSubTile);
       tma_load_2d(dv, &map_v, &v_full[t], 0, row);
@@ -300,7 +322,7 @@ __global__ void __launch_bounds__(kThreads, 2)
         }
         uint8_t* dst = sKV + s * kKVStage + (is_k ? 0 : 2 * kSubTile);
         mbar_expect_tx(&full[s], 2 * kSubTile);
-        const int row = kv_row0 + (t_begin + t) * BNK;
+        const int row = kv_row0 + tile_of(t) * BNK;
         tma_load_2d(dst, map, &full[s], 0, row);
         tma_load_2d(dst + kSubTile, map, &full[s], 64, row);
       }
@@ -397,7 +419,7 @@ __global__ void __launch_bounds__(kThreads, 2)
       __syncwarp();
       if (lane == 0) mbar_arrive(s_empty);
       // visibility of the tile's 64 keys for this row as one 64-bit word
-      const int j0 = (t_begin + t) * BNK;
+      const int j0 = tile_of(t) * BNK;
       uint64_t vis;
       if (j0 + BNK <= base) {
         vis = ~0ull;  // the whole tile lies in the cached prefix
@@ -421,6 +443,14 @@ __global__ void __launch_bounds__(kThreads, 2)
       if (j0 + BNK > kv_end) {
         const int n_in = kv_end - j0;  // 1..63 keys of the tile exist
         vis &= (n_in <= 0) ? 0ull : ((1ull << n_in) - 1ull);
+      }
+      if (WIN) {
+        // position of the query; keys before p - window + 1 are gone unless they are among the kept ones
+        const int p = mode == RD_ATTN_CAUSAL ? base + qi : (live ? win.tok_pos[rs + qi] : base);
+        const int gone = p - win.window + 1 - j0, kept = win.keep_first - j0;
+        const uint64_t in_window = gone <= 0 ? ~0ull : (gone >= 64 ? 0ull : ~0ull << gone);
+        const uint64_t among_kept = kept <= 0 ? 0ull : (kept >= 64 ? ~0ull : (1ull << kept) - 1ull);
+        vis &= in_window | among_kept;
       }
       // Running max over the RAW scores (the scale is positive), masked keys set to -inf first.
       // exp2 then takes one FFMA per element: p = 2^(s*scale - m*scale).
@@ -516,7 +546,8 @@ __global__ void __launch_bounds__(kThreads, 2)
       }
     } else if (ok) {
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      if (WIN && win.gate != nullptr && live) inv /= 1.0f + __expf(-__bfloat162float(win.gate[(int64_t)(rs + qi) * win.ld_gate + h]));
       uint4* dst = reinterpret_cast<uint4*>(out + ((int64_t)(rs + qi) * nh + h) * HD);
 #pragma unroll 1
       for (int c = 0; c < HD / 32; ++c) {
@@ -617,7 +648,8 @@ extern "C" int64_t rd_attention_split_workspace_bytes(int m_max, int nh, int n_s
 
 static int attention_tc_launch(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
                                const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
-                               int n_split, void* workspace, int64_t workspace_bytes, int32_t* status, void* stream) {
+                               int n_split, void* workspace, int64_t workspace_bytes, int32_t* status, void* stream,
+                               const WindowArgs* win, float scale) {
   RD_REQUIRE(plan && out && row_start && kv_begin && base_len, RD_ERR_ARG);
   RD_REQUIRE(mode == RD_ATTN_CAUSAL || (mode == RD_ATTN_TREE && tree_mask && mask_words >= 1 && mask_words <= kMaxMaskWords),
              RD_ERR_ARG);
@@ -629,17 +661,17 @@ static int attention_tc_launch(const void* plan, void* out, const int32_t* row_s
     RD_REQUIRE(workspace && ((uintptr_t)workspace & 15) == 0, RD_ERR_ARG);
     RD_REQUIRE(workspace_bytes >= rd_attention_split_workspace_bytes(p->m_max, p->nh, n_split), RD_ERR_CAPACITY);
   }
-  auto kern = attention_umma_kernel;
-  static bool smem_set = false;  // set once, so that steady-state launches are pure launches
-  if (!smem_set) {
+  auto kern = win ? attention_umma_kernel<true> : attention_umma_kernel<false>;
+  static bool smem_set[2] = {false, false};  // set once each, so that steady-state launches are pure launches
+  if (!smem_set[win != nullptr]) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
-    smem_set = true;
+    smem_set[win != nullptr] = true;
   }
   dim3 grid(((max_new + BMQ - 1) / BMQ) * n_split, p->nh, p->B);
-  const float scale_log2 = 1.4426950408889634f / sqrtf((float)HD);
+  const float scale_log2 = 1.4426950408889634f * scale;
   cudaError_t err = rd::launch_chained(kern, grid, dim3(kThreads), kSmemBytes, (cudaStream_t)stream, 1, p->map_q, p->map_k, p->map_v,
                                        (__nv_bfloat16*)out, row_start, kv_begin, base_len, p->nh, p->nkv, p->max_len, mode,
-                                       tree_mask, mask_words, scale_log2, status, n_split, (float*)workspace);
+                                       tree_mask, mask_words, scale_log2, status, n_split, (float*)workspace, win ? *win : WindowArgs{});
   RD_CHECK_CHAINED(err);
   if (n_split > 1) {
     attention_merge_kernel<<<dim3(p->m_max, p->nh), HD, 0, (cudaStream_t)stream>>>((const float*)workspace, (__nv_bfloat16*)out,
@@ -657,12 +689,24 @@ extern "C" int rd_attention_tc(const void* plan, void* out, const int32_t* row_s
                                const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
                                int32_t* status, void* stream) {
   return attention_tc_launch(plan, out, row_start, kv_begin, base_len, max_new, mode, tree_mask, mask_words, 1, nullptr, 0,
-                             status, stream);
+                             status, stream, nullptr, 1.0f / sqrtf((float)HD));
 }
 
 extern "C" int rd_attention_tc_split(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
                                      const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
                                      int n_split, void* workspace, int64_t workspace_bytes, int32_t* status, void* stream) {
   return attention_tc_launch(plan, out, row_start, kv_begin, base_len, max_new, mode, tree_mask, mask_words, n_split, workspace,
-                             workspace_bytes, status, stream);
+                             workspace_bytes, status, stream, nullptr, 1.0f / sqrtf((float)HD));
+}
+
+extern "C" int rd_attention_tc_window(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
+                                      const int32_t* base_len, int max_new, int mode, const int32_t* tok_pos,
+                                      const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first,
+                                      const void* gate, int64_t ld_gate, int32_t* status, void* stream) {
+  // the kernel's running maximum is taken before the scale, and a tree's own tokens must lie inside every window
+  RD_REQUIRE(scale > 0.f && window >= (mode == RD_ATTN_TREE ? RD_MAX_BEAM_LENGTH : 1) && keep_first >= 0, RD_ERR_SIZE);
+  RD_REQUIRE(mode != RD_ATTN_TREE || tok_pos, RD_ERR_ARG);
+  const WindowArgs win{window, keep_first, (const __nv_bfloat16*)gate, ld_gate, tok_pos};
+  return attention_tc_launch(plan, out, row_start, kv_begin, base_len, max_new, mode, tree_mask, mask_words, 1, nullptr, 0, status,
+                             stream, &win, scale);
 }

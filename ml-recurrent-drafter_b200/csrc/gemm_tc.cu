@@ -242,6 +242,9 @@ struct EpiArgs {
   const float* cos_t;
   const float* sin_t;
   int n_pos, nh, nkv, max_len;
+  int rot_half;               // rotated pairs per head (64 = the whole head): feature i is paired with i + rot_half
+  __nv_bfloat16* gate_out;    // output features past the v heads (one per query head): [tok, ld_gate], plain
+  int64_t ld_gate;
   // LlamaRMSNorm folded into the two GEMMs around it (optional; bf16 output, N a multiple of 32).
   // Producer (residual epilogues, gamma != nullptr): besides C the kernel writes C2 = bf16(C) * gamma and, per token
   // and 128-feature slice (a CTA's rows), the sum of squares of the rounded C values to
@@ -638,7 +641,7 @@ __device__ __forceinline__ void norm_scale_stage(const EpiArgs& e, float* s_scal
 
 // Epilogue block of the QKV projection with fused rotary embedding (head_dim 128 = one CTA's 128
 // weight rows = one head).  v: this lane's feature d = 32*quarter + lane for the block's 32 tokens.
-// The rotation pairs feature d with d +- 64, which lives in the warp two quarters away, so the four
+// The rotation pairs feature d with d +- rot_half, which may live in another warp, so the four
 // epilogue warps exchange their transposed blocks through the scratch and meet at a named barrier.
 // Values are rounded to bf16 first, as a separate projection would have stored them, so the result
 // equals projection -> rope bit for bit.  After the exchange four lanes share a token row (8 features
@@ -650,7 +653,9 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
   const bool is_v = head >= e.nh + e.nkv;
   const int sub = lane & 3, row0 = lane >> 2;
   const int d0 = quarter * 32 + sub * 8;
-  const float sign = quarter < 2 ? -1.0f : 1.0f;  // rotate_half: (-x2, x1)
+  const float sign = d0 < e.rot_half ? -1.0f : 1.0f;  // rotate_half: (-x2, x1)
+  // this lane's eight features are paired with those at pd (unrotated features with themselves: their sines are 0)
+  const int pd = d0 < e.rot_half ? d0 + e.rot_half : (d0 < 2 * e.rot_half ? d0 - e.rot_half : d0);
   // the cos/sin rows of the block's tokens are requested first (volatile asm keeps them here): their latency
   // runs under the transposition and the exchange below
   float4 cs[4][4];
@@ -689,7 +694,7 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
       for (int j = 0; j < 8; ++j) o[p][j] = __bfloat162float(__float2bfloat16_rn(o[p][j] * sc));
     }
     if (!is_v) {
-      const float* oth = scr_all + (quarter ^ 2) * 32 * kScrLd + r * kScrLd + sub * 8;
+      const float* oth = scr_all + (pd >> 5) * 32 * kScrLd + r * kScrLd + (pd & 31);
       float4 b0 = *reinterpret_cast<const float4*>(oth), b1 = *reinterpret_cast<const float4*>(oth + 4);
       if (s_scale != nullptr) {
         b0.x = __bfloat162float(__float2bfloat16_rn(b0.x * sc)), b0.y = __bfloat162float(__float2bfloat16_rn(b0.y * sc));
@@ -727,6 +732,14 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
       *reinterpret_cast<uint4*>(dst) = pk;
     }
   }
+}
+
+// Output features past the v heads, one per query head: lane = feature, a token's piece is one coalesced store.
+__device__ __forceinline__ void epilogue_gate_block(const float* v, const EpiArgs& e, int lane, int f0, int tok0, int tok_limit) {
+  if (f0 + lane >= e.nh) return;
+#pragma unroll
+  for (int i = 0; i < 32; ++i)
+    if (tok0 + i < tok_limit) e.gate_out[(int64_t)(tok0 + i) * e.ld_gate + f0 + lane] = __float2bfloat16_rn(v[i]);
 }
 
 struct SmemLayout {
@@ -940,7 +953,9 @@ __global__ void __launch_bounds__(kThreads, 1)
         float v[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-        if (EPI == kEpiQkvRope) {
+        if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
+          epilogue_gate_block(v, epi, lane, n_warp0 - (epi.nh + 2 * epi.nkv) * 128, tok_base + c, tok_limit);
+        } else if (EPI == kEpiQkvRope) {
           epilogue_rope_block(v, epi, scratch, quarter, lane, rope_head, tok_base + c, tok_limit, s_pos + c, s_dst + c,
                               norm_in ? s_scale + c : nullptr);
         } else if (EPI == kEpiArgmax) {
@@ -1264,7 +1279,9 @@ __global__ void __launch_bounds__(kThreads, 1)
         float v[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-        if (EPI == kEpiQkvRope) {
+        if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
+          epilogue_gate_block(v, epi, lane, n_warp0 - (epi.nh + 2 * epi.nkv) * 128, tok_base + c, tok_limit);
+        } else if (EPI == kEpiQkvRope) {
           epilogue_rope_block(v, epi, scratch, quarter, lane, rope_head, tok_base + c, tok_limit, s_pos + c, s_dst + c,
                               norm_in ? s_scale + c : nullptr);
         } else if (EPI == kEpiArgmax) {
@@ -1561,11 +1578,12 @@ extern "C" int rd_gemm_bf16_tc_swiglu_normed(const void* plan, void* C, int64_t 
 static int qkv_rope_launch(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,
                            const int32_t* tok_row, const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_table,
                            const float* sin_table, int n_pos, int nh, int nkv, int hd, int max_len, const float* ss_in,
-                           int64_t ss_ld, int ss_slices, int norm_dim, float eps, int32_t* status, void* stream) {
+                           int64_t ss_ld, int ss_slices, int norm_dim, float eps, int32_t* status, void* stream,
+                           int rot_dims = 128, void* gate_out = nullptr, int64_t ld_gate = 0) {
   RD_REQUIRE(plan && q_out && k_cache && v_cache && tok_row && tok_pos && tok_slot && cos_table && sin_table, RD_ERR_ARG);
   const GemmPlan* p = static_cast<const GemmPlan*>(plan);
   RD_REQUIRE(hd == 128 && nh >= 1 && nkv >= 1 && n_pos >= 1 && max_len >= 1, RD_ERR_SIZE);
-  RD_REQUIRE(p->N == (nh + 2 * nkv) * hd, RD_ERR_SIZE);
+  RD_REQUIRE(p->N == (nh + 2 * nkv) * hd + (gate_out ? nh : 0) && rot_dims % 16 == 0 && rot_dims >= 0 && rot_dims <= hd, RD_ERR_SIZE);
   RD_REQUIRE((((uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos_table | (uintptr_t)sin_table) & 15) == 0,
              RD_ERR_ALIGN);
   EpiArgs e{};
@@ -1583,6 +1601,9 @@ static int qkv_rope_launch(const void* plan, const int32_t* m_dev, void* q_out, 
   e.nh = nh;
   e.nkv = nkv;
   e.max_len = max_len;
+  e.rot_half = rot_dims / 2;
+  e.gate_out = (__nv_bfloat16*)gate_out;
+  e.ld_gate = ld_gate;
   if (ss_in) {
     RD_REQUIRE(norm_in_ok(p, ss_in, ss_ld, ss_slices, norm_dim, eps), RD_ERR_SIZE);
     e.ss_in = ss_in;
@@ -1600,6 +1621,15 @@ extern "C" int rd_gemm_bf16_tc_qkv_rope(const void* plan, const int32_t* m_dev, 
                                         int max_len, int32_t* status, void* stream) {
   return qkv_rope_launch(plan, m_dev, q_out, k_cache, v_cache, tok_row, tok_pos, tok_slot, cos_table, sin_table, n_pos, nh, nkv,
                          hd, max_len, nullptr, 0, 0, 0, 0.f, status, stream);
+}
+
+extern "C" int rd_gemm_bf16_tc_qkvg_rope(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,
+                                         void* gate_out, int64_t ld_gate, const int32_t* tok_row, const int32_t* tok_pos,
+                                         const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos,
+                                         int nh, int nkv, int hd, int rot_dims, int max_len, int32_t* status, void* stream) {
+  RD_REQUIRE(gate_out && ld_gate >= nh, RD_ERR_ARG);
+  return qkv_rope_launch(plan, m_dev, q_out, k_cache, v_cache, tok_row, tok_pos, tok_slot, cos_table, sin_table, n_pos, nh, nkv,
+                         hd, max_len, nullptr, 0, 0, 0, 0.f, status, stream, rot_dims, gate_out, ld_gate);
 }
 
 extern "C" int rd_gemm_bf16_tc_qkv_rope_normed(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,

@@ -9,14 +9,13 @@
 
 namespace {
 
-constexpr int kNormThreads = 256;
-constexpr int kNormWarps = kNormThreads / 32;
+constexpr int kNormMaxThreads = 1024;
 
 // One block per token.  The row is formed in fp32 (embedding gather, or the weighted sum of `n_hist` stored
 // rows), written to x when asked for, kept in shared memory, and normalised in groups of H / groups
 // features: each group over its own sqrt(mean of squares + eps), the whole times w.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
+__global__ void __launch_bounds__(kNormMaxThreads) stream_norm_kernel(
     const T* table, const int64_t* ids, float embed_scale, const float* hist,
     int64_t hist_stride, const float* coeff, int n_hist, float* x_out, const T* w,
     T* y, int m_max, const int32_t* m_dev, int H, int groups, int parts, float eps) {
@@ -27,16 +26,16 @@ __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
   rd::pdl_wait();
   const int t = blockIdx.x;
   if (t >= rd::live_rows(m_dev, m_max)) return;
-  const int tid = threadIdx.x;
+  const int tid = threadIdx.x, n_thr = blockDim.x;
   if (table != nullptr) {
     const T* src = table + ids[t] * (int64_t)H;
-    for (int d = tid * VEC; d < H; d += kNormThreads * VEC) {
+    for (int d = tid * VEC; d < H; d += n_thr * VEC) {
 #pragma unroll
       for (int e = 0; e < VEC; ++e) row[d + e] = rd::Num<T>::to_f(src[d + e]) * embed_scale;
     }
   } else {
     const float* src = hist + (int64_t)t * H;
-    for (int d = tid * VEC; d < H; d += kNormThreads * VEC) {
+    for (int d = tid * VEC; d < H; d += n_thr * VEC) {
       float acc[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
@@ -68,7 +67,7 @@ __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
   __syncthreads();
   if (x_out != nullptr) {
     float* dst = x_out + (int64_t)t * H;
-    for (int d = tid * VEC; d < H; d += kNormThreads * VEC) {
+    for (int d = tid * VEC; d < H; d += n_thr * VEC) {
       if constexpr (VEC == 4)
         *reinterpret_cast<float4*>(dst + d) = *reinterpret_cast<const float4*>(row + d);
       else
@@ -78,7 +77,7 @@ __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
   // sums of squares: every group is cut into `parts` interleaved shares, one warp each
   const int warp = tid >> 5, lane = tid & 31;
   const int gsize = H / groups;
-  for (int u = warp; u < groups * parts; u += kNormWarps) {
+  for (int u = warp; u < groups * parts; u += (n_thr / 32)) {
     const float* g0 = row + (u / parts) * gsize;
     float ss = 0.f;
     for (int d = (u % parts) * 32 + lane; d < gsize; d += 32 * parts) ss = fmaf(g0[d], g0[d], ss);
@@ -87,7 +86,7 @@ __global__ void __launch_bounds__(kNormThreads) stream_norm_kernel(
   }
   __syncthreads();
   T* dst = y + (int64_t)t * H;
-  for (int d = tid * VEC; d < H; d += kNormThreads * VEC) {
+  for (int d = tid * VEC; d < H; d += n_thr * VEC) {
     T o[VEC];
     int g = -1;
     float rs = 0.f;
@@ -220,11 +219,16 @@ extern "C" int rd_stream_norm(int dtype, const void* table, const int64_t* ids, 
   RD_REQUIRE(weight && y && ((table && ids && !hist) || (!table && hist)), RD_ERR_ARG);
   RD_REQUIRE(m_max >= 1 && H >= 1 && groups >= 1 && H % groups == 0 && (table || n_hist >= 1), RD_ERR_SIZE);
   RD_REQUIRE(coeff || table || n_hist == 1, RD_ERR_ARG);
-  int parts = groups >= kNormWarps ? 1 : (kNormWarps + groups - 1) / groups;
-  const size_t smem = ((size_t)H + (size_t)groups * parts) * sizeof(float);
-  RD_REQUIRE(smem <= 200 * 1024, RD_ERR_SIZE);
   const uintptr_t bits = (uintptr_t)hist | (uintptr_t)x_out | (uintptr_t)y;
   const bool vec = H % 4 == 0 && bits % 16 == 0 && hist_stride % 4 == 0;
+  int threads = ((vec ? H / 4 : H) + 31) / 32 * 32;
+  // few tokens: the row's loads all in flight at once; many tokens: small blocks, several per SM
+  const int most = m_max <= 2 * 148 ? kNormMaxThreads : 256;
+  threads = threads > most ? most : threads;
+  const int warps = threads / 32;
+  const int parts = groups >= warps ? 1 : (warps + groups - 1) / groups;
+  const size_t smem = ((size_t)H + (size_t)groups * parts) * sizeof(float);
+  RD_REQUIRE(smem <= 200 * 1024, RD_ERR_SIZE);
   cudaError_t err = cudaSuccess;
   RD_DISPATCH_T(dtype, {
     auto kern = vec ? stream_norm_kernel<T, 4> : stream_norm_kernel<T, 1>;
@@ -232,7 +236,7 @@ extern "C" int rd_stream_norm(int dtype, const void* table, const int64_t* ids, 
       err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       RD_CHECK_CHAINED(err);
     }
-    err = rd::launch_chained(kern, dim3(m_max), dim3(kNormThreads), smem, (cudaStream_t)stream, 1, (const T*)table, ids,
+    err = rd::launch_chained(kern, dim3(m_max), dim3(threads), smem, (cudaStream_t)stream, 1, (const T*)table, ids,
                              embed_scale, hist, hist_stride, coeff, n_hist, x_out, (const T*)weight, (T*)y, m_max, m_dev, H,
                              groups, parts, eps);
   });

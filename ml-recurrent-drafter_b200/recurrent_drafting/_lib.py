@@ -42,6 +42,7 @@ SIGNATURES = {
     "rd_gemm_plan_destroy": (None, [_P]),
     "rd_gemm_bf16_tc": (_I, [_P, _I, _P, _L, _P, _P, _L, _P, _I, _P, _P]),
     "rd_gemm_bf16_tc_qkv_rope": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P]),
+    "rd_gemm_bf16_tc_qkvg_rope": (_I, [_P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P]),
     "rd_gemm_bf16_tc_res_norm": (_I, [_P, _P, _L, _P, _L, _P, _P, _P, _L, _P, _L, _P, _P]),
     "rd_gemm_bf16_tc_swiglu_normed": (_I, [_P, _P, _L, _P, _P, _L, _I, _I, _F, _P, _P]),
     "rd_gemm_bf16_tc_qkv_rope_normed": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _L, _I, _I, _F,
@@ -57,6 +58,7 @@ SIGNATURES = {
     "rd_attention_plan_create": (_P, [_P, _I, _P, _P, _I, _I, _I, _I, _I]),
     "rd_attention_plan_destroy": (None, [_P]),
     "rd_attention_tc": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P]),
+    "rd_attention_tc_window": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _P, _L, _P, _P]),
     "rd_attention_split_workspace_bytes": (_L, [_I, _I, _I]),
     "rd_attention_tc_split": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P, _L, _P, _P]),
     "rd_argmax_rows": (_I, [_P, _L, _I, _P, _I, _P, _P, _P]),
@@ -73,7 +75,7 @@ SIGNATURES = {
     "rd_rotary_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
     "rd_attention_window": (_I, [_I, _P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P]),
     "rd_mlstm_chunk_workspace_bytes": (_L, [_I, _I, _I, _I, _I]),
-    "rd_mlstm_chunk": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _L, _P]),
+    "rd_mlstm_chunk": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _L, _P]),
     "rd_mlstm_tree": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _L, _P]),
     "rd_mlstm_scan": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P]),
     "rd_cache_commit": (_I, [_I, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _P]),
@@ -137,7 +139,7 @@ def check(rc: int, what: str) -> None:
 # kernels enqueued per entry point where that is not one; `launches` counts the kernels this process has enqueued
 # through call() (a replayed CUDA graph adds the number of kernels captured in it, see count_replay)
 KERNELS_PER_CALL = {"rd_tree_pack": 2, "rd_gemm_bf16_tc_argmax": 2, "rd_attention_tc_split": 2, "rd_cache_unpack": 2,
-                    "rd_cache_unpack_static": 2, "rd_mlstm_chunk": 2, "rd_mlstm_tree": 2}
+                    "rd_cache_unpack_static": 2, "rd_mlstm_chunk": 3, "rd_mlstm_tree": 2}
 launches = 0
 
 

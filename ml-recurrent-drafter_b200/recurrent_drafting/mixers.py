@@ -2,6 +2,7 @@
 matrix-memory recurrence, the dense xIELU feed-forward.  A block owns its weights in the layouts the kernels consume
 and runs packed tokens (see StepContext); every constant is a parameter of the block."""
 import math
+import os
 from dataclasses import dataclass
 from typing import Callable, Dict, List, Optional, Tuple
 
@@ -63,21 +64,28 @@ class Scratch:
 
 
 class RotaryTables:
-    """cos/sin tables [n_pos, dims/2] in fp32, formed in fp64 on the host; one pair per (dims, base), grown on demand."""
+    """cos/sin tables in fp32, formed in fp64 on the host; one pair per (dims, base, head), grown on demand."""
 
     def __init__(self):
-        self._tables: Dict[Tuple[int, float], Tuple[torch.Tensor, torch.Tensor]] = {}
+        self._tables: Dict[Tuple[int, float, int], Tuple[torch.Tensor, torch.Tensor]] = {}
 
-    def get(self, dims: int, base: float, n_pos: int, device) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
-        if dims == 0:
+    def get(self, dims: int, base: float, n_pos: int, device, head: int = 0) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
+        """[n_pos, dims/2], one column per rotated pair; with head given [n_pos, head], one column per feature of the head
+        (cos 1, sin 0 past dims)."""
+        if dims == 0 and head == 0:
             return None, None
-        have = self._tables.get((dims, base))
+        key = (dims, base, head)
+        have = self._tables.get(key)
         if have is None or have[0].shape[0] < n_pos or have[0].device != torch.device(device):
             n = max(n_pos, 2048)
-            freq = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+            freq = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1))
             a = torch.arange(n, dtype=torch.float64)[:, None] * freq[None, :]
-            have = (a.cos().float().contiguous().to(device), a.sin().float().contiguous().to(device))
-            self._tables[(dims, base)] = have
+            cos, sin = a.cos(), a.sin()
+            if head:
+                rest = torch.zeros(n, head - dims, dtype=torch.float64)
+                cos, sin = torch.cat([cos, cos, rest + 1.0], dim=1), torch.cat([sin, sin, rest], dim=1)
+            have = (cos.float().contiguous().to(device), sin.float().contiguous().to(device))
+            self._tables[key] = have
         return have
 
 
@@ -94,6 +102,20 @@ class WindowAttention(nn.Module):
         self.w_in = weight(sum(self.sizes), width)
         self.w_out = weight(width, c.heads * c.vdim)
         self.lin: Optional[Tuple[Linear, Linear]] = None
+        self._plans: Dict[Tuple, int] = {}  # TMA descriptors of the tcgen05 attention, by the buffers they address
+
+    def drop_plans(self) -> None:
+        plans, self._plans = self._plans, {}
+        if plans:
+            lib = _lib.load()
+            for p in plans.values():
+                lib.rd_attention_plan_destroy(p)
+
+    def __del__(self):
+        try:
+            self.drop_plans()
+        except Exception:
+            pass
 
     def cache_spec(self) -> kv_cache.LayerSpec:
         return kv_cache.KeyValueSpec(self.cfg.kv_heads, self.cfg.dim, self.cfg.vdim)
@@ -121,6 +143,9 @@ class WindowAttention(nn.Module):
     def run(self, ctx: StepContext, state: kv_cache.LayerKeyValues, xn: torch.Tensor, residual: torch.Tensor, out: torch.Tensor) -> None:
         """out = residual + mixer(xn); residual and out are fp32 rows, xn the normed rows in the model's dtype."""
         c, ws, st = self.cfg, ctx.ws, _lib.stream()
+        if self._heads_of_128() and os.environ.get("RD_FUSED_ROPE", "1") != "0":
+            self._run_128(ctx, state, xn, residual, out)
+            return
         code = _lib.dtype_code(self.w_in.dtype)
         ld = row_stride(self.proj_width())
         proj = rows_of(ws["proj"], ld)
@@ -136,6 +161,46 @@ class WindowAttention(nn.Module):
                   _lib.ptr(mixed), _lib.ptr(ctx.row_start), _lib.ptr(ctx.kv_begin), _lib.ptr(ctx.base_len), ctx.batch, c.heads, c.kv_heads,
                   c.dim, c.vdim, max_len, ctx.max_new, ctx.mode, _lib.ptr(ctx.tok_pos), _lib.ptr(ctx.tree_mask), ctx.mask_words,
                   c.scale, c.window, c.keep_first, ctx.max_kv, st)
+        self.lin[1](mixed, out, _lib.EPI_RES, residual=residual, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
+
+    def _heads_of_128(self) -> bool:
+        c, w = self.cfg, self.w_in
+        return (w.dtype == torch.bfloat16 and c.dim == 128 and c.vdim == 128 and c.rot_dims % 16 == 0 and w.shape[1] >= 64
+                and w.shape[1] % 8 == 0)
+
+    def _run_128(self, ctx: StepContext, state: kv_cache.LayerKeyValues, xn, residual, out) -> None:
+        """Heads of 128 features in bf16: rotary embedding and cache append ride on the projection's epilogue, prompts and
+        draft trees take the tcgen05 attention."""
+        c, ws, st = self.cfg, ctx.ws, _lib.stream()
+        q = rows_of(ws["proj"], c.heads * 128)
+        ldg = row_stride(c.heads)
+        gate = rows_of(ws["head_gate"], ldg)
+        mixed = rows_of(ws["mixed"], c.heads * 128)
+        cos, sin = self.rotary.get(c.rot_dims, c.rot_base, ctx.n_pos, xn.device, head=128)
+        self.lin[0].qkvg_rope(xn, q, state.keys, state.values, gate, ctx.tok_row, ctx.tok_pos, ctx.tok_slot, cos, sin, c.heads, c.kv_heads,
+                              c.rot_dims, ctx.m_dev, ctx.m_max, ctx.status)
+        max_len = state.keys.shape[2]
+        few = (c.heads // c.kv_heads) * ctx.max_new <= 32  # the kernel that shares keys among a group's heads
+        tree = ctx.mode == _lib.ATTN_TREE
+        if few or c.scale <= 0 or (tree and (c.window < _lib.MAX_BEAM_LENGTH or ctx.mask_words > 16)):
+            _lib.call("rd_attention_window", _lib.BF16, _lib.ptr(q), c.heads * 128, _lib.ptr(state.keys), _lib.ptr(state.values), _lib.ptr(gate),
+                      ldg, _lib.ptr(mixed), _lib.ptr(ctx.row_start), _lib.ptr(ctx.kv_begin), _lib.ptr(ctx.base_len), ctx.batch, c.heads,
+                      c.kv_heads, 128, 128, max_len, ctx.max_new, ctx.mode, _lib.ptr(ctx.tok_pos), _lib.ptr(ctx.tree_mask),
+                      ctx.mask_words, c.scale, c.window, c.keep_first, ctx.max_kv, st)
+        else:
+            key = (q.data_ptr(), ctx.m_max, state.keys.data_ptr(), state.values.data_ptr(), ctx.batch, max_len)
+            plan = self._plans.get(key)
+            if plan is None:
+                plan = _lib.load().rd_attention_plan_create(_lib.ptr(q), ctx.m_max, _lib.ptr(state.keys), _lib.ptr(state.values), ctx.batch,
+                                                            c.heads, c.kv_heads, 128, max_len)
+                if not plan:
+                    raise _lib.RedrafterError("rd_attention_plan_create failed (TMA descriptor could not be encoded)")
+                if len(self._plans) >= 8:
+                    self.drop_plans()
+                self._plans[key] = plan
+            _lib.call("rd_attention_tc_window", plan, _lib.ptr(mixed), _lib.ptr(ctx.row_start), _lib.ptr(ctx.kv_begin), _lib.ptr(ctx.base_len),
+                      ctx.max_new, ctx.mode, _lib.ptr(ctx.tok_pos), _lib.ptr(ctx.tree_mask), ctx.mask_words, c.scale, c.window,
+                      c.keep_first, _lib.ptr(gate), ldg, _lib.ptr(ctx.status), st)
         self.lin[1](mixed, out, _lib.EPI_RES, residual=residual, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
 
     def commit_draft(self, state: kv_cache.LayerKeyValues, kv_begin, fp, n_accepted, seq_in_beam, beam_shape) -> None:
@@ -222,9 +287,10 @@ class MatrixMemory(nn.Module):
         self.lin[1](mixed, out, _lib.EPI_RES, residual=residual, m_dev=ctx.m_dev, m_max=ctx.m_max, status=ctx.status)
 
     def _chunked(self, ctx: StepContext) -> bool:
-        """Prompts of a bf16 model; a portion shorter than a quarter of a chunk is run token by token."""
+        """Prompts of a bf16 model; portions of a few tokens are run one after the other."""
         c = self.cfg
-        return self.w_in.dtype == torch.bfloat16 and ctx.max_new >= 16 and c.dim % 8 == 0 and c.dim <= 256 and c.vdim % 8 == 0
+        return (self.w_in.dtype == torch.bfloat16 and ctx.max_new >= 16 and c.dim % 8 == 0 and c.dim <= 256 and c.vdim % 8 == 0
+                and c.vdim <= 512)
 
     def _common(self, proj, gates, mixed, state, row_start, base_len):
         c = self.cfg
@@ -237,7 +303,7 @@ class MatrixMemory(nn.Module):
         need = _lib.load().rd_mlstm_chunk_workspace_bytes(ctx.m_max, ctx.batch, c.heads, c.dim, c.vdim)
         buf = self.scratch.get(need, proj.device)
         _lib.call("rd_mlstm_chunk", *self._common(proj, gates, mixed, state, ctx.row_start, ctx.base_len), ctx.batch, c.heads, c.dim,
-                  c.vdim, ctx.m_max, _lib.ptr(buf), buf.numel(), _lib.stream())
+                  c.vdim, ctx.m_max, ctx.max_new, _lib.ptr(buf), buf.numel(), _lib.stream())
 
     def _tree(self, ctx: StepContext, state, proj, gates, mixed) -> None:
         c = self.cfg

@@ -74,6 +74,18 @@ class Linear:
                   _lib.ptr(tok_row), _lib.ptr(tok_pos), _lib.ptr(tok_slot), _lib.ptr(cos), _lib.ptr(sin), cos.shape[0], nh, nkv,
                   hd, k_cache.shape[2], _lib.ptr(status), _lib.stream())
 
+    def qkvg_rope(self, a: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, gate_out: torch.Tensor,
+                  tok_row, tok_pos, tok_slot, cos: torch.Tensor, sin: torch.Tensor, nh: int, nkv: int, rot_dims: int, m_dev,
+                  m_max: int, status: Optional[torch.Tensor]) -> None:
+        """This weight as the packed q, k, v and head-gate projection of heads of 128 features, with rotary embedding on
+        rot_dims of them and the cache append in the epilogue (rd_gemm_bf16_tc_qkvg_rope); tensor-core path only."""
+        if not self._tc_ok(a, a.stride(0)):
+            raise _lib.RedrafterError("the fused QKV projection needs the tensor-core GEMM path (bf16, aligned operands)")
+        plan = self._plan(a, a.stride(0), m_max)
+        _lib.call("rd_gemm_bf16_tc_qkvg_rope", plan, _lib.ptr(m_dev), _lib.ptr(q_out), _lib.ptr(k_cache), _lib.ptr(v_cache),
+                  _lib.ptr(gate_out), gate_out.stride(0), _lib.ptr(tok_row), _lib.ptr(tok_pos), _lib.ptr(tok_slot), _lib.ptr(cos),
+                  _lib.ptr(sin), cos.shape[0], nh, nkv, 128, rot_dims, k_cache.shape[2], _lib.ptr(status), _lib.stream())
+
     def residual_with_norm(self, a: torch.Tensor, c: torch.Tensor, residual: torch.Tensor, gamma: torch.Tensor,
                            c2: torch.Tensor, ss: torch.Tensor, m_dev, m_max: int, status: Optional[torch.Tensor]) -> None:
         """c = a @ weight^T + residual, and the producer half of the RMS norm that follows: c2 = c * gamma and the

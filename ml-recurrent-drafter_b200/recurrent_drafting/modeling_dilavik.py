@@ -188,6 +188,8 @@ class DilavikForCausalLM(LMHead, nn.Module):
     def _drop_plans(self) -> None:
         if self._ready:
             for l in self.layers:
+                if isinstance(l.mixer, mixers.WindowAttention):
+                    l.mixer.drop_plans()
                 for lin in l.mixer.linears() + (l.mlp.linears() if l.mlp is not None else []):
                     lin.drop_plans()
             self._head.drop_plans()
@@ -208,6 +210,7 @@ class DilavikForCausalLM(LMHead, nn.Module):
             gates = max([2 * m.cfg.heads for m in mix if isinstance(m, mixers.MatrixMemory)] or [1])
             for name, width, t in (("x", H, torch.float32), ("mid", H, torch.float32), ("xn", H, dt), ("hidden", H, dt),
                                    ("proj", max(mixers.row_stride(m.proj_width()) for m in mix), dt), ("gates", gates, torch.float32),
+                                   ("head_gate", mixers.row_stride(max([m.cfg.heads for m in mix if isinstance(m, mixers.WindowAttention)] or [1])), dt),
                                    ("mixed", max(m.out_width() for m in mix), dt),
                                    ("act", mixers.row_stride(max([l.mlp.ff for l in self.layers if l.mlp is not None] or [1])), dt)):
                 full[name] = torch.empty(cap_m, width, dtype=t, device=dev)

@@ -298,7 +298,7 @@ class Memory:
         else:
             need = _lib.load().rd_mlstm_chunk_workspace_bytes(M, self.B, m["heads"], m["dim"], m["vdim"])
             ws = torch.empty(need, dtype=torch.uint8, device="cuda")
-            _lib.call("rd_mlstm_chunk", *common, M, ptr(ws), need, st)
+            _lib.call("rd_mlstm_chunk", *common, M, max(len(p[0]) for p in portions), ptr(ws), need, st)
         for r in range(self.B):
             if len(portions[r][0]):
                 self.state[r], want = self.plain(r, portions[r])
@@ -313,7 +313,7 @@ class Memory:
                     close(got, want, torch.float32, 2e-4)
 
 
-MEMORY_SIZES = [(2, 32, 64), (1, 256, 96), (3, 16, 40), (2, 64, 32), (1, 128, 200), (2, 72, 8)]
+MEMORY_SIZES = [(2, 32, 64), (1, 256, 96), (3, 16, 40), (2, 64, 32), (1, 128, 200), (2, 72, 8), (1, 200, 512)]
 
 
 @pytest.mark.parametrize("dt,kernel", [("fp32", "scan"), ("bf16", "scan"), ("bf16", "chunk")])
@@ -322,7 +322,7 @@ def test_matrix_memory_in_portions(dt, kernel, heads, d, dv):
     mix = db.mlstm(heads, d, dv, 5.0)["mixer"]
     mem = Memory(mix, 3, DTYPES[dt])
     seed = 0
-    for counts in ((70, 1, 64), (2, 0, 63), (1, 130, 2), (65, 3, 0)):
+    for counts in ((70, 1, 128), (2, 0, 127), (1, 260, 2), (65, 129, 0)):
         seed += 1
         mem.feed([mlstm_inputs(mix, n, mem.dtype, 100 * seed + r) for r, n in enumerate(counts)], kernel)
     # rows 0 and 2 are given back: their next tokens start from zero, row 1 goes on
@@ -350,7 +350,7 @@ def test_matrix_memory_with_gates_wide_open_and_shut(dt, kernel):
         mem.feed([mlstm_inputs(mix, n, mem.dtype, 31 * k + n, extreme=True) for n in (90, 64)], kernel)
 
 
-def test_many_rows_take_the_wide_slices():
+def test_matrix_memory_of_many_unequal_rows():
     mix = db.mlstm(8, 16, 64, 5.0)["mixer"]
     mem = Memory(mix, 20, torch.bfloat16)
     mem.feed([mlstm_inputs(mix, 20 + 5 * r, mem.dtype, r) for r in range(20)], "chunk")
