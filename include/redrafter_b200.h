@@ -461,7 +461,7 @@ RD_API int64_t rd_mlstm_chunk_workspace_bytes(int m_max, int B, int nh, int dim,
 RD_API int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
                    const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S, float* n,
                    float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim, int vdim, int m_max,
-                   int max_new, void* workspace, int64_t workspace_bytes, void* stream);
+                   int max_new, void* workspace, int64_t workspace_bytes, int32_t* status, void* stream);
 
 /* The same recurrence over packed draft trees: every new token continues its row's state along its own ancestors
  * (tree_mask, at most RD_MAX_BEAM_LENGTH of them, itself included); the state is left as it was.  workspace:

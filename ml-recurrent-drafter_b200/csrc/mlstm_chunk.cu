@@ -1,5 +1,6 @@
-// The matrix-memory recurrence of mlstm.cu for prompts: chunks of 128 tokens on the tensor cores (bf16 operands, fp32
-// accumulators).
+// The matrix-memory recurrence of mlstm.cu for prompts: chunks of 128 tokens on the tensor cores (tcgen05, bf16 operands,
+// fp32 accumulators in TMEM; operands staged by cp.async in the 128-byte swizzle).  Waits are bounded: on give-up a
+// kernel writes a code to *status, frees its TMEM and returns.
 //
 // Within a chunk, with F_t the running sum of the log forget gates and m_t the running maximum of the recurrence,
 //   m_t   = F_t + max(m_in, max_{j <= t} (i_j - F_j))
@@ -8,14 +9,15 @@
 //   S_out = e^(F_L + m_in - m_L) S_in + sum_j e^(F_L - F_j + i_j - m_L) k_j v_j^T      (n likewise with k alone)
 // so every exponent is <= 0, and the result is the token-by-token recurrence up to rounding.  Three kernels:
 //   gates    one CTA per (head, row): the scalars above for every token; only the chunks' maxima follow one another
-//   states   one CTA per 64 x 64 tile of S: walks the chunks, the tile in fp32 accumulators, and leaves S and n at the
-//            start of every chunk in the workspace
-//   outputs  one CTA per 64 tokens of a head: scores, both products, the head's RMS norm, the norm weight and the output
-//            gate, independent of all other chunks
+//   states   one CTA per 128 value columns x 128 dims of S: walks the chunks, the tile in TMEM (fp32), and leaves S and n
+//            at the start of every chunk in the workspace
+//   outputs  one CTA per chunk of a head: scores, both products (accumulated in TMEM), the head's RMS norm, the norm
+//            weight and the output gate, independent of all other chunks
 // The fp32 operands of the products - P, S and what enters the state, e^(...) v_j - are each split into two bf16 parts
 // (their rounding error is then about 2^-17).
 #include "mlstm_common.cuh"
 #include "mma_sync.cuh"
+#include "umma.cuh"
 
 namespace {
 
@@ -23,6 +25,11 @@ using namespace rd_mma;
 using namespace rd_mlstm;
 
 constexpr int L = 128;  // tokens per chunk
+
+// Bounded wait by whole warps; the answer is the same for all lanes.
+__device__ __forceinline__ bool wait_warp(uint64_t* bar, uint32_t parity) {
+  return __all_sync(0xffffffffu, rd_umma::mbar_wait(bar, parity));
+}
 constexpr int kThreads = 256;
 
 struct ChunkArgs {
@@ -42,6 +49,7 @@ struct ChunkArgs {
   const int32_t* row_start;
   const int32_t* base_len;
   int nh, dim, vdim, dpad, vpad, m_max;
+  int32_t* status;
   // workspace.  Per head and token [nh][m_max]:
   float* Fm;     // F_t - m_t
   float* iF;     // i_j - F_j
@@ -51,7 +59,7 @@ struct ChunkArgs {
   // per chunk slot and head; row b's chunk c has slot row_start[b] / L + b + c
   float* decay;  // e^(F_L + m_in - m_L)
   float* nc;     // [dpad] n at the chunk's start
-  __nv_bfloat16* Shi;  // [dpad][vpad] S at the chunk's start
+  __nv_bfloat16* Shi;  // [vpad][dpad] S^T at the chunk's start
   __nv_bfloat16* Slo;
 };
 
@@ -164,258 +172,288 @@ __global__ void __launch_bounds__(kThreads) mlstm_gates_kernel(const ChunkArgs a
 }
 
 // ------------------------------------------------------------------------------------------------ states
+// Rows of a [128 x 64] box are 128 bytes, 16-byte chunks permuted by the row: the tensor core's 128-byte swizzle.
+constexpr int kBox = 128 * 128;  // bytes
+
+template <int DN>
 struct StateSmem {
-  static constexpr int kTile = L * 64 * 2;  // [L tokens][64 features]
-  static constexpr int kBytes = 4 * kTile + 2 * kTile + (2 * L + 64) * 4;  // two stages of K and V, wV hi and lo, w, n
+  static constexpr int kK = (DN / 64) * kBox, kV = 2 * kBox;  // [128 tokens] x DN dims, x 128 value columns
+  static constexpr int kStage = kK + kV;
+  static constexpr int kMisc = (2 * L + DN + 8) * 4 + 64;
+  static constexpr int kBytes = 2 * kStage + 2 * kV + kMisc + 1024;  // two stages, w V hi and lo, alignment
 };
 
-// grid (dim tiles * value tiles, nh, B).  Warp: 16 dims x 32 value columns.
-__global__ void __launch_bounds__(kThreads, 2) mlstm_states_kernel(const ChunkArgs a) {
-  extern __shared__ __align__(128) uint8_t smem[];
+// grid (value tiles of 128 * dim tiles of DN, nh, B).  S^T tile [128 value columns = TMEM lanes][DN dims = TMEM columns].
+// Per chunk: the tile is read out, written to the workspace, scaled and put back, then (w V)^T K is added by tcgen05.mma
+// (both operands MN-major: value columns and dims contiguous, tokens along K).
+template <int DN>
+__global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkArgs a) {
+  using Y = StateSmem<DN>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int b = blockIdx.z, h = blockIdx.y;
-  const int v_tiles = a.vpad / 64;
-  const int d0 = (blockIdx.x / v_tiles) * 64, v0 = (blockIdx.x % v_tiles) * 64;
+  const int d_tiles = a.dpad / DN;
+  const int v0 = (blockIdx.x / d_tiles) * 128, d0 = (blockIdx.x % d_tiles) * DN;
   const int rs = a.row_start[b], n_tok = a.row_start[b + 1] - rs;
   if (n_tok <= 0) return;
   const int n_chunks = (n_tok + L - 1) / L;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int dm = (warp >> 1) * 16, vn = (warp & 1) * 32;
-  constexpr int T = StateSmem::kTile;
-  uint8_t* sHi = smem + 4 * T;
-  uint8_t* sLo = sHi + T;
-  float* s_w = reinterpret_cast<float*>(sLo + T);  // [2][L]
-  float* s_n = s_w + 2 * L;                         // [64]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  uint8_t* sHi = smem + 2 * Y::kStage;
+  uint8_t* sLo = sHi + Y::kV;
+  float* s_w = reinterpret_cast<float*>(sLo + Y::kV);  // [2][L]
+  float* s_n = s_w + 2 * L;                             // [DN]
+  uint64_t* bar = reinterpret_cast<uint64_t*>(s_n + DN);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 1);
+  if (tid == 0) {
+    rd_umma::mbar_init(bar, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 0) rd_umma::tmem_alloc(tmem_slot, DN);
   const bool fresh = a.base_len[b] == 0, owns_n = v0 == 0;
   const int64_t at = (int64_t)h * a.m_max + rs;
   float* S_g = a.S + ((int64_t)b * a.nh + h) * a.dim * a.vdim;
   float* n_g = a.n + ((int64_t)b * a.nh + h) * a.dim;
-
-  float acc[4][4];
-  auto each_state = [&](auto&& fn) {
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = d0 + dm + g + (e >> 1) * 8, v = v0 + vn + nt * 8 + t4 * 2 + (e & 1);
-        fn(acc[nt][e], d < a.dim && v < a.vdim, (int64_t)d * a.vdim + v);
-      }
-  };
-  each_state([&](float& s, bool in, int64_t off) { s = (in && !fresh) ? S_g[off] : 0.f; });
-  if (tid < 64) s_n[tid] = (d0 + tid < a.dim && !fresh) ? n_g[d0 + tid] : 0.f;
+  if (tid < DN) s_n[tid] = (d0 + tid < a.dim && !fresh) ? n_g[d0 + tid] : 0.f;
 
   auto load = [&](int c) {
-    uint8_t* sK = smem + (c & 1) * 2 * T;
-#pragma unroll
-    for (int i = 0; i < L * 8 / kThreads; ++i) {
-      const int idx = i * kThreads + tid, r = idx >> 3, ch = idx & 7;
-      const bool live = c * L + r < n_tok;
-      const bool in_k = live && d0 + ch * 8 < a.dim, in_v = live && v0 + ch * 8 < a.vdim;
-      const __nv_bfloat16* row = a.proj + (int64_t)(rs + (live ? c * L + r : 0)) * a.ld;
-      cp_async16(sK + swz<8>(r, ch), row + (a.nh + h) * a.dim + (in_k ? d0 + ch * 8 : 0), in_k);
-      cp_async16(sK + T + swz<8>(r, ch), row + 2 * a.nh * a.dim + h * a.vdim + (in_v ? v0 + ch * 8 : 0), in_v);
+    uint8_t* sK = smem + (c & 1) * Y::kStage;
+    uint8_t* sV = sK + Y::kK;
+    for (int i = tid; i < L * (DN / 8); i += kThreads) {
+      const int r = i / (DN / 8), ch = i % (DN / 8);
+      const bool in = c * L + r < n_tok && d0 + ch * 8 < a.dim;
+      cp_async16(sK + (ch >> 3) * kBox + swz<8>(r, ch & 7),
+                 a.proj + (int64_t)(rs + (in ? c * L + r : 0)) * a.ld + (a.nh + h) * a.dim + (in ? d0 + ch * 8 : 0), in);
+    }
+    for (int i = tid; i < L * 16; i += kThreads) {
+      const int r = i >> 4, ch = i & 15;
+      const bool in = c * L + r < n_tok && v0 + ch * 8 < a.vdim;
+      cp_async16(sV + (ch >> 3) * kBox + swz<8>(r, ch & 7),
+                 a.proj + (int64_t)(rs + (in ? c * L + r : 0)) * a.ld + 2 * a.nh * a.dim + h * a.vdim + (in ? v0 + ch * 8 : 0), in);
     }
     cp_async_commit();
-    if (tid < L) s_w[(c & 1) * L + tid] = c * L + tid < n_tok ? a.w[at + c * L + tid] : 0.f;
   };
   load(0);
+  auto w_of = [&](int c) { return (tid < L && c * L + tid < n_tok) ? a.w[at + c * L + tid] : 0.f; };
+  auto decay_of = [&](int c) { return a.decay[(int64_t)chunk_slot(rs, b, c) * a.nh + h]; };
+  if (tid < L) s_w[tid] = w_of(0);
+  float A = decay_of(0);
+  rd_umma::fence_before();
+  __syncthreads();
+  rd_umma::fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const int quarter = warp & 3, half = warp >> 2;
+  const int v = v0 + quarter * 32 + lane;  // this thread's value column
+  const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16) + half * (DN / 2);
+  bool ok = true;
+
   for (int c = 0; c < n_chunks; ++c) {
-    const int64_t slot = (int64_t)chunk_slot(rs, b, c) * a.nh + h;
-    const float A = a.decay[slot];
-    // the state at the chunk's start
-    {
-      uint32_t* hi = reinterpret_cast<uint32_t*>(a.Shi + slot * a.dpad * a.vpad);
-      uint32_t* lo = reinterpret_cast<uint32_t*>(a.Slo + slot * a.dpad * a.vpad);
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-        for (int hh = 0; hh < 2; ++hh) {
-          const int64_t off = ((int64_t)(d0 + dm + g + hh * 8) * a.vpad + v0 + vn + nt * 8 + t4 * 2) >> 1;
-          uint32_t x, y;
-          split2(acc[nt][hh * 2], acc[nt][hh * 2 + 1], x, y);
-          hi[off] = x;
-          lo[off] = y;
-        }
-    }
+    // the products of chunk c - 1 are in the tile, and its operands' shared memory is free
+    if (c > 0) ok = wait_warp(bar, (c - 1) & 1);
     cp_async_wait<0>();
-    __syncthreads();  // chunk c is here; everyone has left chunk c - 1
+    if (!__syncthreads_and(ok)) break;
+    rd_umma::fence_after();
+    const float w_next = c + 1 < n_chunks ? w_of(c + 1) : 0.f, A_next = c + 1 < n_chunks ? decay_of(c + 1) : 0.f;
     if (c + 1 < n_chunks) load(c + 1);
-    const uint8_t* sK = smem + (c & 1) * 2 * T;
-    const uint8_t* sV = sK + T;
+    const uint8_t* sK = smem + (c & 1) * Y::kStage;
+    const uint8_t* sV = sK + Y::kK;
     const float* w = s_w + (c & 1) * L;
+    const int64_t slot = (int64_t)chunk_slot(rs, b, c) * a.nh + h;
+    // w_j v_j as hi + lo, in the same swizzled boxes
 #pragma unroll 4
-    for (int i = 0; i < L * 32 / kThreads; ++i) {
-      const int idx = i * kThreads + tid, r = idx >> 5, cc = (idx & 31) * 2;
-      const int off = swz<8>(r, cc >> 3) + (cc & 7) * 2;
-      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sV + off));
-      split2(v.x * w[r], v.y * w[r], *reinterpret_cast<uint32_t*>(sHi + off), *reinterpret_cast<uint32_t*>(sLo + off));
+    for (int i = tid; i < L * 16; i += kThreads) {
+      const int r = i >> 4, ch = i & 15;
+      const int off = (ch >> 3) * kBox + swz<8>(r, ch & 7);
+      const float wr = w[r];
+      const uint4 u = *reinterpret_cast<const uint4*>(sV + off);
+      const __nv_bfloat162* x2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+      uint4 hi, lo;
+      uint32_t* hp = reinterpret_cast<uint32_t*>(&hi);
+      uint32_t* lp = reinterpret_cast<uint32_t*>(&lo);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(x2[e]);
+        split2(f.x * wr, f.y * wr, hp[e], lp[e]);
+      }
+      *reinterpret_cast<uint4*>(sHi + off) = hi;
+      *reinterpret_cast<uint4*>(sLo + off) = lo;
+    }
+    // the state at the chunk's start goes to the workspace; scaled, it becomes the accumulator of this chunk's products
+#pragma unroll
+    for (int q = 0; q < DN / 64; ++q) {
+      float s[32];
+      const int dq = d0 + half * (DN / 2) + q * 32;
+      if (c == 0) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) s[i] = (!fresh && v < a.vdim && dq + i < a.dim) ? S_g[(int64_t)(dq + i) * a.vdim + v] : 0.f;
+      } else {
+        rd_umma::tmem_ld32(t_row + q * 32, s);
+      }
+      const int64_t off = (slot * a.vpad + v) * a.dpad + dq;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        uint4 hi, lo;
+        split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
+        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
+        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
+        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
+        *reinterpret_cast<uint4*>(a.Shi + off + 8 * i) = hi;
+        *reinterpret_cast<uint4*>(a.Slo + off + 8 * i) = lo;
+      }
+#pragma unroll
+      for (int i = 0; i < 32; ++i) s[i] *= A;
+      rd_umma::tmem_st32(t_row + q * 32, s);
+    }
+    rd_umma::fence_async_proxy();
+    rd_umma::fence_before();
+    __syncthreads();
+    if (tid == 0) {
+      rd_umma::fence_after();
+      const uint32_t idesc = rd_umma::idesc_f16(DN, true, true);
+#pragma unroll
+      for (int k = 0; k < L / 16; ++k) {
+        const uint64_t dk = rd_umma::desc_mn_major(rd_umma::smem_u32(sK + k * 2048), kBox);
+        rd_umma::mma_ss(tmem, rd_umma::desc_mn_major(rd_umma::smem_u32(sHi + k * 2048), kBox), dk, idesc, 1);
+        rd_umma::mma_ss(tmem, rd_umma::desc_mn_major(rd_umma::smem_u32(sLo + k * 2048), kBox), dk, idesc, 1);
+      }
+      rd_umma::commit(bar);
     }
     if (owns_n) {
-      // four threads per dim, 32 tokens each
-      const int d = tid >> 2, part = tid & 3;
+      // n of this tile's dims: kThreads / DN threads per dim
+      constexpr int PER = kThreads / DN;
+      const int d = tid / PER, part = tid % PER;
       float sum = 0.f;
 #pragma unroll 8
-      for (int j = part; j < L; j += 4)
-        sum = fmaf(w[j], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sK + swz<8>(j, d >> 3) + (d & 7) * 2)), sum);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      for (int j = part; j < L; j += PER)
+        sum = fmaf(w[j], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sK + (d >> 6) * kBox + swz<8>(j, (d & 63) >> 3) + (d & 7) * 2)), sum);
+#pragma unroll
+      for (int o = 1; o < PER; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       if (part == 0) {
         a.nc[slot * a.dpad + d0 + d] = s_n[d];
         s_n[d] = fmaf(A, s_n[d], sum);  // this thread's alone
       }
     }
-    __syncthreads();
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[nt][e] *= A;
-#pragma unroll
-    for (int kj = 0; kj < L / 16; ++kj) {
-      uint32_t af[4];
-      ldmatrix_x4_trans(af[0], af[1], af[2], af[3],
-                        smem_addr(sK + swz<8>(kj * 16 + ((lane >> 4) << 3) + (lane & 7), (dm >> 3) + ((lane >> 3) & 1))));
-#pragma unroll
-      for (int nt = 0; nt < 4; nt += 2) {
-        const int off = swz<8>(kj * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), (vn >> 3) + nt + (lane >> 4));
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_addr(sHi + off));
-        mma_bf16(acc[nt], af, b0, b1);
-        mma_bf16(acc[nt + 1], af, b2, b3);
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_addr(sLo + off));
-        mma_bf16(acc[nt], af, b0, b1);
-        mma_bf16(acc[nt + 1], af, b2, b3);
-      }
-    }
+    if (tid < L) s_w[((c + 1) & 1) * L + tid] = w_next;
+    A = A_next;
   }
-  each_state([&](float& s, bool in, int64_t off) {
-    if (in) S_g[off] = s;
-  });
-  if (owns_n && (tid & 3) == 0 && d0 + (tid >> 2) < a.dim) n_g[d0 + (tid >> 2)] = s_n[tid >> 2];
+  cp_async_wait<0>();
+  if (ok) ok = wait_warp(bar, (n_chunks - 1) & 1);
+  ok = __syncthreads_and(ok);
+  if (ok) {
+    rd_umma::fence_after();
+#pragma unroll
+    for (int q = 0; q < DN / 64; ++q) {
+      float s[32];
+      const int dq = d0 + half * (DN / 2) + q * 32;
+      rd_umma::tmem_ld32(t_row + q * 32, s);
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (v < a.vdim && dq + i < a.dim) S_g[(int64_t)(dq + i) * a.vdim + v] = s[i];
+    }
+    constexpr int PER = kThreads / DN;
+    if (owns_n && tid % PER == 0 && d0 + tid / PER < a.dim) n_g[d0 + tid / PER] = s_n[tid / PER];
+  } else if (tid == 0 && a.status) {
+    atomicExch(a.status, 31);
+  }
+  rd_umma::fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    rd_umma::fence_after();
+    rd_umma::tmem_dealloc(tmem, DN);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ outputs
-constexpr int BT = 64;  // query tokens per CTA
-constexpr int BK = 32;  // dims or tokens per streamed block
+constexpr int kOutStages = 4;
+constexpr int kItem = kBox;  // bytes of one streamed operand tile: [128 value columns x 64 dims] or [64 tokens x 128 value columns]
 
-template <int DP, int WN>
+template <int DP>
 struct OutSmem {
-  static constexpr int kCols = WN * 64;
-  static constexpr int kQ = BT * DP * 2, kK = L * DP * 2, kP = BT * L * 2;
-  static constexpr int kBlock = BK * kCols * 2;    // one streamed block of one operand
-  static constexpr int kStage = 2 * kBlock;        // hi and lo
-  static constexpr int kRing = 2 * kStage > kK ? 2 * kStage : kK;  // K is dead once the scores are formed
-  static constexpr int kMisc = (5 * BT + L + DP + 2 * BT + WN * BT) * 4;
-  static constexpr int kBytes = kQ + 2 * kP + kRing + kMisc;
+  static constexpr int kQ = (DP / 64) * kBox;
+  static constexpr int kRing = kOutStages * kItem > kQ ? kOutStages * kItem : kQ;  // K first, then the ring
+  static constexpr int kP = 2 * kBox;
+  static constexpr int kMisc = (5 * L + DP + 4 * L) * 4 + 128;
+  static constexpr int kBytes = kQ + kRing + 2 * kP + kMisc + 1024;
 };
 
-// grid (64-token tiles, nh, B).  WN warps along the value columns (64 each), 8 / WN along the tokens.
-template <int DP, int WN>
+// grid (chunks, nh, B).  O [128 tokens = TMEM lanes][value columns = TMEM columns]:
+//   scores Q K^T (in O's columns, before O exists) -> P hi / lo in shared memory -> O = Q S (hi, lo) -> O *= e_t ->
+//   O += P V (hi, lo) -> / denominator, RMS, norm weight, output gate.
+template <int DP>
 __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkArgs a) {
-  using Y = OutSmem<DP, WN>;
-  constexpr int WM = 8 / WN < 4 ? 8 / WN : 4;  // warps along the tokens
-  constexpr int MT = 4 / WM;                   // 16-token tiles per warp
-  constexpr int CQ = DP / 8, CP = L / 8, CB = Y::kCols / 8;
-  extern __shared__ __align__(128) uint8_t smem[];
+  using Y = OutSmem<DP>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   rd::pdl_launch_dependents();
   rd::pdl_wait();
-  const int b = blockIdx.z, h = blockIdx.y;
+  const int b = blockIdx.z, h = blockIdx.y, c = blockIdx.x;
   const int rs = a.row_start[b], n_tok = a.row_start[b + 1] - rs;
-  const int t0 = blockIdx.x * BT;  // first token of the tile within the row
+  const int t0 = c * L;
   if (t0 >= n_tok) return;
-  const int c = t0 / L, j0 = c * L, n_keys = t0 - j0 + BT;  // keys j0 .. j0 + n_keys - 1 (64 or 128)
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int64_t slot = (int64_t)chunk_slot(rs, b, c) * a.nh + h, at = (int64_t)h * a.m_max + rs;
   uint8_t* sQ = smem;
-  uint8_t* sPh = sQ + Y::kQ;
+  uint8_t* ring = sQ + Y::kQ;
+  uint8_t* sPh = ring + Y::kRing;
   uint8_t* sPl = sPh + Y::kP;
-  uint8_t* ring = sPl + Y::kP;
-  uint8_t* sK = ring;
-  float* s_Fm = reinterpret_cast<float*>(ring + Y::kRing);
-  float* s_e = s_Fm + BT;
-  float* s_floor = s_e + BT;
-  float* s_nq = s_floor + BT;
-  float* s_inv = s_nq + BT;
-  float* s_iF = s_inv + BT;   // [L]
-  float* s_n = s_iF + L;      // [DP]
-  float* s_rs = s_n + DP;     // [2][BT]
-  float* s_ss = s_rs + 2 * BT;  // [WN][BT]
+  float* s_Fm = reinterpret_cast<float*>(sPl + Y::kP);
+  float* s_iF = s_Fm + L;
+  float* s_e = s_iF + L;
+  float* s_floor = s_e + L;
+  float* s_nq = s_floor + L;
+  float* s_n = s_nq + L;       // [DP]
+  float* s_rs = s_n + DP;      // [2][L]
+  float* s_ss = s_rs + 2 * L;  // [2][L]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 2 * L);  // [kOutStages] an item's products are done; [+1] the scores
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + kOutStages + 1);
+  const uint32_t n_cols = a.vpad <= 128 ? 128 : (a.vpad <= 256 ? 256 : 512);
+  if (tid == 0) {
+    for (int i = 0; i <= kOutStages; ++i) rd_umma::mbar_init(&bars[i], 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 0) rd_umma::tmem_alloc(tmem_slot, n_cols);
   const float qs = rsqrtf((float)a.dim);
 
-  for (int idx = tid; idx < BT * CQ; idx += kThreads) {
-    const int r = idx / CQ, ch = idx % CQ;
+  for (int i = tid; i < L * (DP / 8); i += kThreads) {
+    const int r = i / (DP / 8), ch = i % (DP / 8);
     const bool in = t0 + r < n_tok && ch * 8 < a.dim;
-    cp_async16(sQ + swz<CQ>(r, ch), a.proj + (int64_t)(rs + (in ? t0 + r : 0)) * a.ld + h * a.dim + (in ? ch * 8 : 0), in);
-  }
-  for (int idx = tid; idx < n_keys * CQ; idx += kThreads) {
-    const int r = idx / CQ, ch = idx % CQ;
-    const bool in = j0 + r < n_tok && ch * 8 < a.dim;
-    cp_async16(sK + swz<CQ>(r, ch), a.proj + (int64_t)(rs + (in ? j0 + r : 0)) * a.ld + (a.nh + h) * a.dim + (in ? ch * 8 : 0), in);
+    const __nv_bfloat16* src = a.proj + (int64_t)(rs + (in ? t0 + r : 0)) * a.ld + h * a.dim + (in ? ch * 8 : 0);
+    const int off = (ch >> 3) * kBox + swz<8>(r, ch & 7);
+    cp_async16(sQ + off, src, in);
+    cp_async16(ring + off, src + a.nh * a.dim, in);
   }
   cp_async_commit();
-  if (tid < BT) {
+  if (tid < L) {
     const bool in = t0 + tid < n_tok;
     s_Fm[tid] = in ? a.Fm[at + t0 + tid] : 0.f;
+    s_iF[tid] = in ? a.iF[at + t0 + tid] : -INFINITY;
     s_e[tid] = in ? a.e[at + t0 + tid] : 0.f;
     s_floor[tid] = in ? a.floor[at + t0 + tid] : 1.f;
   }
-  if (tid < L) s_iF[tid] = (tid < n_keys && j0 + tid < n_tok) ? a.iF[at + j0 + tid] : -INFINITY;
   for (int d = tid; d < DP; d += kThreads) s_n[d] = d < a.dpad ? a.nc[slot * a.dpad + d] : 0.f;
   cp_async_wait<0>();
+  rd_umma::fence_async_proxy();
+  rd_umma::fence_before();
   __syncthreads();
-
-  // ---- P = (Q K^T) o weights: warp -> 16 tokens x half of the keys
-  {
-    const int tw = (warp & 3) * 16, half = n_keys / 2, jw = (warp >> 2) * half;
-    const bool first_half = n_keys == BT;  // the chunk's first 64 tokens: keys and queries coincide
-    float s[8][4];
+  rd_umma::fence_after();
+  const uint32_t tmem = *tmem_slot;
+  if (tid == 0) {
+    const uint32_t idesc = rd_umma::idesc_f16(128, false, false);
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
-    const int n_nt = half / 8;  // 4 or 8
-    const int q_off = first_half ? 0 : BT;
-    if (jw <= tw + 15 + q_off) {
-#pragma unroll 2
-      for (int kd = 0; kd < DP / 16; ++kd) {
-        uint32_t af[4];
-        ldmatrix_x4(af[0], af[1], af[2], af[3], smem_addr(sQ + swz<CQ>(tw + (lane & 15), kd * 2 + (lane >> 4))));
-#pragma unroll
-        for (int nb = 0; nb < 8; nb += 2) {
-          if (nb < n_nt) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4(b0, b1, b2, b3, smem_addr(sK + swz<CQ>(jw + nb * 8 + ((lane >> 4) << 3) + (lane & 7), kd * 2 + ((lane >> 3) & 1))));
-            mma_bf16(s[nb], af, b0, b1);
-            mma_bf16(s[nb + 1], af, b2, b3);
-          }
-        }
-      }
+    for (int k = 0; k < DP / 16; ++k) {
+      const int off = (k >> 2) * kBox + (k & 3) * 32;
+      rd_umma::mma_ss(tmem, rd_umma::desc_k_major(rd_umma::smem_u32(sQ + off)), rd_umma::desc_k_major(rd_umma::smem_u32(ring + off)), idesc, k != 0);
     }
-#pragma unroll
-    for (int hh = 0; hh < 2; ++hh) {
-      const int t = tw + g + hh * 8, tk = t + q_off;  // tk: the query's place among the keys
-      const float Fm = s_Fm[t];
-      float sum = 0.f;
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
-        if (nt < n_nt) {
-          const int j = jw + nt * 8 + t4 * 2;
-          const float p0 = j <= tk ? s[nt][hh * 2] * qs * expf(Fm + s_iF[j]) : 0.f;
-          const float p1 = j + 1 <= tk ? s[nt][hh * 2 + 1] * qs * expf(Fm + s_iF[j + 1]) : 0.f;
-          sum += p0 + p1;
-          const int off = swz<CP>(t, j >> 3) + (j & 7) * 2;
-          split2(p0, p1, *reinterpret_cast<uint32_t*>(sPh + off), *reinterpret_cast<uint32_t*>(sPl + off));
-        }
-      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-      if (t4 == 0) s_rs[(warp >> 2) * BT + t] = sum;
-    }
+    rd_umma::commit(&bars[kOutStages]);
   }
-  // ---- n_in . q_t: four threads per token
+  // n_in . q_t meanwhile: two threads per token
   {
-    const int t = tid >> 2, part = tid & 3;
+    const int t = tid >> 1, part = tid & 1;
     float acc = 0.f;
 #pragma unroll 2
-    for (int ch = part; ch < CQ; ch += 4) {
-      const uint4 u = *reinterpret_cast<const uint4*>(sQ + swz<CQ>(t, ch));
+    for (int ch = part; ch < DP / 8; ch += 2) {
+      const uint4 u = *reinterpret_cast<const uint4*>(sQ + (ch >> 3) * kBox + swz<8>(t, ch & 7));
       const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(&u);
       const float4 n0 = *reinterpret_cast<const float4*>(s_n + ch * 8), n1 = *reinterpret_cast<const float4*>(s_n + ch * 8 + 4);
       const float2 f0 = __bfloat1622float2(q2[0]), f1 = __bfloat1622float2(q2[1]);
@@ -424,210 +462,220 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
       acc = fmaf(f2.x, n1.x, fmaf(f2.y, n1.y, fmaf(f3.x, n1.z, fmaf(f3.y, n1.w, acc))));
     }
     acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-    acc += __shfl_xor_sync(0xffffffffu, acc, 2);
     if (part == 0) s_nq[t] = acc;
   }
-  __syncthreads();  // P is complete, K is dead
-  if (tid < BT) {
-    const float den = s_rs[tid] + s_rs[BT + tid] + s_e[tid] * s_nq[tid];
-    s_inv[tid] = 1.0f / (fmaxf(fabsf(den), s_floor[tid]) + kDenEps);
+  const int quarter = warp & 3, half = warp >> 2;
+  const int t = quarter * 32 + lane;  // this thread's token of the chunk
+  const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16);
+  bool ok = wait_warp(&bars[kOutStages], 0);
+  rd_umma::fence_after();
+  // P of this thread's token and half of the keys
+  if (ok) {
+    const float Fm = s_Fm[t];
+    float sum = 0.f;
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      float s[32];
+      const int j0 = half * 64 + q * 32;
+      rd_umma::tmem_ld32(t_row + j0, s);
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        s[i] = j0 + i <= t ? s[i] * qs * __expf(Fm + s_iF[j0 + i]) : 0.f;
+        sum += s[i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        uint4 hi, lo;
+        split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
+        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
+        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
+        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
+        const int off = half * kBox + swz<8>(t, q * 4 + i);
+        *reinterpret_cast<uint4*>(sPh + off) = hi;
+        *reinterpret_cast<uint4*>(sPl + off) = lo;
+      }
+    }
+    s_rs[half * L + t] = sum;
   }
+  rd_umma::fence_before();
+  ok = __syncthreads_and(ok);  // P is complete, K is dead, the scores have been read
 
-  // ---- O = e_t Q S + P V, the second operands streamed in blocks of 32 rows
-  const int n_dim = (a.dpad < DP ? a.dpad : DP) / BK, n_blocks = n_dim + n_keys / BK;
-  auto load = [&](int blk) {
-    if (blk < n_blocks) {
-      uint8_t* dst = ring + (blk & 1) * Y::kStage;
-      if (blk < n_dim) {
-        const __nv_bfloat16* hi = a.Shi + (slot * a.dpad + blk * BK) * a.vpad;
-        const __nv_bfloat16* lo = a.Slo + (slot * a.dpad + blk * BK) * a.vpad;
+  // ---- the streamed second operands: S tiles (dim block, value tile, hi / lo), then V tiles (64 tokens, value tile)
+  const int v_tiles = a.vpad / 128, d_blocks = a.dpad / 64;
+  const int n_state = d_blocks * v_tiles * 2, n_items = n_state + ((t0 + 64 < n_tok) ? 2 : 1) * v_tiles;
+  auto load = [&](int i) {
+    if (i < n_items) {
+      uint8_t* dst = ring + (i % kOutStages) * kItem;
+      if (i < n_state) {
+        const int lo = i & 1, vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
+        const __nv_bfloat16* src = (lo ? a.Slo : a.Shi) + (slot * a.vpad + vt * 128) * a.dpad + db * 64;
 #pragma unroll
-        for (int i = 0; i < BK * CB / kThreads; ++i) {
-          const int idx = i * kThreads + tid, r = idx / CB, ch = idx % CB;
-          const bool in = ch * 8 < a.vpad;
-          const int64_t off = (int64_t)r * a.vpad + (in ? ch * 8 : 0);
-          cp_async16(dst + swz<CB>(r, ch), hi + off, in);
-          cp_async16(dst + Y::kBlock + swz<CB>(r, ch), lo + off, in);
+        for (int u = 0; u < 4; ++u) {
+          const int idx = u * kThreads + tid, r = idx >> 3, ch = idx & 7;
+          cp_async16(dst + swz<8>(r, ch), src + (int64_t)r * a.dpad + ch * 8, true);
         }
       } else {
-        const int jb = j0 + (blk - n_dim) * BK;
+        const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
 #pragma unroll
-        for (int i = 0; i < BK * CB / kThreads; ++i) {
-          const int idx = i * kThreads + tid, r = idx / CB, ch = idx % CB;
-          const bool in = jb + r < n_tok && ch * 8 < a.vdim;
-          cp_async16(dst + swz<CB>(r, ch),
-                     a.proj + (int64_t)(rs + (in ? jb + r : 0)) * a.ld + 2 * a.nh * a.dim + h * a.vdim + (in ? ch * 8 : 0), in);
+        for (int u = 0; u < 4; ++u) {
+          const int idx = u * kThreads + tid, r = idx >> 4, ch = idx & 15;
+          const int tok = t0 + jb * 64 + r, v = vt * 128 + ch * 8;
+          const bool in = tok < n_tok && v < a.vdim;
+          cp_async16(dst + (ch >> 3) * (kItem / 2) + swz<8>(r, ch & 7),
+                     a.proj + (int64_t)(rs + (in ? tok : 0)) * a.ld + 2 * a.nh * a.dim + h * a.vdim + (in ? v : 0), in);
         }
       }
     }
-    cp_async_commit();
+    cp_async_commit();  // one group per item, empty or not
   };
-  const int wn = warp % WN, wm = warp / WN;
-  const bool works = wm < WM;  // WN == 1 would leave warps idle; WN >= 2 uses all eight
-  float o[MT][8][4];
+  if (ok) {
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+    for (int i = 0; i < kOutStages - 1; ++i) load(i);
+  }
+  for (int i = 0; i < n_items; ++i) {  // left by all threads together, see the barrier below
+    if (i == n_state && ok) {
+      // the state's part is complete: scale it by the tokens' e_t before the scores' part is added
+      ok = wait_warp(&bars[(i - 1) % kOutStages], ((i - 1) / kOutStages) & 1);
+      rd_umma::fence_after();
+      const float e = s_e[t];
+      if (ok) {
+        for (int q = half * (v_tiles * 2); q < (half + 1) * (v_tiles * 2); ++q) {
+          float o[32];
+          rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) o[m][nt][0] = o[m][nt][1] = o[m][nt][2] = o[m][nt][3] = 0.f;
-  load(0);
-  for (int blk = 0; blk < n_blocks; ++blk) {
-    cp_async_wait<0>();
-    __syncthreads();  // block blk is here; everyone has left block blk - 1
-    load(blk + 1);
-    if (!works) continue;
-    const uint8_t* sB = ring + (blk & 1) * Y::kStage;
-    if (blk == n_dim) {
-      // the state's part is complete: scale it before the scores' part is added
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const float e0 = s_e[(wm * MT + m) * 16 + g], e1 = s_e[(wm * MT + m) * 16 + g + 8];
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt) {
-          o[m][nt][0] *= e0;
-          o[m][nt][1] *= e0;
-          o[m][nt][2] *= e1;
-          o[m][nt][3] *= e1;
+          for (int k = 0; k < 32; ++k) o[k] *= e;
+          rd_umma::tmem_st32(t_row + q * 32, o);
         }
       }
+      rd_umma::fence_before();
     }
-    const bool state = blk < n_dim;
+    cp_async_wait<kOutStages - 2>();  // item i is here
+    rd_umma::fence_async_proxy();
+    if (!__syncthreads_and(ok)) {
+      ok = false;
+      break;
+    }
+    const uint8_t* sB = ring + (i % kOutStages) * kItem;
+    if (tid == 0) {
+      rd_umma::fence_after();
+      if (i < n_state) {
+        const int lo = i & 1, vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
+        const uint32_t idesc = rd_umma::idesc_f16(128, false, false);
 #pragma unroll
-    for (int k16 = 0; k16 < BK / 16; ++k16) {
-      const int row = k16 * 16 + (((lane >> 3) & 1) << 3) + (lane & 7);
-      if (state) {
-        uint32_t af[MT][4];
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-          ldmatrix_x4(af[m][0], af[m][1], af[m][2], af[m][3],
-                      smem_addr(sQ + swz<CQ>((wm * MT + m) * 16 + (lane & 15), blk * (BK / 8) + k16 * 2 + (lane >> 4))));
-#pragma unroll
-        for (int nt = 0; nt < 8; nt += 2) {
-          const int off = swz<CB>(row, wn * 8 + nt + (lane >> 4));
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(b0, b1, b2, b3, smem_addr(sB + off));
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            mma_bf16(o[m][nt], af[m], b0, b1);
-            mma_bf16(o[m][nt + 1], af[m], b2, b3);
-          }
-          ldmatrix_x4_trans(b0, b1, b2, b3, smem_addr(sB + Y::kBlock + off));
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            mma_bf16(o[m][nt], af[m], b0, b1);
-            mma_bf16(o[m][nt + 1], af[m], b2, b3);
-          }
-        }
+        for (int k = 0; k < 4; ++k)
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sQ + db * kBox + k * 32)),
+                          rd_umma::desc_k_major(rd_umma::smem_u32(sB + k * 32)), idesc, (db | lo | k) != 0);
       } else {
+        const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
+        const uint32_t idesc = rd_umma::idesc_f16(128, false, true);
 #pragma unroll
-        for (int part = 0; part < 2; ++part) {
-          const uint8_t* sP = part ? sPl : sPh;
-          uint32_t af[MT][4];
-#pragma unroll
-          for (int m = 0; m < MT; ++m)
-            ldmatrix_x4(af[m][0], af[m][1], af[m][2], af[m][3],
-                        smem_addr(sP + swz<CP>((wm * MT + m) * 16 + (lane & 15), (blk - n_dim) * (BK / 8) + k16 * 2 + (lane >> 4))));
-#pragma unroll
-          for (int nt = 0; nt < 8; nt += 2) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_addr(sB + swz<CB>(row, wn * 8 + nt + (lane >> 4))));
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-              mma_bf16(o[m][nt], af[m], b0, b1);
-              mma_bf16(o[m][nt + 1], af[m], b2, b3);
-            }
-          }
+        for (int k = 0; k < 4; ++k) {
+          const uint64_t dv = rd_umma::desc_mn_major(rd_umma::smem_u32(sB + k * 2048), kItem / 2);
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPh + jb * kBox + k * 32)), dv, idesc, 1);
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPl + jb * kBox + k * 32)), dv, idesc, 1);
         }
       }
+      rd_umma::commit(&bars[i % kOutStages]);
     }
+    // the stage of item i - 1 takes item i + kOutStages - 1 once that item's products are done
+    if (ok && i > 0 && i + kOutStages - 1 < n_items) ok = wait_warp(&bars[(i - 1) % kOutStages], ((i - 1) / kOutStages) & 1);
+    load(ok ? i + kOutStages - 1 : n_items);
   }
   cp_async_wait<0>();
-
-  // ---- o / denominator, RMS over the head, norm weight, output gate
-  if (works) {
+  if (ok) ok = wait_warp(&bars[(n_items - 1) % kOutStages], ((n_items - 1) / kOutStages) & 1);
+  ok = __syncthreads_and(ok);
+  if (ok) {
+    rd_umma::fence_after();
+    const float den = s_rs[t] + s_rs[L + t] + s_e[t] * s_nq[t];
+    const float inv = 1.0f / (fmaxf(fabsf(den), s_floor[t]) + kDenEps);
+    const int q_lo = half * (v_tiles * 2), q_hi = q_lo + v_tiles * 2;  // this thread's 32-column blocks
+    float ss = 0.f;
+    for (int q = q_lo; q < q_hi; ++q) {
+      float o[32];
+      rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+      for (int k = 0; k < 32; ++k) ss = fmaf(o[k] * inv, o[k] * inv, ss);
+    }
+    s_ss[half * L + t] = ss;
+    __syncthreads();
+    const float r = inv / sqrtf((s_ss[t] + s_ss[L + t]) / (float)a.vdim + a.eps);
+    const int64_t tok = rs + t0 + t;
+    const bool live = t0 + t < n_tok;
+    const __nv_bfloat16* gp = a.proj + (live ? tok : (int64_t)rs) * a.ld + 2 * a.nh * a.dim + (a.nh + h) * a.vdim;
+    const __nv_bfloat16* wp = a.norm_w + (int64_t)h * a.vdim;
+    __nv_bfloat16* dst = a.out + (tok * a.nh + h) * a.vdim;
+    for (int q = q_lo; q < q_hi; ++q) {
+      float o[32];
+      rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const int t = (wm * MT + m) * 16 + g + hh * 8;
-        const float inv = s_inv[t];
-        float ss = 0.f;
+      for (int i = 0; i < 4; ++i) {
+        const int v = q * 32 + i * 8;
+        if (live && v < a.vdim) {
+          const uint4 gu = *reinterpret_cast<const uint4*>(gp + v), wu = *reinterpret_cast<const uint4*>(wp + v);
+          const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu);
+          const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&wu);
+          uint4 pk;
+          uint32_t* pp = reinterpret_cast<uint32_t*>(&pk);
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) {
-          o[m][nt][hh * 2] *= inv;
-          o[m][nt][hh * 2 + 1] *= inv;
-          ss = fmaf(o[m][nt][hh * 2], o[m][nt][hh * 2], ss);
-          ss = fmaf(o[m][nt][hh * 2 + 1], o[m][nt][hh * 2 + 1], ss);
-        }
-        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
-        ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-        if (t4 == 0) s_ss[wn * BT + t] = ss;
-      }
-  }
-  __syncthreads();
-  if (!works) return;
-  const __nv_bfloat16* w_h = a.norm_w + (int64_t)h * a.vdim;
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int hh = 0; hh < 2; ++hh) {
-      const int t = (wm * MT + m) * 16 + g + hh * 8;
-      if (t0 + t >= n_tok) continue;
-      float ss = 0.f;
-#pragma unroll
-      for (int k = 0; k < WN; ++k) ss += s_ss[k * BT + t];
-      const float r = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
-      const int64_t tok = rs + t0 + t;
-      const __nv_bfloat16* gp = a.proj + tok * a.ld + 2 * a.nh * a.dim + (a.nh + h) * a.vdim;
-      __nv_bfloat16* dst = a.out + (tok * a.nh + h) * a.vdim;
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const int v = wn * 64 + nt * 8 + t4 * 2;
-        if (v < a.vdim) {
-          const float2 gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + v));
-          const float2 ww = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w_h + v));
-          *reinterpret_cast<uint32_t*>(dst + v) = pack_bf16(o[m][nt][hh * 2] * r * ww.x / (1.f + __expf(-gg.x)),
-                                                            o[m][nt][hh * 2 + 1] * r * ww.y / (1.f + __expf(-gg.y)));
+          for (int e = 0; e < 4; ++e) {
+            const float2 gg = __bfloat1622float2(g2[e]), ww = __bfloat1622float2(w2[e]);
+            pp[e] = pack_bf16(__fdividef(o[8 * i + 2 * e] * r * ww.x, 1.f + __expf(-gg.x)),
+                              __fdividef(o[8 * i + 2 * e + 1] * r * ww.y, 1.f + __expf(-gg.y)));
+          }
+          *reinterpret_cast<uint4*>(dst + v) = pk;
         }
       }
     }
+  } else if (tid == 0 && a.status) {
+    atomicExch(a.status, 32);
+  }
+  rd_umma::fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    rd_umma::fence_after();
+    rd_umma::tmem_dealloc(tmem, n_cols);
+  }
 }
 
-template <int DP, int WN>
-int launch_outputs(const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
-  auto kern = mlstm_outputs_kernel<DP, WN>;
-  constexpr int smem = OutSmem<DP, WN>::kBytes;
-  static bool set = false;
+template <typename Kern>
+int launch_big(Kern kern, bool& set, dim3 grid, int smem, const ChunkArgs& a, cudaStream_t s) {
+  cudaError_t err = cudaSuccess;
   if (!set) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    RD_CHECK_CHAINED(e);
+    err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    RD_CHECK_CHAINED(err);
     set = true;
   }
-  cudaError_t err = rd::launch_chained(kern, dim3((max_new + BT - 1) / BT, a.nh, B), dim3(kThreads), smem, s, 1, a);
+  err = rd::launch_chained(kern, grid, dim3(kThreads), smem, s, 1, a);
   RD_CHECK_CHAINED(err);
   return RD_OK;
 }
-
+template <int DN>
+int launch_states(const ChunkArgs& a, int B, cudaStream_t s) {
+  static bool set = false;
+  return launch_big(mlstm_states_kernel<DN>, set, dim3((a.vpad / 128) * (a.dpad / DN), a.nh, B), StateSmem<DN>::kBytes, a, s);
+}
 template <int DP>
-int launch_outputs_dim(const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
-  if (a.vdim <= 128) return launch_outputs<DP, 2>(a, B, max_new, s);
-  if (a.vdim <= 256) return launch_outputs<DP, 4>(a, B, max_new, s);
-  return launch_outputs<DP, 8>(a, B, max_new, s);
+int launch_outputs(const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
+  static bool set = false;
+  return launch_big(mlstm_outputs_kernel<DP>, set, dim3((max_new + L - 1) / L, a.nh, B), OutSmem<DP>::kBytes, a, s);
 }
 
-inline int64_t pad64(int64_t n) { return (n + 63) / 64 * 64; }
+inline int64_t pad_dim(int64_t n) { return n <= 64 ? 64 : (n + 127) / 128 * 128; }
+inline int64_t pad_v(int64_t n) { return (n + 127) / 128 * 128; }
 inline int64_t slots_of(int64_t m_max, int64_t B) { return m_max / L + B; }
 
 }  // namespace
 
 extern "C" int64_t rd_mlstm_chunk_workspace_bytes(int m_max, int B, int nh, int dim, int vdim) {
   const int64_t slots = slots_of(m_max, B) * nh;
-  return slots * pad64(dim) * pad64(vdim) * 4 + (5 * (int64_t)nh * m_max + slots * (1 + pad64(dim)) + 64) * (int64_t)sizeof(float);
+  return slots * pad_dim(dim) * pad_v(vdim) * 4 + (5 * (int64_t)nh * m_max + slots * (1 + pad_dim(dim)) + 64) * (int64_t)sizeof(float);
 }
 
 extern "C" int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i,
                               const float* bias_f, float gate_cap, const void* norm_weight, float eps, void* out, float* S,
                               float* n, float* m, const int32_t* row_start, const int32_t* base_len, int B, int nh, int dim,
-                              int vdim, int m_max, int max_new, void* workspace, int64_t workspace_bytes, void* stream) {
+                              int vdim, int m_max, int max_new, void* workspace, int64_t workspace_bytes, int32_t* status,
+                              void* stream) {
   RD_REQUIRE(proj && gates && bias_i && bias_f && norm_weight && out && S && n && m && row_start && base_len && workspace, RD_ERR_ARG);
   RD_REQUIRE(B >= 1 && B <= 65535 && nh >= 1 && nh <= 65535 && dim >= 8 && dim <= 256 && dim % 8 == 0 && vdim >= 8 && vdim <= 512 &&
                  vdim % 8 == 0 && m_max >= 1 && max_new >= 1 && max_new <= m_max && gate_cap > 0.f &&
@@ -654,9 +702,10 @@ extern "C" int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, 
   a.nh = nh;
   a.dim = dim;
   a.vdim = vdim;
-  a.dpad = (int)pad64(dim);
-  a.vpad = (int)pad64(vdim);
+  a.dpad = (int)pad_dim(dim);
+  a.vpad = (int)pad_v(vdim);
   a.m_max = m_max;
+  a.status = status;
   const int64_t slots = slots_of(m_max, B) * nh, tile = (int64_t)a.dpad * a.vpad;
   a.Shi = (__nv_bfloat16*)workspace;
   a.Slo = a.Shi + slots * tile;
@@ -673,15 +722,9 @@ extern "C" int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, 
   RD_REQUIRE(gates_smem <= 48 * 1024, RD_ERR_SIZE);
   cudaError_t err = rd::launch_chained(mlstm_gates_kernel, dim3(nh, B), dim3(kThreads), gates_smem, s, 1, a);
   RD_CHECK_CHAINED(err);
-  static bool set = false;
-  if (!set) {
-    err = cudaFuncSetAttribute(mlstm_states_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, StateSmem::kBytes);
-    RD_CHECK_CHAINED(err);
-    set = true;
-  }
-  err = rd::launch_chained(mlstm_states_kernel, dim3((a.dpad / 64) * (a.vpad / 64), nh, B), dim3(kThreads), StateSmem::kBytes, s, 1, a);
-  RD_CHECK_CHAINED(err);
-  if (dim <= 64) return launch_outputs_dim<64>(a, B, max_new, s);
-  if (dim <= 128) return launch_outputs_dim<128>(a, B, max_new, s);
-  return launch_outputs_dim<256>(a, B, max_new, s);
+  int rc = dim <= 64 ? launch_states<64>(a, B, s) : launch_states<128>(a, B, s);
+  if (rc != RD_OK) return rc;
+  if (dim <= 64) return launch_outputs<64>(a, B, max_new, s);
+  if (dim <= 128) return launch_outputs<128>(a, B, max_new, s);
+  return launch_outputs<256>(a, B, max_new, s);
 }

@@ -75,7 +75,7 @@ SIGNATURES = {
     "rd_rotary_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
     "rd_attention_window": (_I, [_I, _P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P]),
     "rd_mlstm_chunk_workspace_bytes": (_L, [_I, _I, _I, _I, _I]),
-    "rd_mlstm_chunk": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _L, _P]),
+    "rd_mlstm_chunk": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _L, _P, _P]),
     "rd_mlstm_tree": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _L, _P]),
     "rd_mlstm_scan": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P]),
     "rd_cache_commit": (_I, [_I, _P, _I, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _P]),

@@ -303,7 +303,7 @@ class MatrixMemory(nn.Module):
         need = _lib.load().rd_mlstm_chunk_workspace_bytes(ctx.m_max, ctx.batch, c.heads, c.dim, c.vdim)
         buf = self.scratch.get(need, proj.device)
         _lib.call("rd_mlstm_chunk", *self._common(proj, gates, mixed, state, ctx.row_start, ctx.base_len), ctx.batch, c.heads, c.dim,
-                  c.vdim, ctx.m_max, ctx.max_new, _lib.ptr(buf), buf.numel(), _lib.stream())
+                  c.vdim, ctx.m_max, ctx.max_new, _lib.ptr(buf), buf.numel(), _lib.ptr(ctx.status), _lib.stream())
 
     def _tree(self, ctx: StepContext, state, proj, gates, mixed) -> None:
         c = self.cfg

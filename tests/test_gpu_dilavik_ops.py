@@ -297,8 +297,9 @@ class Memory:
             _lib.call("rd_mlstm_scan", _lib.dtype_code(self.dtype), *common, max(len(p[0]) for p in portions), None, 0, 0, None, None, st)
         else:
             need = _lib.load().rd_mlstm_chunk_workspace_bytes(M, self.B, m["heads"], m["dim"], m["vdim"])
-            ws = torch.empty(need, dtype=torch.uint8, device="cuda")
-            _lib.call("rd_mlstm_chunk", *common, M, max(len(p[0]) for p in portions), ptr(ws), need, st)
+            ws, status = torch.empty(need, dtype=torch.uint8, device="cuda"), i32([0])
+            _lib.call("rd_mlstm_chunk", *common, M, max(len(p[0]) for p in portions), ptr(ws), need, ptr(status), st)
+            assert int(status.item()) == 0
         for r in range(self.B):
             if len(portions[r][0]):
                 self.state[r], want = self.plain(r, portions[r])
