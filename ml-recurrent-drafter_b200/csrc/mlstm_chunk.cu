@@ -1,5 +1,5 @@
 // The matrix-memory recurrence of mlstm.cu for prompts: chunks of 128 tokens on the tensor cores (tcgen05, bf16 operands,
-// fp32 accumulators in TMEM; operands staged by cp.async in the 128-byte swizzle).  Waits are bounded: on give-up a
+// fp32 accumulators in TMEM; operands staged by TMA, or by cp.async where a tile's edge must be zero).  Waits are bounded: on give-up a
 // kernel writes a code to *status, frees its TMEM and returns.
 //
 // Within a chunk, with F_t the running sum of the log forget gates and m_t the running maximum of the recurrence,
@@ -31,6 +31,7 @@ __device__ __forceinline__ bool wait_warp(uint64_t* bar, uint32_t parity) {
   return __all_sync(0xffffffffu, rd_umma::mbar_wait(bar, parity));
 }
 constexpr int kThreads = 256;
+constexpr int kGateThreads = 1024;
 
 struct ChunkArgs {
   const __nv_bfloat16* proj;  // [m, ld]: q | k | v | g
@@ -80,7 +81,7 @@ __device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_
 }
 
 // ------------------------------------------------------------------------------------------------ gates
-__global__ void __launch_bounds__(kThreads) mlstm_gates_kernel(const ChunkArgs a) {
+__global__ void __launch_bounds__(kGateThreads) mlstm_gates_kernel(const ChunkArgs a) {
   extern __shared__ __align__(128) uint8_t smem[];
   rd::pdl_launch_dependents();
   rd::pdl_wait();
@@ -94,7 +95,7 @@ __global__ void __launch_bounds__(kThreads) mlstm_gates_kernel(const ChunkArgs a
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float bi = a.bias_i[h], bf = a.bias_f[h];
   const int64_t at = (int64_t)h * a.m_max + rs;
-  for (int c = warp; c < n_chunks; c += kThreads / 32) {
+  for (int c = warp; c < n_chunks; c += kGateThreads / 32) {
     // lane owns four consecutive tokens
     float f[4], x[4], F = 0.f, mx = -INFINITY;
 #pragma unroll
@@ -154,7 +155,7 @@ __global__ void __launch_bounds__(kThreads) mlstm_gates_kernel(const ChunkArgs a
   }
   __syncthreads();
   const float qs = rsqrtf((float)a.dim);
-  for (int c = warp; c < n_chunks; c += kThreads / 32) {
+  for (int c = warp; c < n_chunks; c += kGateThreads / 32) {
     const float m_in = c_m[c], FL = c_F[c], mL = FL + fmaxf(m_in, c_M[c]);
     if (lane == 0) a.decay[(int64_t)chunk_slot(rs, b, c) * a.nh + h] = expf(FL + m_in - mL);
 #pragma unroll
@@ -179,7 +180,7 @@ template <int DN>
 struct StateSmem {
   static constexpr int kK = (DN / 64) * kBox, kV = 2 * kBox;  // [128 tokens] x DN dims, x 128 value columns
   static constexpr int kStage = kK + kV;
-  static constexpr int kMisc = (2 * L + DN + 8) * 4 + 64;
+  static constexpr int kMisc = (2 * L + DN + 8) * 4 + 64;  // w, n, barriers
   static constexpr int kBytes = 2 * kStage + 2 * kV + kMisc + 1024;  // two stages, w V hi and lo, alignment
 };
 
@@ -187,7 +188,7 @@ struct StateSmem {
 // Per chunk: the tile is read out, written to the workspace, scaled and put back, then (w V)^T K is added by tcgen05.mma
 // (both operands MN-major: value columns and dims contiguous, tokens along K).
 template <int DN>
-__global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkArgs a) {
+__global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_constant__ CUtensorMap map_proj, const ChunkArgs a) {
   using Y = StateSmem<DN>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -204,10 +205,11 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
   uint8_t* sLo = sHi + Y::kV;
   float* s_w = reinterpret_cast<float*>(sLo + Y::kV);  // [2][L]
   float* s_n = s_w + 2 * L;                             // [DN]
-  uint64_t* bar = reinterpret_cast<uint64_t*>(s_n + DN);
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 1);
+  uint64_t* bar = reinterpret_cast<uint64_t*>(s_n + DN);  // a chunk's products are done
+  uint64_t* full = bar + 1;                               // [2] a stage's K and V have landed
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 3);
   if (tid == 0) {
-    rd_umma::mbar_init(bar, 1);
+    for (int i = 0; i < 3; ++i) rd_umma::mbar_init(&bar[i], 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 0) rd_umma::tmem_alloc(tmem_slot, DN);
@@ -217,24 +219,17 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
   float* n_g = a.n + ((int64_t)b * a.nh + h) * a.dim;
   if (tid < DN) s_n[tid] = (d0 + tid < a.dim && !fresh) ? n_g[d0 + tid] : 0.f;
 
+  // One thread: K and V of chunk c by TMA.  Boxes may reach into the next row's tokens (their w is 0 and they are finite),
+  // into the next head's dims (never read from the state: q is zero there) or columns (never stored).
   auto load = [&](int c) {
     uint8_t* sK = smem + (c & 1) * Y::kStage;
-    uint8_t* sV = sK + Y::kK;
-    for (int i = tid; i < L * (DN / 8); i += kThreads) {
-      const int r = i / (DN / 8), ch = i % (DN / 8);
-      const bool in = c * L + r < n_tok && d0 + ch * 8 < a.dim;
-      cp_async16(sK + (ch >> 3) * kBox + swz<8>(r, ch & 7),
-                 a.proj + (int64_t)(rs + (in ? c * L + r : 0)) * a.ld + (a.nh + h) * a.dim + (in ? d0 + ch * 8 : 0), in);
-    }
-    for (int i = tid; i < L * 16; i += kThreads) {
-      const int r = i >> 4, ch = i & 15;
-      const bool in = c * L + r < n_tok && v0 + ch * 8 < a.vdim;
-      cp_async16(sV + (ch >> 3) * kBox + swz<8>(r, ch & 7),
-                 a.proj + (int64_t)(rs + (in ? c * L + r : 0)) * a.ld + 2 * a.nh * a.dim + h * a.vdim + (in ? v0 + ch * 8 : 0), in);
-    }
-    cp_async_commit();
+    rd_umma::mbar_expect_tx(&full[c & 1], Y::kStage);
+    const int row = rs + c * L, k0 = (a.nh + h) * a.dim + d0, w0 = 2 * a.nh * a.dim + h * a.vdim + v0;
+#pragma unroll
+    for (int i = 0; i < DN / 64; ++i) rd_umma::tma_load_2d(sK + i * kBox, &map_proj, &full[c & 1], k0 + i * 64, row);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) rd_umma::tma_load_2d(sK + Y::kK + i * kBox, &map_proj, &full[c & 1], w0 + i * 64, row);
   };
-  load(0);
   auto w_of = [&](int c) { return (tid < L && c * L + tid < n_tok) ? a.w[at + c * L + tid] : 0.f; };
   auto decay_of = [&](int c) { return a.decay[(int64_t)chunk_slot(rs, b, c) * a.nh + h]; };
   if (tid < L) s_w[tid] = w_of(0);
@@ -242,6 +237,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
   rd_umma::fence_before();
   __syncthreads();
   rd_umma::fence_after();
+  if (tid == 0) load(0);  // the barriers are initialised
   const uint32_t tmem = *tmem_slot;
   const int quarter = warp & 3, half = warp >> 2;
   const int v = v0 + quarter * 32 + lane;  // this thread's value column
@@ -251,11 +247,11 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
   for (int c = 0; c < n_chunks; ++c) {
     // the products of chunk c - 1 are in the tile, and its operands' shared memory is free
     if (c > 0) ok = wait_warp(bar, (c - 1) & 1);
-    cp_async_wait<0>();
     if (!__syncthreads_and(ok)) break;
+    if (tid == 0 && c + 1 < n_chunks) load(c + 1);
+    ok = wait_warp(&full[c & 1], (c >> 1) & 1);
     rd_umma::fence_after();
     const float w_next = c + 1 < n_chunks ? w_of(c + 1) : 0.f, A_next = c + 1 < n_chunks ? decay_of(c + 1) : 0.f;
-    if (c + 1 < n_chunks) load(c + 1);
     const uint8_t* sK = smem + (c & 1) * Y::kStage;
     const uint8_t* sV = sK + Y::kK;
     const float* w = s_w + (c & 1) * L;
@@ -307,7 +303,10 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
     }
     rd_umma::fence_async_proxy();
     rd_umma::fence_before();
-    __syncthreads();
+    if (!__syncthreads_and(ok)) {
+      ok = false;
+      break;
+    }
     if (tid == 0) {
       rd_umma::fence_after();
       const uint32_t idesc = rd_umma::idesc_f16(DN, true, true);
@@ -337,7 +336,6 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
     if (tid < L) s_w[((c + 1) & 1) * L + tid] = w_next;
     A = A_next;
   }
-  cp_async_wait<0>();
   if (ok) ok = wait_warp(bar, (n_chunks - 1) & 1);
   ok = __syncthreads_and(ok);
   if (ok) {
@@ -353,8 +351,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const ChunkAr
     }
     constexpr int PER = kThreads / DN;
     if (owns_n && tid % PER == 0 && d0 + tid / PER < a.dim) n_g[d0 + tid / PER] = s_n[tid / PER];
-  } else if (tid == 0 && a.status) {
-    atomicExch(a.status, 31);
+  } else if (tid == 0) {
+    if (a.status) atomicExch(a.status, 31);
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);  // copies in flight land before the shared memory goes away
   }
   rd_umma::fence_before();
   __syncthreads();
@@ -373,7 +372,7 @@ struct OutSmem {
   static constexpr int kQ = (DP / 64) * kBox;
   static constexpr int kRing = kOutStages * kItem > kQ ? kOutStages * kItem : kQ;  // K first, then the ring
   static constexpr int kP = 2 * kBox;
-  static constexpr int kMisc = (5 * L + DP + 4 * L) * 4 + 128;
+  static constexpr int kMisc = (5 * L + DP + 4 * L) * 4 + 160;  // per-token scalars, n, barriers
   static constexpr int kBytes = kQ + kRing + 2 * kP + kMisc + 1024;
 };
 
@@ -381,7 +380,9 @@ struct OutSmem {
 //   scores Q K^T (in O's columns, before O exists) -> P hi / lo in shared memory -> O = Q S (hi, lo) -> O *= e_t ->
 //   O += P V (hi, lo) -> / denominator, RMS, norm weight, output gate.
 template <int DP>
-__global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkArgs a) {
+__global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid_constant__ CUtensorMap map_v,
+                                                                    const __grid_constant__ CUtensorMap map_hi,
+                                                                    const __grid_constant__ CUtensorMap map_lo, const ChunkArgs a) {
   using Y = OutSmem<DP>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -405,11 +406,15 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
   float* s_n = s_nq + L;       // [DP]
   float* s_rs = s_n + DP;      // [2][L]
   float* s_ss = s_rs + 2 * L;  // [2][L]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 2 * L);  // [kOutStages] an item's products are done; [+1] the scores
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + kOutStages + 1);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 2 * L);  // [kOutStages] an item's products are done
+  uint64_t* full = bars + kOutStages;                           // [kOutStages] an item has landed
+  uint64_t* scores_done = full + kOutStages;
+  uint64_t* state_done = scores_done + 1;
+  uint64_t* all_done = scores_done + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(scores_done + 3);
   const uint32_t n_cols = a.vpad <= 128 ? 128 : (a.vpad <= 256 ? 256 : 512);
   if (tid == 0) {
-    for (int i = 0; i <= kOutStages; ++i) rd_umma::mbar_init(&bars[i], 1);
+    for (int i = 0; i < 2 * kOutStages + 3; ++i) rd_umma::mbar_init(&bars[i], 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 0) rd_umma::tmem_alloc(tmem_slot, n_cols);
@@ -445,7 +450,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
       const int off = (k >> 2) * kBox + (k & 3) * 32;
       rd_umma::mma_ss(tmem, rd_umma::desc_k_major(rd_umma::smem_u32(sQ + off)), rd_umma::desc_k_major(rd_umma::smem_u32(ring + off)), idesc, k != 0);
     }
-    rd_umma::commit(&bars[kOutStages]);
+    rd_umma::commit(scores_done);
   }
   // n_in . q_t meanwhile: two threads per token
   {
@@ -467,8 +472,60 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
   const int quarter = warp & 3, half = warp >> 2;
   const int t = quarter * 32 + lane;  // this thread's token of the chunk
   const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16);
-  bool ok = wait_warp(&bars[kOutStages], 0);
+  bool ok = wait_warp(scores_done, 0);
   rd_umma::fence_after();
+  // The streamed second operands, one thread: S tiles (dim block, value tile, hi / lo), then V tiles (64 tokens, value tile).
+  // V boxes may reach past the row's tokens (P is 0 there) and past the head's columns (never used).
+  const int v_tiles = a.vpad / 128, d_blocks = a.dpad / 64;
+  const int n_state = d_blocks * v_tiles * 2, n_items = n_state + ((t0 + 64 < n_tok) ? 2 : 1) * v_tiles;
+  auto load = [&](int i) {
+    uint8_t* dst = ring + (i % kOutStages) * kItem;
+    uint64_t* bar = &full[i % kOutStages];
+    rd_umma::mbar_expect_tx(bar, kItem);
+    if (i < n_state) {
+      const int vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
+      rd_umma::tma_load_2d(dst, (i & 1) ? &map_lo : &map_hi, bar, db * 64, (int)(slot * a.vpad) + vt * 128);
+    } else {
+      const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
+      const int col = 2 * a.nh * a.dim + h * a.vdim + vt * 128;
+      rd_umma::tma_load_2d(dst, &map_v, bar, col, rs + t0 + jb * 64);
+      rd_umma::tma_load_2d(dst + kItem / 2, &map_v, bar, col + 64, rs + t0 + jb * 64);
+    }
+  };
+  // items [i0, i1): products of each as it lands; its stage is refilled once the products of the item before are done
+  auto run_items = [&](int i0, int i1) {
+    for (int i = i0; i < i1; ++i) {
+      if (!rd_umma::mbar_wait(&full[i % kOutStages], (i / kOutStages) & 1)) return false;
+      rd_umma::fence_after();
+      const uint8_t* sB = ring + (i % kOutStages) * kItem;
+      if (i < n_state) {
+        const int vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
+        const uint32_t idesc = rd_umma::idesc_f16(128, false, false);
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sQ + db * kBox + k * 32)),
+                          rd_umma::desc_k_major(rd_umma::smem_u32(sB + k * 32)), idesc, (db | (i & 1) | k) != 0);
+      } else {
+        const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
+        const uint32_t idesc = rd_umma::idesc_f16(128, false, true);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const uint64_t dv = rd_umma::desc_mn_major(rd_umma::smem_u32(sB + k * 2048), kItem / 2);
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPh + jb * kBox + k * 32)), dv, idesc, 1);
+          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPl + jb * kBox + k * 32)), dv, idesc, 1);
+        }
+      }
+      rd_umma::commit(&bars[i % kOutStages]);
+      if (i > 0 && i + kOutStages - 1 < n_items) {
+        if (!rd_umma::mbar_wait(&bars[(i - 1) % kOutStages], ((i - 1) / kOutStages) & 1)) return false;
+        load(i + kOutStages - 1);
+      }
+    }
+    return true;
+  };
+  if (ok && tid == 0)
+    for (int i = 0; i < kOutStages && i < n_items; ++i) load(i);  // K has been read: its place is the ring
+  __syncwarp();
   // P of this thread's token and half of the keys
   if (ok) {
     const float Fm = s_Fm[t];
@@ -497,92 +554,43 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
     }
     s_rs[half * L + t] = sum;
   }
+  rd_umma::fence_async_proxy();
   rd_umma::fence_before();
-  ok = __syncthreads_and(ok);  // P is complete, K is dead, the scores have been read
+  ok = __syncthreads_and(ok);  // P is complete, the scores have been read
 
-  // ---- the streamed second operands: S tiles (dim block, value tile, hi / lo), then V tiles (64 tokens, value tile)
-  const int v_tiles = a.vpad / 128, d_blocks = a.dpad / 64;
-  const int n_state = d_blocks * v_tiles * 2, n_items = n_state + ((t0 + 64 < n_tok) ? 2 : 1) * v_tiles;
-  auto load = [&](int i) {
-    if (i < n_items) {
-      uint8_t* dst = ring + (i % kOutStages) * kItem;
-      if (i < n_state) {
-        const int lo = i & 1, vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
-        const __nv_bfloat16* src = (lo ? a.Slo : a.Shi) + (slot * a.vpad + vt * 128) * a.dpad + db * 64;
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int idx = u * kThreads + tid, r = idx >> 3, ch = idx & 7;
-          cp_async16(dst + swz<8>(r, ch), src + (int64_t)r * a.dpad + ch * 8, true);
-        }
-      } else {
-        const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int idx = u * kThreads + tid, r = idx >> 4, ch = idx & 15;
-          const int tok = t0 + jb * 64 + r, v = vt * 128 + ch * 8;
-          const bool in = tok < n_tok && v < a.vdim;
-          cp_async16(dst + (ch >> 3) * (kItem / 2) + swz<8>(r, ch & 7),
-                     a.proj + (int64_t)(rs + (in ? tok : 0)) * a.ld + 2 * a.nh * a.dim + h * a.vdim + (in ? v : 0), in);
-        }
-      }
-    }
-    cp_async_commit();  // one group per item, empty or not
-  };
+
+  // ---- O = Q S, then O = e_t O + P V
   if (ok) {
-#pragma unroll
-    for (int i = 0; i < kOutStages - 1; ++i) load(i);
-  }
-  for (int i = 0; i < n_items; ++i) {  // left by all threads together, see the barrier below
-    if (i == n_state && ok) {
-      // the state's part is complete: scale it by the tokens' e_t before the scores' part is added
-      ok = wait_warp(&bars[(i - 1) % kOutStages], ((i - 1) / kOutStages) & 1);
-      rd_umma::fence_after();
-      const float e = s_e[t];
-      if (ok) {
-        for (int q = half * (v_tiles * 2); q < (half + 1) * (v_tiles * 2); ++q) {
-          float o[32];
-          rd_umma::tmem_ld32(t_row + q * 32, o);
-#pragma unroll
-          for (int k = 0; k < 32; ++k) o[k] *= e;
-          rd_umma::tmem_st32(t_row + q * 32, o);
-        }
-      }
-      rd_umma::fence_before();
-    }
-    cp_async_wait<kOutStages - 2>();  // item i is here
-    rd_umma::fence_async_proxy();
-    if (!__syncthreads_and(ok)) {
-      ok = false;
-      break;
-    }
-    const uint8_t* sB = ring + (i % kOutStages) * kItem;
     if (tid == 0) {
       rd_umma::fence_after();
-      if (i < n_state) {
-        const int lo = i & 1, vt = (i >> 1) % v_tiles, db = (i >> 1) / v_tiles;
-        const uint32_t idesc = rd_umma::idesc_f16(128, false, false);
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sQ + db * kBox + k * 32)),
-                          rd_umma::desc_k_major(rd_umma::smem_u32(sB + k * 32)), idesc, (db | lo | k) != 0);
-      } else {
-        const int vt = (i - n_state) % v_tiles, jb = (i - n_state) / v_tiles;
-        const uint32_t idesc = rd_umma::idesc_f16(128, false, true);
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const uint64_t dv = rd_umma::desc_mn_major(rd_umma::smem_u32(sB + k * 2048), kItem / 2);
-          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPh + jb * kBox + k * 32)), dv, idesc, 1);
-          rd_umma::mma_ss(tmem + vt * 128, rd_umma::desc_k_major(rd_umma::smem_u32(sPl + jb * kBox + k * 32)), dv, idesc, 1);
-        }
-      }
-      rd_umma::commit(&bars[i % kOutStages]);
+      ok = run_items(0, n_state);
+      if (ok) rd_umma::commit(state_done);
     }
-    // the stage of item i - 1 takes item i + kOutStages - 1 once that item's products are done
-    if (ok && i > 0 && i + kOutStages - 1 < n_items) ok = wait_warp(&bars[(i - 1) % kOutStages], ((i - 1) / kOutStages) & 1);
-    load(ok ? i + kOutStages - 1 : n_items);
+    __syncwarp();
+    ok = wait_warp(state_done, 0) && ok;
+    rd_umma::fence_after();
+    const float e = s_e[t];
+    if (__all_sync(0xffffffffu, ok)) {
+      for (int q = half * (v_tiles * 2); q < (half + 1) * (v_tiles * 2); ++q) {
+        float o[32];
+        rd_umma::tmem_ld32(t_row + q * 32, o);
+#pragma unroll
+        for (int k = 0; k < 32; ++k) o[k] *= e;
+        rd_umma::tmem_st32(t_row + q * 32, o);
+      }
+    }
+    rd_umma::fence_before();
   }
-  cp_async_wait<0>();
-  if (ok) ok = wait_warp(&bars[(n_items - 1) % kOutStages], ((n_items - 1) / kOutStages) & 1);
+  ok = __syncthreads_and(ok);
+  if (ok) {
+    if (tid == 0) {
+      rd_umma::fence_after();
+      ok = run_items(n_state, n_items);
+      if (ok) rd_umma::commit(all_done);
+    }
+    __syncwarp();
+    ok = wait_warp(all_done, 0) && ok;
+  }
   ok = __syncthreads_and(ok);
   if (ok) {
     rd_umma::fence_after();
@@ -594,7 +602,8 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
       float o[32];
       rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
-      for (int k = 0; k < 32; ++k) ss = fmaf(o[k] * inv, o[k] * inv, ss);
+      for (int k = 0; k < 32; ++k)
+        if (q * 32 + k < a.vdim) ss = fmaf(o[k] * inv, o[k] * inv, ss);
     }
     s_ss[half * L + t] = ss;
     __syncthreads();
@@ -626,8 +635,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
         }
       }
     }
-  } else if (tid == 0 && a.status) {
-    atomicExch(a.status, 32);
+  } else if (tid == 0) {
+    if (a.status) atomicExch(a.status, 32);
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);
   }
   rd_umma::fence_before();
   __syncthreads();
@@ -637,27 +647,30 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const ChunkA
   }
 }
 
-template <typename Kern>
-int launch_big(Kern kern, bool& set, dim3 grid, int smem, const ChunkArgs& a, cudaStream_t s) {
+template <typename Kern, typename... Maps>
+int launch_big(Kern kern, bool& set, dim3 grid, int smem, cudaStream_t s, const Maps&... args) {
   cudaError_t err = cudaSuccess;
   if (!set) {
     err = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     RD_CHECK_CHAINED(err);
     set = true;
   }
-  err = rd::launch_chained(kern, grid, dim3(kThreads), smem, s, 1, a);
+  err = rd::launch_chained(kern, grid, dim3(kThreads), smem, s, 1, args...);
   RD_CHECK_CHAINED(err);
   return RD_OK;
 }
+struct Maps {
+  CUtensorMap proj, v, hi, lo;  // proj in boxes of 128 and of 64 rows; the two halves of S^T
+};
 template <int DN>
-int launch_states(const ChunkArgs& a, int B, cudaStream_t s) {
+int launch_states(const Maps& m, const ChunkArgs& a, int B, cudaStream_t s) {
   static bool set = false;
-  return launch_big(mlstm_states_kernel<DN>, set, dim3((a.vpad / 128) * (a.dpad / DN), a.nh, B), StateSmem<DN>::kBytes, a, s);
+  return launch_big(mlstm_states_kernel<DN>, set, dim3((a.vpad / 128) * (a.dpad / DN), a.nh, B), StateSmem<DN>::kBytes, s, m.proj, a);
 }
 template <int DP>
-int launch_outputs(const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
+int launch_outputs(const Maps& m, const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
   static bool set = false;
-  return launch_big(mlstm_outputs_kernel<DP>, set, dim3((max_new + L - 1) / L, a.nh, B), OutSmem<DP>::kBytes, a, s);
+  return launch_big(mlstm_outputs_kernel<DP>, set, dim3((max_new + L - 1) / L, a.nh, B), OutSmem<DP>::kBytes, s, m.v, m.hi, m.lo, a);
 }
 
 inline int64_t pad_dim(int64_t n) { return n <= 64 ? 64 : (n + 127) / 128 * 128; }
@@ -720,11 +733,16 @@ extern "C" int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, 
   cudaStream_t s = (cudaStream_t)stream;
   const size_t gates_smem = (size_t)3 * ((max_new + L - 1) / L) * sizeof(float);
   RD_REQUIRE(gates_smem <= 48 * 1024, RD_ERR_SIZE);
-  cudaError_t err = rd::launch_chained(mlstm_gates_kernel, dim3(nh, B), dim3(kThreads), gates_smem, s, 1, a);
+  cudaError_t err = rd::launch_chained(mlstm_gates_kernel, dim3(nh, B), dim3(kGateThreads), gates_smem, s, 1, a);
   RD_CHECK_CHAINED(err);
-  int rc = dim <= 64 ? launch_states<64>(a, B, s) : launch_states<128>(a, B, s);
+  Maps maps;
+  const int64_t width = (int64_t)2 * nh * (dim + vdim), s_rows = slots * a.vpad;
+  if (!rd_umma::make_map(&maps.proj, proj, m_max, width, ld, 128) || !rd_umma::make_map(&maps.v, proj, m_max, width, ld, 64) ||
+      !rd_umma::make_map(&maps.hi, a.Shi, s_rows, a.dpad, a.dpad, 128) || !rd_umma::make_map(&maps.lo, a.Slo, s_rows, a.dpad, a.dpad, 128))
+    return RD_ERR_ARG;
+  int rc = dim <= 64 ? launch_states<64>(maps, a, B, s) : launch_states<128>(maps, a, B, s);
   if (rc != RD_OK) return rc;
-  if (dim <= 64) return launch_outputs<64>(a, B, max_new, s);
-  if (dim <= 128) return launch_outputs<128>(a, B, max_new, s);
-  return launch_outputs<256>(a, B, max_new, s);
+  if (dim <= 64) return launch_outputs<64>(maps, a, B, max_new, s);
+  if (dim <= 128) return launch_outputs<128>(maps, a, B, max_new, s);
+  return launch_outputs<256>(maps, a, B, max_new, s);
 }
