@@ -23,6 +23,9 @@ reference: the reference's own PyTorch implementation (installed under baseline/
            timed beside it as a cross-check.  Without baseline/_ref, or without the host memory
            for the fp32 weights, the port alone is timed and the line says so.
 
+--design dilavik [--size 2k|4k]: prefill and decode throughput of that base model beside Llama at equal width, with every
+kernel's time against its roofline (a line of its own shape; not the workload above).
+
 One JSON line is printed by rank 0.
 """
 import argparse
@@ -706,6 +709,220 @@ def run_cpu(args, as_reference_arm: bool):
     return base
 
 
+# ------------------------------------------------------------------------------------------------
+# Prefill and decode throughput of a base model of another design beside Llama at equal width (random weights).
+# name: width, query heads, key/value heads, matrix-memory heads and sizes, window, Llama feed-forward width, layers of each
+DESIGN_SIZES = {
+    "2k": dict(width=2048, heads=16, kv=4, mem=(4, 256, 512), window=1024, ff=5632, blocks=2),
+    "4k": dict(width=4096, heads=32, kv=8, mem=(8, 256, 512), window=1024, ff=11008, blocks=2),
+}
+DESIGN_PREFILL = ((1, 8192), (8, 1024))
+DESIGN_DECODE = ((1, 2048), (8, 2048), (32, 2048))
+
+
+def design_models(size: str, device):
+    """(name, model) pairs: per block attention + feed-forward, two matrix-memory layers, attention + feed-forward; beside
+    it Llama with the same number of attention + feed-forward layers, heads and key/value heads, and as many feed-forward
+    weights (three matrices of ff there, two of 1.5 ff here)."""
+    import torch
+    from transformers.models.llama.configuration_llama import LlamaConfig
+
+    import recurrent_drafting as rd
+
+    z = DESIGN_SIZES[size]
+    att = {"type": "attention", "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2},
+           "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "rot": {"dims": 64, "base": 10000.0},
+                     "scale": 128 ** -0.5, "mask": {"size": z["window"], "keep_first": 4}}}
+    mem = {"type": "mlstm", "mlp": None, "mixer": dict(zip(("heads", "dim", "vdim"), z["mem"]), gate_cap=15.0)}
+    cfg = {"architecture": "Dilavik", "vocab": 32000, "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6, "groups": 8},
+           "layers": [att, mem, mem, att] * z["blocks"]}
+    with torch.device(device):
+        m = rd.modeling_dilavik.DilavikForCausalLM(rd.configuration_dilavik.DilavikConfig.from_dict(cfg)).to(torch.bfloat16)
+    yield "dilavik", m.init_random(0.02, seed=1)
+    del m
+    torch.cuda.empty_cache()
+    lc = LlamaConfig(hidden_size=z["width"], num_attention_heads=z["heads"], num_key_value_heads=z["kv"], num_hidden_layers=2 * z["blocks"],
+                     intermediate_size=z["ff"], vocab_size=32000, rms_norm_eps=1e-6, hidden_act="silu", pad_token_id=0)
+    lc.rope_theta = 10000.0
+    with torch.device(device):
+        m = rd.modeling_llama.LlamaForCausalLM(lc).to(torch.bfloat16)
+    yield "llama", m.init_random(0.02, seed=1)
+
+
+class KernelLog:
+    """Event pairs around every C-ABI launch of a few steps, with each call's least time by the measured peaks: the larger of
+    its FLOPs over the bf16 GEMM peak and its algorithmic bytes over the copy bandwidth."""
+
+    def __init__(self, model, size: str, batch: int, new: int, cached: int):
+        self.z, self.B, self.new, self.cached, self.M = DESIGN_SIZES[size], batch, new, cached, batch * new
+        self.llama = type(model).__name__.startswith("Llama")
+        self.peaks, self.calls, self.shape = _peaks(), [], None
+
+    def least(self, name, args):
+        z, M, B = self.z, self.M, self.B
+        H, heads, kv = z["width"], z["heads"], z["kv"]
+        flops = nbytes = 0.0
+        if name.startswith("rd_gemm") and self.shape is not None:
+            N, K, out = self.shape
+            flops, nbytes = 2.0 * M * N * K, 2.0 * N * K + 2.0 * M * K + out * M * N
+        elif name == "rd_stream_norm":
+            nbytes = M * H * ((2 if args[1] is not None else 4 * args[7]) + (4 if args[8] is not None else 0) + 2.0)
+        elif name in ("rd_rmsnorm", "rd_embed_gather"):
+            nbytes = 4.0 * M * H
+        elif name.startswith("rd_attention"):
+            first, end = self.cached, self.cached + self.new
+            w = end if self.llama else z["window"]
+            pairs = sum(min(p + 1, w) for p in range(first, end)) if self.new > 1 else min(end, w + (0 if self.llama else 4))
+            keys = min(end, w + self.new)
+            flops = 4.0 * 128 * heads * B * pairs
+            nbytes = B * keys * kv * 256 * 2.0 + M * heads * 256 * 2.0
+        elif name == "rd_mlstm_chunk":
+            nh, d, v = z["mem"]
+            flops = M * nh * (4.0 * d * v + 128.0 * (d + v))
+            nbytes = M * nh * (2 * d + 3 * v) * 2.0 + M * nh * 8.0 + B * nh * d * v * 8.0
+        elif name == "rd_mlstm_scan":
+            nh, d, v = z["mem"]
+            nbytes = B * nh * d * v * 8.0 + M * nh * (2 * d + 3 * v) * 2.0
+        else:
+            return None
+        return max(flops / (self.peaks["tflops"] * 1e12), nbytes / (self.peaks["hbm_gbs"] * 1e9)) * 1e3
+
+    def run(self, fn, repeat: int = 3):
+        import torch
+
+        from recurrent_drafting import _lib
+        from recurrent_drafting.modeling_common import Linear
+
+        real_call, saved = _lib.call, {}
+        # bytes per output element: two, four with a fp32 result, eight where a fp32 residual is read as well; none for the arg-max
+        for method in ("__call__", "xielu", "split", "qkvg_rope", "qkv_rope", "argmax"):
+            saved[method] = getattr(Linear, method)
+
+            def wrapped(lin, a, c, *pa, _real=saved[method], _m=method, **kw):
+                per = 0.0 if _m == "argmax" else 2.0
+                if _m == "__call__":
+                    per = float(c.element_size()) * (2 if kw.get("residual") is not None else 1)
+                n = lin.weight.shape[0]
+                self.shape = (n // 2 * 2, lin.weight.shape[1], per * (0.5 if _m == "__call__" and pa and pa[0] == _lib.EPI_SWIGLU else 1.0))
+                _real(lin, a, c, *pa, **kw)
+                self.shape = None
+
+            setattr(Linear, method, wrapped)
+
+        def call(name, *a):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            label = name if self.shape is None else f"{name} N={self.shape[0]} K={self.shape[1]}"
+            least = self.least(name, a)
+            e0.record()
+            real_call(name, *a)
+            e1.record()
+            self.calls.append((label, least, e0, e1))
+
+        _lib.call = call
+        try:
+            for _ in range(repeat):
+                fn()
+            torch.cuda.synchronize()
+        finally:
+            _lib.call = real_call
+            for method, f in saved.items():
+                setattr(Linear, method, f)
+        agg = {}
+        for label, least, e0, e1 in self.calls:
+            v = agg.setdefault(label, [0, 0.0, 0.0])
+            v[0] += 1
+            v[1] += e0.elapsed_time(e1)
+            v[2] += least or 0.0
+        return {k: {"launches": v[0] // repeat, "us": round(1e3 * v[1] / v[0], 1), "roofline_us": round(1e3 * v[2] / v[0], 1),
+                    "frac": round(v[2] / v[1], 3)} for k, v in sorted(agg.items(), key=lambda kv: -kv[1][1]) if v[2] > 0}
+
+
+def run_design(args):
+    for _p in (ROOT, PKG):
+        if _p not in sys.path:
+            sys.path.insert(0, _p)
+    import torch
+
+    import recurrent_drafting as rd
+    from recurrent_drafting import _lib
+    from recurrent_drafting.session import DecodeGraphs, Session
+
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    K, Wm = min(args.steps, 32), max(args.warmup, 3)
+    greedy = rd.SamplingArgs(1.0, True)
+
+    def timed(fn, n):
+        for _ in range(Wm):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(n):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    out = {"metric": "prefill and decode throughput by design", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+           "size": args.size, "config": dict(DESIGN_SIZES[args.size], l2="inputs larger than L2 (the weights are streamed every step)"),
+           "warmup": Wm, "peaks": _peaks(), "models": {}}
+    sampler = ClockSampler(0)
+    sampler.start()
+    time.sleep(0.15)
+    t_wall0, launches0 = datetime.datetime.now(), _lib.launches
+    for name, llm in design_models(args.size, dev):
+        res = {"prefill": [], "decode": []}
+        for B, T in DESIGN_PREFILL:
+            s = Session(llm, B, T + 1)
+            ids = torch.randint(3, 32000, (B * T,), device=dev)
+
+            def prefill():
+                for r in range(B):
+                    s.release(r)
+                s.extend(ids, [T] * B)
+
+            ms = timed(prefill, max(3, K // 4))
+            res["prefill"].append({"batch": B, "tokens": T, "ms": round(ms, 3), "tokens_per_s": round(B * T / ms * 1e3),
+                                   "kernels": KernelLog(llm, args.size, B, T, 0).run(prefill)})
+            s.check()
+        for B, ctx in DESIGN_DECODE:
+            s = Session(llm, B, ctx + K + Wm + 40)
+            s.extend(torch.randint(3, 32000, (B * ctx,), device=dev), [ctx] * B)
+            tokens = torch.zeros(B, s.max_length, dtype=torch.int64, device=dev)
+            columns = torch.zeros(B, dtype=torch.int32, device=dev)
+
+            def step():
+                s.pick(greedy, tokens, columns)
+                s.forward(s.max_length)
+
+            step()
+            kernels = KernelLog(llm, args.size, B, 1, ctx).run(step)
+            graphs = DecodeGraphs(s, greedy, tokens, columns)
+
+            def replay():
+                graphs.pick.replay()
+                graphs.forward.replay()
+                _lib.count_replay(graphs.n_pick + graphs.n_forward)
+
+            ms = timed(replay, K)
+            res["decode"].append({"batch": B, "context": ctx, "ms_per_step": round(ms, 4), "tokens_per_s": round(B / ms * 1e3), "kernels": kernels})
+            s.check()
+            del graphs, s
+        out["models"][name] = res
+        del llm
+        torch.cuda.empty_cache()
+    out["clocks"] = sampler.stop(t_wall0, datetime.datetime.now(), 0.0)
+    out["gpu_launches"] = _lib.launches - launches0
+    if args.verbose:
+        for name, res in out["models"].items():
+            for r in res["prefill"] + res["decode"]:
+                print(name, {k: v for k, v in r.items() if k != "kernels"}, file=sys.stderr)
+                for k, v in list(r["kernels"].items())[:14]:
+                    print(f"    {k:44s} {v['launches']:4d} x {v['us']:8.1f} us  roofline {v['roofline_us']:8.1f}  {v['frac']:.3f}", file=sys.stderr)
+    return out
+
+
 def dt_name() -> str:
     import torch
 
@@ -719,6 +936,9 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--config", default="c2", choices=sorted(CONFIGS))
+    ap.add_argument("--design", default=None, choices=["dilavik"],
+                    help="instead of the workload: prefill and decode throughput of this base model beside Llama at equal size (one GPU)")
+    ap.add_argument("--size", default="4k", choices=sorted(DESIGN_SIZES), help="layer width with --design")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--sample", action="store_true", help="reference arm: bounded sample (prefill + 2 decode steps, no port cross-check)")
     ap.add_argument("--value-only", action="store_true", help="skip the roofline, end-to-end and CPU passes (profiler runs)")
@@ -726,6 +946,10 @@ def main():
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
+    if args.design:
+        if rank == 0:
+            print(json.dumps(run_design(args)), flush=True)
+        return
     if args.impl == "reference":
         if rank == 0:
             print(json.dumps(run_cpu(args, True)), flush=True)

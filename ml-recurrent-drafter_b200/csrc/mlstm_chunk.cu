@@ -30,7 +30,7 @@ constexpr int L = 128;  // tokens per chunk
 __device__ __forceinline__ bool wait_warp(uint64_t* bar, uint32_t parity) {
   return __all_sync(0xffffffffu, rd_umma::mbar_wait(bar, parity));
 }
-constexpr int kThreads = 256;
+constexpr int kThreads = 512;
 constexpr int kGateThreads = 1024;
 
 struct ChunkArgs {
@@ -239,9 +239,10 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
   rd_umma::fence_after();
   if (tid == 0) load(0);  // the barriers are initialised
   const uint32_t tmem = *tmem_slot;
-  const int quarter = warp & 3, half = warp >> 2;
-  const int v = v0 + quarter * 32 + lane;  // this thread's value column
-  const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16) + half * (DN / 2);
+  const int quarter = warp & 3, cg = warp >> 2;
+  const int v = v0 + quarter * 32 + lane, dq = d0 + cg * 32;  // this thread's value column and its 32 dims
+  const bool has_tile = cg * 32 < DN;                         // DN = 64: half of the warps
+  const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16) + cg * 32;
   bool ok = true;
 
   for (int c = 0; c < n_chunks; ++c) {
@@ -276,15 +277,13 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
       *reinterpret_cast<uint4*>(sLo + off) = lo;
     }
     // the state at the chunk's start goes to the workspace; scaled, it becomes the accumulator of this chunk's products
-#pragma unroll
-    for (int q = 0; q < DN / 64; ++q) {
+    if (has_tile) {
       float s[32];
-      const int dq = d0 + half * (DN / 2) + q * 32;
       if (c == 0) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) s[i] = (!fresh && v < a.vdim && dq + i < a.dim) ? S_g[(int64_t)(dq + i) * a.vdim + v] : 0.f;
       } else {
-        rd_umma::tmem_ld32(t_row + q * 32, s);
+        rd_umma::tmem_ld32(t_row, s);
       }
       const int64_t off = (slot * a.vpad + v) * a.dpad + dq;
 #pragma unroll
@@ -299,7 +298,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
       }
 #pragma unroll
       for (int i = 0; i < 32; ++i) s[i] *= A;
-      rd_umma::tmem_st32(t_row + q * 32, s);
+      rd_umma::tmem_st32(t_row, s);
     }
     rd_umma::fence_async_proxy();
     rd_umma::fence_before();
@@ -340,11 +339,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
   ok = __syncthreads_and(ok);
   if (ok) {
     rd_umma::fence_after();
-#pragma unroll
-    for (int q = 0; q < DN / 64; ++q) {
+    if (has_tile) {
       float s[32];
-      const int dq = d0 + half * (DN / 2) + q * 32;
-      rd_umma::tmem_ld32(t_row + q * 32, s);
+      rd_umma::tmem_ld32(t_row, s);
 #pragma unroll
       for (int i = 0; i < 32; ++i)
         if (v < a.vdim && dq + i < a.dim) S_g[(int64_t)(dq + i) * a.vdim + v] = s[i];
@@ -372,7 +369,7 @@ struct OutSmem {
   static constexpr int kQ = (DP / 64) * kBox;
   static constexpr int kRing = kOutStages * kItem > kQ ? kOutStages * kItem : kQ;  // K first, then the ring
   static constexpr int kP = 2 * kBox;
-  static constexpr int kMisc = (5 * L + DP + 4 * L) * 4 + 160;  // per-token scalars, n, barriers
+  static constexpr int kMisc = (5 * L + DP + 8 * L) * 4 + 160;  // per-token scalars, n, barriers
   static constexpr int kBytes = kQ + kRing + 2 * kP + kMisc + 1024;
 };
 
@@ -404,9 +401,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
   float* s_floor = s_e + L;
   float* s_nq = s_floor + L;
   float* s_n = s_nq + L;       // [DP]
-  float* s_rs = s_n + DP;      // [2][L]
-  float* s_ss = s_rs + 2 * L;  // [2][L]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 2 * L);  // [kOutStages] an item's products are done
+  float* s_rs = s_n + DP;      // [4][L]
+  float* s_ss = s_rs + 4 * L;  // [4][L]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ss + 4 * L);  // [kOutStages] an item's products are done
   uint64_t* full = bars + kOutStages;                           // [kOutStages] an item has landed
   uint64_t* scores_done = full + kOutStages;
   uint64_t* state_done = scores_done + 1;
@@ -452,12 +449,12 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
     }
     rd_umma::commit(scores_done);
   }
-  // n_in . q_t meanwhile: two threads per token
+  // n_in . q_t meanwhile: four threads per token
   {
-    const int t = tid >> 1, part = tid & 1;
+    const int t = tid >> 2, part = tid & 3;
     float acc = 0.f;
 #pragma unroll 2
-    for (int ch = part; ch < DP / 8; ch += 2) {
+    for (int ch = part; ch < DP / 8; ch += 4) {
       const uint4 u = *reinterpret_cast<const uint4*>(sQ + (ch >> 3) * kBox + swz<8>(t, ch & 7));
       const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(&u);
       const float4 n0 = *reinterpret_cast<const float4*>(s_n + ch * 8), n1 = *reinterpret_cast<const float4*>(s_n + ch * 8 + 4);
@@ -467,9 +464,10 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
       acc = fmaf(f2.x, n1.x, fmaf(f2.y, n1.y, fmaf(f3.x, n1.z, fmaf(f3.y, n1.w, acc))));
     }
     acc += __shfl_xor_sync(0xffffffffu, acc, 1);
+    acc += __shfl_xor_sync(0xffffffffu, acc, 2);
     if (part == 0) s_nq[t] = acc;
   }
-  const int quarter = warp & 3, half = warp >> 2;
+  const int quarter = warp & 3, cg = warp >> 2;  // cg: this warp's quarter of the TMEM columns
   const int t = quarter * 32 + lane;  // this thread's token of the chunk
   const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16);
   bool ok = wait_warp(scores_done, 0);
@@ -526,33 +524,29 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
   if (ok && tid == 0)
     for (int i = 0; i < kOutStages && i < n_items; ++i) load(i);  // K has been read: its place is the ring
   __syncwarp();
-  // P of this thread's token and half of the keys
+  // P of this thread's token and a quarter of the keys
   if (ok) {
     const float Fm = s_Fm[t];
-    float sum = 0.f;
+    const int j0 = cg * 32;
+    float sum = 0.f, s[32];
+    rd_umma::tmem_ld32(t_row + j0, s);
 #pragma unroll
-    for (int q = 0; q < 2; ++q) {
-      float s[32];
-      const int j0 = half * 64 + q * 32;
-      rd_umma::tmem_ld32(t_row + j0, s);
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        s[i] = j0 + i <= t ? s[i] * qs * __expf(Fm + s_iF[j0 + i]) : 0.f;
-        sum += s[i];
-      }
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        uint4 hi, lo;
-        split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
-        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
-        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
-        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
-        const int off = half * kBox + swz<8>(t, q * 4 + i);
-        *reinterpret_cast<uint4*>(sPh + off) = hi;
-        *reinterpret_cast<uint4*>(sPl + off) = lo;
-      }
+    for (int i = 0; i < 32; ++i) {
+      s[i] = j0 + i <= t ? s[i] * qs * __expf(Fm + s_iF[j0 + i]) : 0.f;
+      sum += s[i];
     }
-    s_rs[half * L + t] = sum;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      uint4 hi, lo;
+      split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
+      split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
+      split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
+      split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
+      const int off = (cg >> 1) * kBox + swz<8>(t, (cg & 1) * 4 + i);
+      *reinterpret_cast<uint4*>(sPh + off) = hi;
+      *reinterpret_cast<uint4*>(sPl + off) = lo;
+    }
+    s_rs[cg * L + t] = sum;
   }
   rd_umma::fence_async_proxy();
   rd_umma::fence_before();
@@ -571,7 +565,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
     rd_umma::fence_after();
     const float e = s_e[t];
     if (__all_sync(0xffffffffu, ok)) {
-      for (int q = half * (v_tiles * 2); q < (half + 1) * (v_tiles * 2); ++q) {
+      for (int q = cg * v_tiles; q < (cg + 1) * v_tiles; ++q) {
         float o[32];
         rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
@@ -594,9 +588,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
   ok = __syncthreads_and(ok);
   if (ok) {
     rd_umma::fence_after();
-    const float den = s_rs[t] + s_rs[L + t] + s_e[t] * s_nq[t];
+    const float den = (s_rs[t] + s_rs[L + t]) + (s_rs[2 * L + t] + s_rs[3 * L + t]) + s_e[t] * s_nq[t];
     const float inv = 1.0f / (fmaxf(fabsf(den), s_floor[t]) + kDenEps);
-    const int q_lo = half * (v_tiles * 2), q_hi = q_lo + v_tiles * 2;  // this thread's 32-column blocks
+    const int q_lo = cg * v_tiles, q_hi = q_lo + v_tiles;  // this warp's 32-column blocks
     float ss = 0.f;
     for (int q = q_lo; q < q_hi; ++q) {
       float o[32];
@@ -605,35 +599,53 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_outputs_kernel(const __grid
       for (int k = 0; k < 32; ++k)
         if (q * 32 + k < a.vdim) ss = fmaf(o[k] * inv, o[k] * inv, ss);
     }
-    s_ss[half * L + t] = ss;
+    s_ss[cg * L + t] = ss;
     __syncthreads();
-    const float r = inv / sqrtf((s_ss[t] + s_ss[L + t]) / (float)a.vdim + a.eps);
-    const int64_t tok = rs + t0 + t;
-    const bool live = t0 + t < n_tok;
-    const __nv_bfloat16* gp = a.proj + (live ? tok : (int64_t)rs) * a.ld + 2 * a.nh * a.dim + (a.nh + h) * a.vdim;
-    const __nv_bfloat16* wp = a.norm_w + (int64_t)h * a.vdim;
-    __nv_bfloat16* dst = a.out + (tok * a.nh + h) * a.vdim;
+    const float r = inv / sqrtf(((s_ss[t] + s_ss[L + t]) + (s_ss[2 * L + t] + s_ss[3 * L + t])) / (float)a.vdim + a.eps);
+    // Blocks of 32 tokens x 32 columns go through shared memory, so that four lanes share a token's 64 bytes in the reads of
+    // the gate and in the stores.
+    constexpr int kLd = 36;  // floats per row: 16-byte accesses without conflicts
+    float* scr = reinterpret_cast<float*>(ring) + warp * 32 * kLd;  // the ring and P are dead
+    const int sub = lane & 3, row0 = lane >> 2;
     for (int q = q_lo; q < q_hi; ++q) {
+      const int col = q * 32 + sub * 8;
+      const bool in = col < a.vdim;
+      uint4 gu[4];
+#pragma unroll
+      for (int p = 0; p < 4; ++p) {
+        const int tt = t0 + quarter * 32 + p * 8 + row0;
+        if (in && tt < n_tok)
+          gu[p] = *reinterpret_cast<const uint4*>(a.proj + (int64_t)(rs + tt) * a.ld + 2 * a.nh * a.dim + (a.nh + h) * a.vdim + col);
+      }
       float o[32];
       rd_umma::tmem_ld32(t_row + q * 32, o);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int v = q * 32 + i * 8;
-        if (live && v < a.vdim) {
-          const uint4 gu = *reinterpret_cast<const uint4*>(gp + v), wu = *reinterpret_cast<const uint4*>(wp + v);
-          const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu);
-          const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&wu);
-          uint4 pk;
-          uint32_t* pp = reinterpret_cast<uint32_t*>(&pk);
+      for (int k = 0; k < 8; ++k)
+        *reinterpret_cast<float4*>(scr + lane * kLd + 4 * k) = make_float4(o[4 * k] * r, o[4 * k + 1] * r, o[4 * k + 2] * r, o[4 * k + 3] * r);
+      __syncwarp();
+      if (in) {
+        const uint4 wu = *reinterpret_cast<const uint4*>(a.norm_w + (int64_t)h * a.vdim + col);
+        const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&wu);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float2 gg = __bfloat1622float2(g2[e]), ww = __bfloat1622float2(w2[e]);
-            pp[e] = pack_bf16(__fdividef(o[8 * i + 2 * e] * r * ww.x, 1.f + __expf(-gg.x)),
-                              __fdividef(o[8 * i + 2 * e + 1] * r * ww.y, 1.f + __expf(-gg.y)));
+        for (int p = 0; p < 4; ++p) {
+          const int tt = t0 + quarter * 32 + p * 8 + row0;
+          if (tt < n_tok) {
+            float y[8];
+            *reinterpret_cast<float4*>(y) = *reinterpret_cast<const float4*>(scr + (p * 8 + row0) * kLd + sub * 8);
+            *reinterpret_cast<float4*>(y + 4) = *reinterpret_cast<const float4*>(scr + (p * 8 + row0) * kLd + sub * 8 + 4);
+            const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gu[p]);
+            uint4 pk;
+            uint32_t* pp = reinterpret_cast<uint32_t*>(&pk);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 gg = __bfloat1622float2(g2[e]), ww = __bfloat1622float2(w2[e]);
+              pp[e] = pack_bf16(__fdividef(y[2 * e] * ww.x, 1.f + __expf(-gg.x)), __fdividef(y[2 * e + 1] * ww.y, 1.f + __expf(-gg.y)));
+            }
+            *reinterpret_cast<uint4*>(a.out + ((int64_t)(rs + tt) * a.nh + h) * a.vdim + col) = pk;
           }
-          *reinterpret_cast<uint4*>(dst + v) = pk;
         }
       }
+      __syncwarp();  // the scratch is reused by the next block
     }
   } else if (tid == 0) {
     if (a.status) atomicExch(a.status, 32);
