@@ -184,6 +184,8 @@ struct StateSmem {
   static constexpr int kBytes = 2 * kStage + 2 * kV + kMisc + 1024;  // two stages, w V hi and lo, alignment
 };
 
+constexpr int kScr = 80;  // bytes per row of the transposition scratch: 64 and a shift of the banks
+
 // grid (value tiles of 128 * dim tiles of DN, nh, B).  S^T tile [128 value columns = TMEM lanes][DN dims = TMEM columns].
 // Per chunk: the tile is read out, written to the workspace, scaled and put back, then (w V)^T K is added by tcgen05.mma
 // (both operands MN-major: value columns and dims contiguous, tokens along K).
@@ -257,6 +259,44 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
     const uint8_t* sV = sK + Y::kK;
     const float* w = s_w + (c & 1) * L;
     const int64_t slot = (int64_t)chunk_slot(rs, b, c) * a.nh + h;
+    // the state at the chunk's start goes to the workspace; scaled, it becomes the accumulator of this chunk's products
+    if (has_tile) {
+      float s[32];
+      if (c == 0) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) s[i] = (!fresh && v < a.vdim && dq + i < a.dim) ? S_g[(int64_t)(dq + i) * a.vdim + v] : 0.f;
+      } else {
+        rd_umma::tmem_ld32(t_row, s);
+      }
+      // through this warp's scratch (in the operand buffers of the chunk before), so that four lanes write a row's 64 bytes
+      uint8_t* scr = sHi + warp * (32 * kScr);
+      uint4 lo[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        uint4 hi;
+        split2(s[8 * i], s[8 * i + 1], hi.x, lo[i].x);
+        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo[i].y);
+        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo[i].z);
+        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo[i].w);
+        *reinterpret_cast<uint4*>(scr + lane * kScr + i * 16) = hi;
+      }
+      __syncwarp();
+      const int64_t off = (slot * a.vpad + v0 + quarter * 32 + (lane >> 2)) * a.dpad + dq + (lane & 3) * 8;
+#pragma unroll
+      for (int p = 0; p < 4; ++p)
+        *reinterpret_cast<uint4*>(a.Shi + off + (int64_t)p * 8 * a.dpad) = *reinterpret_cast<const uint4*>(scr + (p * 8 + (lane >> 2)) * kScr + (lane & 3) * 16);
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4*>(scr + lane * kScr + i * 16) = lo[i];
+      __syncwarp();
+#pragma unroll
+      for (int p = 0; p < 4; ++p)
+        *reinterpret_cast<uint4*>(a.Slo + off + (int64_t)p * 8 * a.dpad) = *reinterpret_cast<const uint4*>(scr + (p * 8 + (lane >> 2)) * kScr + (lane & 3) * 16);
+#pragma unroll
+      for (int i = 0; i < 32; ++i) s[i] *= A;
+      rd_umma::tmem_st32(t_row, s);
+    }
+    __syncthreads();  // the scratch becomes operand space again
     // w_j v_j as hi + lo, in the same swizzled boxes
 #pragma unroll 4
     for (int i = tid; i < L * 16; i += kThreads) {
@@ -275,30 +315,6 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
       }
       *reinterpret_cast<uint4*>(sHi + off) = hi;
       *reinterpret_cast<uint4*>(sLo + off) = lo;
-    }
-    // the state at the chunk's start goes to the workspace; scaled, it becomes the accumulator of this chunk's products
-    if (has_tile) {
-      float s[32];
-      if (c == 0) {
-#pragma unroll
-        for (int i = 0; i < 32; ++i) s[i] = (!fresh && v < a.vdim && dq + i < a.dim) ? S_g[(int64_t)(dq + i) * a.vdim + v] : 0.f;
-      } else {
-        rd_umma::tmem_ld32(t_row, s);
-      }
-      const int64_t off = (slot * a.vpad + v) * a.dpad + dq;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        uint4 hi, lo;
-        split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
-        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
-        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
-        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
-        *reinterpret_cast<uint4*>(a.Shi + off + 8 * i) = hi;
-        *reinterpret_cast<uint4*>(a.Slo + off + 8 * i) = lo;
-      }
-#pragma unroll
-      for (int i = 0; i < 32; ++i) s[i] *= A;
-      rd_umma::tmem_st32(t_row, s);
     }
     rd_umma::fence_async_proxy();
     rd_umma::fence_before();

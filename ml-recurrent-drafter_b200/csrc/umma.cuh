@@ -22,18 +22,14 @@ __device__ __forceinline__ bool mbar_try(uint64_t* bar, uint32_t parity) {
       : "memory");
   return ok != 0;
 }
-__device__ __forceinline__ uint64_t global_ns() {
-  uint64_t t;
-  asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
-  return t;
-}
-// Bounded wait (one second).  Returns false when it gave up.
+// Bounded wait (2^31 SM cycles, about a second).  Returns false when it gave up.  The cycle counter is read here because
+// reading the global timer costs more than many of these waits last.
 __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity) {
   if (mbar_try(bar, parity)) return true;
-  const uint64_t t0 = global_ns();
+  const long long t0 = clock64();
   for (;;) {
     if (mbar_try(bar, parity)) return true;
-    if (global_ns() - t0 > 1000000000ull) return false;
+    if (clock64() - t0 > (1ll << 31)) return false;
   }
 }
 __device__ __forceinline__ void mbar_expect_tx(uint64_t* bar, uint32_t bytes) {
