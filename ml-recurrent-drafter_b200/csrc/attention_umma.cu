@@ -194,11 +194,11 @@ struct WindowArgs {
 template <bool WIN>
 __global__ void __launch_bounds__(kThreads, 2)
     attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                          const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
-                          const int32_t* __restrict__ row_start, const int32_t* __restrict__ kv_begin,
-                          const int32_t* __restrict__ base_len, int nh, int nkv, int max_len, int mode,
-                          const uint32_t* __restrict__ tree_mask, int mask_words, float scale_log2, int32_t* status,
-                          int n_split, float* __restrict__ partial, const WindowArgs win) {
+                          const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* out,
+                          const int32_t* row_start, const int32_t* kv_begin,
+                          const int32_t* base_len, int nh, int nkv, int max_len, int mode,
+                          const uint32_t* tree_mask, int mask_words, float scale_log2, int32_t* status,
+                          int n_split, float* partial, const WindowArgs win) {
   const int b = blockIdx.z, h = blockIdx.y;
   rd::pdl_launch_dependents();
   if (threadIdx.x == 0) {
@@ -578,8 +578,8 @@ __global__ void __launch_bounds__(kThreads, 2)
 }
 
 // Merge of the shares of a split launch: out = sum_s O_s 2^(m_s - m) / sum_s l_s 2^(m_s - m).
-__global__ void __launch_bounds__(HD) attention_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out,
-                                                             const int32_t* __restrict__ row_start, int B, int nh, int n_split) {
+__global__ void __launch_bounds__(HD) attention_merge_kernel(const float* partial, __nv_bfloat16* out,
+                                                             const int32_t* row_start, int B, int nh, int n_split) {
   const int tok = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
   if (tok >= row_start[B]) return;
   const float* p = partial + ((int64_t)tok * nh + h) * n_split * (HD + 2);

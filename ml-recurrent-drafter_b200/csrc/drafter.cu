@@ -8,9 +8,9 @@ namespace {
 // ---------------------------------------------------------------------------------------------
 // rd_drafter_prepare
 template <typename T>
-__global__ void drafter_prepare_kernel(const T* __restrict__ embed, const int64_t* __restrict__ beams,
-                                       const int32_t* __restrict__ parent, const T* __restrict__ ctx, T* __restrict__ a,
-                                       T* __restrict__ x, int W, int Lb, int H, int k, int vec, int additive) {
+__global__ void drafter_prepare_kernel(const T* embed, const int64_t* beams,
+                                       const int32_t* parent, const T* ctx, T* a,
+                                       T* x, int W, int Lb, int H, int k, int vec, int additive) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int r = blockIdx.x;
@@ -226,10 +226,10 @@ __device__ void topk_radix_path(const RowReader<T>& row, TopkShared& sh, int top
 
 template <typename T>
 __global__ void __launch_bounds__(kTopkThreads) vocab_topk_kernel(
-    const T* __restrict__ logits, int64_t ld, int rows_max, const int32_t* __restrict__ rows_dev, int V, int top_k,
-    float mask_value, int subtract_max, float temperature, int vec_ok, const float* __restrict__ slice_max, int64_t slice_ld,
-    float* __restrict__ kept_val, int32_t* __restrict__ kept_idx, int32_t* __restrict__ kept_cnt,
-    float* __restrict__ masked_logp) {
+    const T* logits, int64_t ld, int rows_max, const int32_t* rows_dev, int V, int top_k,
+    float mask_value, int subtract_max, float temperature, int vec_ok, const float* slice_max, int64_t slice_ld,
+    float* kept_val, int32_t* kept_idx, int32_t* kept_cnt,
+    float* masked_logp) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int row_id = blockIdx.x;
@@ -403,10 +403,10 @@ constexpr int kSelThreads = 256;
 constexpr int kSelSplit = 8;  // CTAs per batch row: each ranks its share of the candidates against all lists
 
 __global__ void __launch_bounds__(kSelThreads) beam_select_kernel(
-    int W, int Lb, int k, int V, const float* __restrict__ kept_val, const int32_t* __restrict__ kept_idx,
-    const int32_t* __restrict__ kept_cnt, const float* __restrict__ score_in, float* __restrict__ score_out,
-    const int64_t* __restrict__ beams_in, int64_t* __restrict__ beams_out, const int32_t* __restrict__ anc_in,
-    int32_t* __restrict__ anc_out, int32_t* __restrict__ parent_out) {
+    int W, int Lb, int k, int V, const float* kept_val, const int32_t* kept_idx,
+    const int32_t* kept_cnt, const float* score_in, float* score_out,
+    const int64_t* beams_in, int64_t* beams_out, const int32_t* anc_in,
+    int32_t* anc_out, int32_t* parent_out) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int b = blockIdx.x;
@@ -485,8 +485,8 @@ struct SparseLists {
   const float* masked[RD_MAX_BEAM_LENGTH];
 };
 
-__global__ void dense_log_probs_kernel(int W, int Lb, int V, SparseLists s, const int32_t* __restrict__ anc,
-                                       float* __restrict__ out) {
+__global__ void dense_log_probs_kernel(int W, int Lb, int V, SparseLists s, const int32_t* anc,
+                                       float* out) {
   // block = (b*W + w)*(Lb-1) + j
   const int j = blockIdx.x % (Lb - 1);
   const int bw = blockIdx.x / (Lb - 1);
@@ -502,9 +502,9 @@ __global__ void dense_log_probs_kernel(int W, int Lb, int V, SparseLists s, cons
 
 // ---------------------------------------------------------------------------------------------
 // rd_sample_from_sparse: one warp per row.
-__global__ void sample_sparse_kernel(const float* __restrict__ kept_val, const int32_t* __restrict__ kept_idx,
-                                     const int32_t* __restrict__ kept_cnt, int rows, const float* __restrict__ uniforms,
-                                     int64_t* __restrict__ out) {
+__global__ void sample_sparse_kernel(const float* kept_val, const int32_t* kept_idx,
+                                     const int32_t* kept_cnt, int rows, const float* uniforms,
+                                     int64_t* out) {
   const int row = blockIdx.x;
   __shared__ float p[kKept];
   __shared__ int id[kKept];

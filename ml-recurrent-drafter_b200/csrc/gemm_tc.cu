@@ -754,7 +754,7 @@ struct SmemLayout {
 template <int EPI, bool OUT_F32>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, EpiArgs epi,
-                   int m_max, const int32_t* __restrict__ m_dev, int N, int K, int32_t* status) {
+                   int m_max, const int32_t* m_dev, int N, int K, int32_t* status) {
   using L = SmemLayout;
   constexpr int kStages = L::kStages;
   extern __shared__ uint8_t smem_raw[];
@@ -1060,7 +1060,7 @@ struct SmemLayoutPair {
 template <int EPI, bool OUT_F32>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tc_pair_kernel(const __grid_constant__ TokMaps maps_a, const __grid_constant__ CUtensorMap map_w, EpiArgs epi,
-                        int m_max, const int32_t* __restrict__ m_dev, int N, int K, int32_t* status) {
+                        int m_max, const int32_t* m_dev, int N, int K, int32_t* status) {
   using L = SmemLayoutPair;
   constexpr int kStages = L::kStages;
   extern __shared__ uint8_t smem_raw[];
@@ -1317,10 +1317,10 @@ __global__ void __launch_bounds__(kThreads, 1)
 // (logit descending, id ascending), so the merge is a plain maximum.  A block serves 8 tokens with 32
 // groups of threads walking the slices (each 32-byte sector of the [slice][token] array is read once).
 constexpr int kMergeTok = 8, kMergeGroups = 32;
-__global__ void __launch_bounds__(kMergeTok* kMergeGroups) argmax_merge_kernel(const unsigned long long* __restrict__ part_key, int64_t ld,
+__global__ void __launch_bounds__(kMergeTok* kMergeGroups) argmax_merge_kernel(const unsigned long long* part_key, int64_t ld,
                                                                               int n_slices, int m_max,
-                                                                              const int32_t* __restrict__ m_dev,
-                                                                              int32_t* __restrict__ out32, int64_t* __restrict__ out64) {
+                                                                              const int32_t* m_dev,
+                                                                              int32_t* out32, int64_t* out64) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int M = rd::live_rows(m_dev, m_max);

@@ -6,8 +6,8 @@
 namespace {
 
 template <typename T>
-__global__ void embed_gather_kernel(const T* __restrict__ table, const int64_t* __restrict__ ids, T* __restrict__ out,
-                                    int m_max, const int32_t* __restrict__ m_dev, int H, int vec) {
+__global__ void embed_gather_kernel(const T* table, const int64_t* ids, T* out,
+                                    int m_max, const int32_t* m_dev, int H, int vec) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int t = blockIdx.x;
@@ -23,8 +23,8 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int64_t* 
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) rmsnorm_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ y,
-                                                      int m_max, const int32_t* __restrict__ m_dev, int H, float eps,
+__global__ void __launch_bounds__(256) rmsnorm_kernel(const T* x, const T* w, T* y,
+                                                      int m_max, const int32_t* m_dev, int H, float eps,
                                                       int vectorised) {
   constexpr int VEC = 16 / sizeof(T);
   const int t = blockIdx.x;
@@ -85,10 +85,10 @@ constexpr int kRopeThreads = 512;
 
 template <typename T>
 __global__ void __launch_bounds__(kRopeThreads) rope_kv_write_kernel(
-    const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
-    const int32_t* __restrict__ tok_row, const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ tok_slot,
-    const float* __restrict__ cos_t, const float* __restrict__ sin_t, int n_pos, int m_max,
-    const int32_t* __restrict__ m_dev, int nh, int nkv, int hd, int max_len) {
+    const T* qkv, T* q_out, T* k_cache, T* v_cache,
+    const int32_t* tok_row, const int32_t* tok_pos, const int32_t* tok_slot,
+    const float* cos_t, const float* sin_t, int n_pos, int m_max,
+    const int32_t* m_dev, int nh, int nkv, int hd, int max_len) {
   constexpr int VEC = 16 / sizeof(T);
   const int t = blockIdx.x;
   rd::pdl_launch_dependents();
@@ -152,9 +152,9 @@ __global__ void __launch_bounds__(kRopeThreads) rope_kv_write_kernel(
   }
 }
 
-__global__ void __launch_bounds__(256) argmax_rows_kernel(const float* __restrict__ logits, int64_t ld, int m_max,
-                                                          const int32_t* __restrict__ m_dev, int V,
-                                                          int32_t* __restrict__ out32, int64_t* __restrict__ out64) {
+__global__ void __launch_bounds__(256) argmax_rows_kernel(const float* logits, int64_t ld, int m_max,
+                                                          const int32_t* m_dev, int V,
+                                                          int32_t* out32, int64_t* out64) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int t = blockIdx.x;
@@ -197,9 +197,9 @@ __global__ void __launch_bounds__(256) argmax_rows_kernel(const float* __restric
   }
 }
 
-__global__ void emit_tokens_kernel(const int64_t* __restrict__ token_buf, int max_len, const int32_t* __restrict__ kv_begin,
-                                   const int32_t* __restrict__ kv_len, const int64_t* __restrict__ next_tokens,
-                                   int64_t pad_id, int out_len, int64_t* __restrict__ out) {
+__global__ void emit_tokens_kernel(const int64_t* token_buf, int max_len, const int32_t* kv_begin,
+                                   const int32_t* kv_len, const int64_t* next_tokens,
+                                   int64_t pad_id, int out_len, int64_t* out) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int b = blockIdx.x;
@@ -217,10 +217,10 @@ __global__ void emit_tokens_kernel(const int64_t* __restrict__ token_buf, int ma
   }
 }
 
-__global__ void commit_reference_slots_kernel(int W, int Lb, const int32_t* __restrict__ unpacker,
-                                              const int32_t* __restrict__ n_accepted,
-                                              const int32_t* __restrict__ seq_in_beam, int S, int S2,
-                                              int64_t* __restrict__ out) {
+__global__ void commit_reference_slots_kernel(int W, int Lb, const int32_t* unpacker,
+                                              const int32_t* n_accepted,
+                                              const int32_t* seq_in_beam, int S, int S2,
+                                              int64_t* out) {
   const int b = blockIdx.x, j = threadIdx.x;
   if (j >= Lb) return;
   const int A = n_accepted[b], seq = seq_in_beam[b];
@@ -236,8 +236,8 @@ __global__ void commit_reference_slots_kernel(int W, int Lb, const int32_t* __re
 
 // Cache.unpack of the reference layout: gather into scratch, then write back.
 template <typename T>
-__global__ void cache_unpack_gather_kernel(const T* __restrict__ cache, int B, int nkv, int max_len, int hd, int S,
-                                           const int64_t* __restrict__ unpacker, int n_flat, T* __restrict__ scratch) {
+__global__ void cache_unpack_gather_kernel(const T* cache, int B, int nkv, int max_len, int hd, int S,
+                                           const int64_t* unpacker, int n_flat, T* scratch) {
   // grid (n_flat, B*nkv, NL*2)
   const int f = blockIdx.x, bh = blockIdx.y, lk = blockIdx.z;
   const int b = bh / nkv;
@@ -247,8 +247,8 @@ __global__ void cache_unpack_gather_kernel(const T* __restrict__ cache, int B, i
   for (int d = threadIdx.x; d < hd; d += blockDim.x) dst[d] = src[d];
 }
 template <typename T>
-__global__ void cache_unpack_scatter_kernel(T* __restrict__ cache, int B, int nkv, int max_len, int hd, int S, int n_flat,
-                                            const T* __restrict__ scratch) {
+__global__ void cache_unpack_scatter_kernel(T* cache, int B, int nkv, int max_len, int hd, int S, int n_flat,
+                                            const T* scratch) {
   const int f = blockIdx.x, bh = blockIdx.y, lk = blockIdx.z;
   const T* src = scratch + (((int64_t)lk * B * nkv + bh) * n_flat + f) * hd;
   T* dst = cache + (((int64_t)lk * B * nkv + bh) * max_len + S + f) * hd;
