@@ -60,13 +60,16 @@ __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.0f + _
 // expf with full fp32 accuracy (used where parity with a CPU fp32 path matters)
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
 
-// xIELU: pos z^2 + z/2 above zero, neg (e^z - 1 - z) + z/2 elsewhere
+// xIELU: pos z^2 + z/2 above zero, neg (e^z - 1 - z) + z/2 elsewhere.  Each part vanishes on the other's side, so neither
+// needs a branch.
 __device__ __forceinline__ float xielu_exact(float z, float pos, float neg) {
-  return (z > 0.f ? pos * z * z : neg * (expm1f(z) - z)) + 0.5f * z;
+  const float p = fmaxf(z, 0.f), m = fminf(z, 0.f);
+  return fmaf(pos * p, p, neg * (expm1f(m) - m)) + 0.5f * z;
 }
 // form for rounded (bf16) outputs: e^z - 1 carries an absolute error of about 1e-7 near zero
 __device__ __forceinline__ float xielu_f(float z, float pos, float neg) {
-  return (z > 0.f ? pos * z * z : neg * (__expf(fminf(z, 0.f)) - 1.0f - z)) + 0.5f * z;
+  const float p = fmaxf(z, 0.f), m = fminf(z, 0.f);
+  return fmaf(pos * p, p, fmaf(neg, __expf(m) - 1.0f - m, 0.5f * z));
 }
 
 __device__ __forceinline__ float warp_max(float v) {
