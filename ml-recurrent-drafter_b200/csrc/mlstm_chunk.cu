@@ -9,7 +9,7 @@
 //   S_out = e^(F_L + m_in - m_L) S_in + sum_j e^(F_L - F_j + i_j - m_L) k_j v_j^T      (n likewise with k alone)
 // so every exponent is <= 0, and the result is the token-by-token recurrence up to rounding.  Three kernels:
 //   gates    one CTA per (head, row): the scalars above for every token; only the chunks' maxima follow one another
-//   states   one CTA per 128 value columns x 128 dims of S: walks the chunks, the tile in TMEM (fp32), and leaves S and n
+//   states   one CTA per 128 value columns x 64 dims of S: walks the chunks, the tile in TMEM (fp32), and leaves S and n
 //            at the start of every chunk in the workspace
 //   outputs  one CTA per chunk of a head: scores, both products (accumulated in TMEM), the head's RMS norm, the norm
 //            weight and the output gate, independent of all other chunks
@@ -176,22 +176,22 @@ __global__ void __launch_bounds__(kGateThreads) mlstm_gates_kernel(const ChunkAr
 // Rows of a [128 x 64] box are 128 bytes, 16-byte chunks permuted by the row: the tensor core's 128-byte swizzle.
 constexpr int kBox = 128 * 128;  // bytes
 
-template <int DN>
+constexpr int DN = 64;  // dims per CTA of the states kernel
+
 struct StateSmem {
-  static constexpr int kK = (DN / 64) * kBox, kV = 2 * kBox;  // [128 tokens] x DN dims, x 128 value columns
+  static constexpr int kK = kBox, kV = 2 * kBox;  // [128 tokens] x 64 dims, x 128 value columns
   static constexpr int kStage = kK + kV;
   static constexpr int kMisc = (2 * L + DN + 8) * 4 + 64;  // w, n, barriers
-  static constexpr int kBytes = 2 * kStage + 2 * kV + kMisc + 1024;  // two stages, w V hi and lo, alignment
+  static constexpr int kBytes = 2 * kStage + 2 * kV + 2 * kBox + kMisc + 1024;  // two stages, w V and S^T as hi and lo, alignment
 };
 
-constexpr int kScr = 80;  // bytes per row of the transposition scratch: 64 and a shift of the banks
-
 // grid (value tiles of 128 * dim tiles of DN, nh, B).  S^T tile [128 value columns = TMEM lanes][DN dims = TMEM columns].
-// Per chunk: the tile is read out, written to the workspace, scaled and put back, then (w V)^T K is added by tcgen05.mma
+// Per chunk: the tile is read out, stored to the workspace (TMA), scaled and put back, then (w V)^T K is added by tcgen05.mma
 // (both operands MN-major: value columns and dims contiguous, tokens along K).
-template <int DN>
-__global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_constant__ CUtensorMap map_proj, const ChunkArgs a) {
-  using Y = StateSmem<DN>;
+__global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_constant__ CUtensorMap map_proj,
+                                                                   const __grid_constant__ CUtensorMap map_hi,
+                                                                   const __grid_constant__ CUtensorMap map_lo, const ChunkArgs a) {
+  using Y = StateSmem;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   rd::pdl_launch_dependents();
@@ -205,7 +205,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   uint8_t* sHi = smem + 2 * Y::kStage;
   uint8_t* sLo = sHi + Y::kV;
-  float* s_w = reinterpret_cast<float*>(sLo + Y::kV);  // [2][L]
+  uint8_t* sShi = sLo + Y::kV;  // the tile on its way to the workspace
+  uint8_t* sSlo = sShi + kBox;
+  float* s_w = reinterpret_cast<float*>(sSlo + kBox);  // [2][L]
   float* s_n = s_w + 2 * L;                             // [DN]
   uint64_t* bar = reinterpret_cast<uint64_t*>(s_n + DN);  // a chunk's products are done
   uint64_t* full = bar + 1;                               // [2] a stage's K and V have landed
@@ -227,8 +229,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
     uint8_t* sK = smem + (c & 1) * Y::kStage;
     rd_umma::mbar_expect_tx(&full[c & 1], Y::kStage);
     const int row = rs + c * L, k0 = (a.nh + h) * a.dim + d0, w0 = 2 * a.nh * a.dim + h * a.vdim + v0;
-#pragma unroll
-    for (int i = 0; i < DN / 64; ++i) rd_umma::tma_load_2d(sK + i * kBox, &map_proj, &full[c & 1], k0 + i * 64, row);
+    rd_umma::tma_load_2d(sK, &map_proj, &full[c & 1], k0, row);
 #pragma unroll
     for (int i = 0; i < 2; ++i) rd_umma::tma_load_2d(sK + Y::kK + i * kBox, &map_proj, &full[c & 1], w0 + i * 64, row);
   };
@@ -243,13 +244,14 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
   const uint32_t tmem = *tmem_slot;
   const int quarter = warp & 3, cg = warp >> 2;
   const int v = v0 + quarter * 32 + lane, dq = d0 + cg * 32;  // this thread's value column and its 32 dims
-  const bool has_tile = cg * 32 < DN;                         // DN = 64: half of the warps
+  const bool has_tile = cg * 32 < DN;                         // half of the warps
   const uint32_t t_row = tmem + ((uint32_t)(quarter * 32) << 16) + cg * 32;
   bool ok = true;
 
   for (int c = 0; c < n_chunks; ++c) {
     // the products of chunk c - 1 are in the tile, and its operands' shared memory is free
     if (c > 0) ok = wait_warp(bar, (c - 1) & 1);
+    if (tid == 0) rd_umma::tma_store_wait_read();
     if (!__syncthreads_and(ok)) break;
     if (tid == 0 && c + 1 < n_chunks) load(c + 1);
     ok = wait_warp(&full[c & 1], (c >> 1) & 1);
@@ -268,35 +270,21 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
       } else {
         rd_umma::tmem_ld32(t_row, s);
       }
-      // through this warp's scratch (in the operand buffers of the chunk before), so that four lanes write a row's 64 bytes
-      uint8_t* scr = sHi + warp * (32 * kScr);
-      uint4 lo[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        uint4 hi;
-        split2(s[8 * i], s[8 * i + 1], hi.x, lo[i].x);
-        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo[i].y);
-        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo[i].z);
-        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo[i].w);
-        *reinterpret_cast<uint4*>(scr + lane * kScr + i * 16) = hi;
+        uint4 hi, lo;
+        split2(s[8 * i], s[8 * i + 1], hi.x, lo.x);
+        split2(s[8 * i + 2], s[8 * i + 3], hi.y, lo.y);
+        split2(s[8 * i + 4], s[8 * i + 5], hi.z, lo.z);
+        split2(s[8 * i + 6], s[8 * i + 7], hi.w, lo.w);
+        const int off = swz<8>(quarter * 32 + lane, cg * 4 + i);
+        *reinterpret_cast<uint4*>(sShi + off) = hi;
+        *reinterpret_cast<uint4*>(sSlo + off) = lo;
       }
-      __syncwarp();
-      const int64_t off = (slot * a.vpad + v0 + quarter * 32 + (lane >> 2)) * a.dpad + dq + (lane & 3) * 8;
-#pragma unroll
-      for (int p = 0; p < 4; ++p)
-        *reinterpret_cast<uint4*>(a.Shi + off + (int64_t)p * 8 * a.dpad) = *reinterpret_cast<const uint4*>(scr + (p * 8 + (lane >> 2)) * kScr + (lane & 3) * 16);
-      __syncwarp();
-#pragma unroll
-      for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4*>(scr + lane * kScr + i * 16) = lo[i];
-      __syncwarp();
-#pragma unroll
-      for (int p = 0; p < 4; ++p)
-        *reinterpret_cast<uint4*>(a.Slo + off + (int64_t)p * 8 * a.dpad) = *reinterpret_cast<const uint4*>(scr + (p * 8 + (lane >> 2)) * kScr + (lane & 3) * 16);
 #pragma unroll
       for (int i = 0; i < 32; ++i) s[i] *= A;
       rd_umma::tmem_st32(t_row, s);
     }
-    __syncthreads();  // the scratch becomes operand space again
     // w_j v_j as hi + lo, in the same swizzled boxes
 #pragma unroll 4
     for (int i = tid; i < L * 16; i += kThreads) {
@@ -332,6 +320,9 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
         rd_umma::mma_ss(tmem, rd_umma::desc_mn_major(rd_umma::smem_u32(sLo + k * 2048), kBox), dk, idesc, 1);
       }
       rd_umma::commit(bar);
+      rd_umma::tma_store_2d(&map_hi, sShi, d0, (int)(slot * a.vpad) + v0);
+      rd_umma::tma_store_2d(&map_lo, sSlo, d0, (int)(slot * a.vpad) + v0);
+      rd_umma::tma_store_commit();
     }
     if (owns_n) {
       // n of this tile's dims: kThreads / DN threads per dim
@@ -340,7 +331,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
       float sum = 0.f;
 #pragma unroll 8
       for (int j = part; j < L; j += PER)
-        sum = fmaf(w[j], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sK + (d >> 6) * kBox + swz<8>(j, (d & 63) >> 3) + (d & 7) * 2)), sum);
+        sum = fmaf(w[j], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sK + swz<8>(j, d >> 3) + (d & 7) * 2)), sum);
 #pragma unroll
       for (int o = 1; o < PER; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       if (part == 0) {
@@ -351,6 +342,7 @@ __global__ void __launch_bounds__(kThreads, 1) mlstm_states_kernel(const __grid_
     if (tid < L) s_w[((c + 1) & 1) * L + tid] = w_next;
     A = A_next;
   }
+  if (tid == 0) rd_umma::tma_store_wait();
   if (ok) ok = wait_warp(bar, (n_chunks - 1) & 1);
   ok = __syncthreads_and(ok);
   if (ok) {
@@ -690,10 +682,9 @@ int launch_big(Kern kern, bool& set, dim3 grid, int smem, cudaStream_t s, const 
 struct Maps {
   CUtensorMap proj, v, hi, lo;  // proj in boxes of 128 and of 64 rows; the two halves of S^T
 };
-template <int DN>
-int launch_states(const Maps& m, const ChunkArgs& a, int B, cudaStream_t s) {
+inline int launch_states(const Maps& m, const ChunkArgs& a, int B, cudaStream_t s) {
   static bool set = false;
-  return launch_big(mlstm_states_kernel<DN>, set, dim3((a.vpad / 128) * (a.dpad / DN), a.nh, B), StateSmem<DN>::kBytes, s, m.proj, a);
+  return launch_big(mlstm_states_kernel, set, dim3((a.vpad / 128) * (a.dpad / DN), a.nh, B), StateSmem::kBytes, s, m.proj, m.hi, m.lo, a);
 }
 template <int DP>
 int launch_outputs(const Maps& m, const ChunkArgs& a, int B, int max_new, cudaStream_t s) {
@@ -701,7 +692,7 @@ int launch_outputs(const Maps& m, const ChunkArgs& a, int B, int max_new, cudaSt
   return launch_big(mlstm_outputs_kernel<DP>, set, dim3((max_new + L - 1) / L, a.nh, B), OutSmem<DP>::kBytes, s, m.v, m.hi, m.lo, a);
 }
 
-inline int64_t pad_dim(int64_t n) { return n <= 64 ? 64 : (n + 127) / 128 * 128; }
+inline int64_t pad_dim(int64_t n) { return (n + DN - 1) / DN * DN; }
 inline int64_t pad_v(int64_t n) { return (n + 127) / 128 * 128; }
 inline int64_t slots_of(int64_t m_max, int64_t B) { return m_max / L + B; }
 
@@ -768,7 +759,7 @@ extern "C" int rd_mlstm_chunk(const void* proj, int64_t ld, const float* gates, 
   if (!rd_umma::make_map(&maps.proj, proj, m_max, width, ld, 128) || !rd_umma::make_map(&maps.v, proj, m_max, width, ld, 64) ||
       !rd_umma::make_map(&maps.hi, a.Shi, s_rows, a.dpad, a.dpad, 128) || !rd_umma::make_map(&maps.lo, a.Slo, s_rows, a.dpad, a.dpad, 128))
     return RD_ERR_ARG;
-  int rc = dim <= 64 ? launch_states<64>(maps, a, B, s) : launch_states<128>(maps, a, B, s);
+  int rc = launch_states(maps, a, B, s);
   if (rc != RD_OK) return rc;
   if (dim <= 64) return launch_outputs<64>(maps, a, B, max_new, s);
   if (dim <= 128) return launch_outputs<128>(maps, a, B, max_new, s);
