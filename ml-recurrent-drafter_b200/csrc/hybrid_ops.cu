@@ -85,21 +85,28 @@ __global__ void __launch_bounds__(kNormMaxThreads) stream_norm_kernel(
     if (lane == 0) part_sum[u] = ss;
   }
   __syncthreads();
+  // one scale per group, left in the place of its first share
+  for (int g = tid; g < groups; g += n_thr) {
+    float tot = 0.f;
+    for (int p = 0; p < parts; ++p) tot += part_sum[g * parts + p];
+    part_sum[g * parts] = 1.0f / sqrtf(tot / (float)gsize + eps);
+  }
+  __syncthreads();
   T* dst = y + (int64_t)t * H;
+  const bool whole = gsize % VEC == 0;  // a vector lies in one group
   for (int d = tid * VEC; d < H; d += n_thr * VEC) {
-    T o[VEC];
-    int g = -1;
-    float rs = 0.f;
+    T o[VEC], g[VEC];
+    if constexpr (VEC == 4 && sizeof(T) == 2)
+      *reinterpret_cast<uint2*>(g) = *reinterpret_cast<const uint2*>(w + d);
+    else if constexpr (VEC == 4)
+      *reinterpret_cast<float4*>(g) = *reinterpret_cast<const float4*>(w + d);
+    else
+      g[0] = w[d];
+    float rs = part_sum[(d / gsize) * parts];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
-      const int ge = (d + e) / gsize;
-      if (ge != g) {
-        g = ge;
-        float tot = 0.f;
-        for (int p = 0; p < parts; ++p) tot += part_sum[g * parts + p];
-        rs = 1.0f / sqrtf(tot / (float)gsize + eps);
-      }
-      o[e] = rd::Num<T>::from_f(row[d + e] * rs * rd::Num<T>::to_f(w[d + e]));
+      if (!whole) rs = part_sum[((d + e) / gsize) * parts];
+      o[e] = rd::Num<T>::from_f(row[d + e] * rs * rd::Num<T>::to_f(g[e]));
     }
     if constexpr (VEC == 4 && sizeof(T) == 2)
       *reinterpret_cast<uint2*>(dst + d) = *reinterpret_cast<const uint2*>(o);
@@ -190,7 +197,7 @@ __global__ void decode_advance_kernel(const int64_t* next_tok, int64_t* token_bu
   if (b >= B) return;
   const int len = kv_len[b];
   int s = begin[b] + len;
-  if (s >= limit) s = limit - 1;  // host contract violated: stay inside the buffers
+  if (s >= limit) s = limit - 1;  // the host keeps rows shorter; stay inside the buffers in any case
   if (token_buf != nullptr) {
     const int64_t c = buf_begin[b] + len;
     if (c < buf_ld) token_buf[(int64_t)b * buf_ld + c] = next_tok[b];
@@ -219,7 +226,7 @@ extern "C" int rd_stream_norm(int dtype, const void* table, const int64_t* ids, 
   RD_REQUIRE(weight && y && ((table && ids && !hist) || (!table && hist)), RD_ERR_ARG);
   RD_REQUIRE(m_max >= 1 && H >= 1 && groups >= 1 && H % groups == 0 && (table || n_hist >= 1), RD_ERR_SIZE);
   RD_REQUIRE(coeff || table || n_hist == 1, RD_ERR_ARG);
-  const uintptr_t bits = (uintptr_t)hist | (uintptr_t)x_out | (uintptr_t)y;
+  const uintptr_t bits = (uintptr_t)hist | (uintptr_t)x_out | (uintptr_t)y | (uintptr_t)weight;
   const bool vec = H % 4 == 0 && bits % 16 == 0 && hist_stride % 4 == 0;
   int threads = ((vec ? H / 4 : H) + 31) / 32 * 32;
   // few tokens: the row's loads all in flight at once; many tokens: small blocks, several per SM

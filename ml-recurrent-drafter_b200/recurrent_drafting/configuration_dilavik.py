@@ -22,7 +22,8 @@ class AttentionConfig:
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "AttentionConfig":
-        c = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), int(d["rot"]["dims"]), float(d["rot"]["base"]),
+        rot = d.get("rot") or {"dims": 0, "base": 1.0}
+        c = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), int(rot["dims"]), float(rot["base"]),
                 float(d["scale"]), int(d["mask"]["size"]), int(d["mask"]["keep_first"]))
         if c.heads % c.kv_heads or c.rot_dims % 2 or c.rot_dims > c.dim or c.window < 1 or c.keep_first < 0:
             raise ValueError(f"inconsistent attention configuration {d}")

@@ -189,7 +189,7 @@ def check_attention(res, dtype):
         assert np.abs(got - want).max() < (3e-5 if dtype == torch.float32 else 3e-2), np.abs(got - want).max()
 
 
-SIZES = [(32, 24, 16, 4, 2), (64, 48, 32, 8, 2), (128, 128, 128, 4, 1), (128, 64, 20, 2, 2), (40, 120, 40, 3, 1), (200, 256, 64, 2, 1),
+SIZES = [(32, 24, 16, 4, 2), (64, 56, 24, 6, 2), (128, 128, 128, 4, 1), (128, 64, 20, 2, 2), (40, 120, 40, 3, 1), (200, 256, 64, 2, 1),
          (10, 14, 6, 3, 3), (12, 5, 0, 6, 2)]
 
 
@@ -208,7 +208,7 @@ def test_window_attention(dt, d, dv, rot, H, G, window, keep):
 def test_one_key_at_every_edge_of_the_window(dt, cached, new, window, keep):
     """A key that outweighs all others sits just inside or just outside the window, or among or behind the kept tokens:
     the output is its value, or is not moved by it."""
-    mix = db.attention(4, 2, 64, 48, 32, 3000.0, 0.125, window, keep)["mixer"]
+    mix = db.attention(4, 2, 64, 56, 24, 3000.0, 0.125, window, keep)["mixer"]
     q = 199
     for key in (q - window + 1, q - window, q - window - 1, 0, max(keep - 1, 0), keep, keep + 1, 64, 63, 128, q, q - 1):
         res = run_attention(mix, [(cached, new)], DTYPES[dt], boost=(0, q, key, 4.0))
@@ -314,7 +314,7 @@ class Memory:
                     close(got, want, torch.float32, 2e-4)
 
 
-MEMORY_SIZES = [(2, 32, 64), (1, 256, 96), (3, 16, 40), (2, 64, 32), (1, 128, 200), (2, 72, 8), (1, 200, 512)]
+MEMORY_SIZES = [(2, 32, 72), (1, 256, 96), (3, 16, 40), (2, 64, 32), (1, 128, 200), (2, 72, 8), (1, 200, 512)]
 
 
 @pytest.mark.parametrize("dt,kernel", [("fp32", "scan"), ("bf16", "scan"), ("bf16", "chunk")])
@@ -359,7 +359,7 @@ def test_matrix_memory_of_many_unequal_rows():
 
 
 @pytest.mark.parametrize("dt", ["fp32", "bf16"])
-@pytest.mark.parametrize("heads,d,dv", [(2, 32, 64), (1, 256, 96), (2, 6, 10)])
+@pytest.mark.parametrize("heads,d,dv", [(2, 24, 64), (1, 256, 96), (2, 6, 10)])
 def test_matrix_memory_over_a_draft_tree_and_its_commit(dt, heads, d, dv):
     from recurrent_drafting import _lib
 
