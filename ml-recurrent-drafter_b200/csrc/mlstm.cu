@@ -377,8 +377,7 @@ int launch_tree(const MlstmArgs& a, int B, int m_max, const uint32_t* tree_mask,
                                        tree_mask, mask_words, o);
   RD_CHECK_CHAINED(err);
   const T* gp = (const T*)a.proj + (int64_t)2 * a.nh * a.dim + (int64_t)a.nh * a.vdim;
-  return launch_norm_gate<T>(o, gp, a.ld, a.norm_w, a.out, a.eps, m_max, a.row_start, B, a.nh, a.dim, a.vdim, nullptr, nullptr,
-                             nullptr, s);
+  return launch_norm_gate<T>(o, gp, a.ld, a.norm_w, a.out, a.eps, m_max, a.row_start, B, a.nh, a.vdim, s);
 }
 
 }  // namespace

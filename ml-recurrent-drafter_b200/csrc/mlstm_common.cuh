@@ -9,28 +9,16 @@ constexpr float kDenEps = 1e-6f;
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
-// Per token and head: o / rms(o) * norm weight * sigmoid(g), one warp per head.  With nm given, block b < B also moves row
-// b's n and m to the state: every CTA of the kernel before has read the old ones by now.
+// Per token and head: o / rms(o) * norm weight * sigmoid(g), one warp per head.
 constexpr int kNormThreads = 256;
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kNormThreads) norm_gate_kernel(
     const float* o, const T* g, int64_t ld, const T* w, T* out, float eps,
-    const int32_t* row_start, int B, int nh, int dim, int vdim, const float* nm, float* n,
-    float* m) {
+    const int32_t* row_start, int B, int nh, int vdim) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (nm != nullptr && t < B && row_start[t + 1] > row_start[t]) {
-    for (int i = threadIdx.x; i < nh * (dim + 1); i += kNormThreads) {
-      const int h = i / (dim + 1), d = i % (dim + 1);
-      const float v = nm[(int64_t)t * nh * (dim + 1) + i];
-      if (d < dim)
-        n[((int64_t)t * nh + h) * dim + d] = v;
-      else
-        m[(int64_t)t * nh + h] = v;
-    }
-  }
   if (t >= row_start[B]) return;
   for (int h = warp; h < nh; h += kNormThreads / 32) {
     const int64_t base = ((int64_t)t * nh + h) * vdim;
@@ -78,17 +66,17 @@ __global__ void __launch_bounds__(kNormThreads) norm_gate_kernel(
 // rows: upper bound of the packed tokens
 template <typename T>
 int launch_norm_gate(const float* o, const void* g, int64_t ld, const void* w, void* out, float eps, int rows, const int32_t* row_start,
-                     int B, int nh, int dim, int vdim, const float* nm, float* n, float* m, cudaStream_t s) {
+                     int B, int nh, int vdim, cudaStream_t s) {
   const bool vec = sizeof(T) == 2 && vdim % 4 == 0 && ld % 4 == 0 && (((uintptr_t)o | (uintptr_t)out) & 15) == 0 &&
                    (((uintptr_t)g | (uintptr_t)w) & 7) == 0;
-  const dim3 grid(rows > B ? rows : B);
+  const dim3 grid(rows);
   cudaError_t err;
   if constexpr (sizeof(T) == 2) {
     err = rd::launch_chained(vec ? norm_gate_kernel<T, 4> : norm_gate_kernel<T, 1>, grid, dim3(kNormThreads), 0, s, 1, o, (const T*)g, ld,
-                             (const T*)w, (T*)out, eps, row_start, B, nh, dim, vdim, nm, n, m);
+                             (const T*)w, (T*)out, eps, row_start, B, nh, vdim);
   } else {
     err = rd::launch_chained(norm_gate_kernel<T, 1>, grid, dim3(kNormThreads), 0, s, 1, o, (const T*)g, ld, (const T*)w, (T*)out, eps,
-                             row_start, B, nh, dim, vdim, nm, n, m);
+                             row_start, B, nh, vdim);
   }
   RD_CHECK_CHAINED(err);
   return RD_OK;
