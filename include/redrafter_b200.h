@@ -51,6 +51,7 @@ extern "C" {
 #define RD_EPI_RES 4           /* C = R[m,n] + acc (R may alias C) */
 #define RD_EPI_SWIGLU 5        /* C[m,i] = silu(acc[m,2i]) * acc[m,2i+1]; C has N/2 columns */
 #define RD_EPI_XIELU 9         /* C = xIELU(acc); through rd_gemm_xielu / rd_gemm_bf16_tc_xielu, which take its coefficients */
+#define RD_EPI_CLAMPED_GLU 11  /* gated unit with cut inputs; through rd_gemm_clamped_glu / rd_gemm_bf16_tc_clamped_glu */
 
 /* Attention visibility of the new tokens among themselves. */
 #define RD_ATTN_CAUSAL 0 /* new token i sees new tokens 0..i */
@@ -183,6 +184,18 @@ RD_API int rd_gemm_xielu(int dtype, const void* A, int64_t lda, const void* W, i
 RD_API int rd_gemm_bf16_tc_xielu(const void* plan, void* C, int64_t ldc, const int32_t* m_dev, float pos, float neg,
                           int32_t* status, void* stream);
 
+/* C[m,i] = g sigmoid(alpha g) (u + 1) with g = min(acc[m,2i], limit) and u = acc[m,2i+1] cut to [-limit, limit]; C has N/2
+ * columns.  No counterpart in the reference. */
+RD_API int rd_gemm_clamped_glu(int dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int m_max,
+                        const int32_t* m_dev, int N, int K, float limit, float alpha, void* stream);
+RD_API int rd_gemm_bf16_tc_clamped_glu(const void* plan, void* C, int64_t ldc, const int32_t* m_dev, float limit, float alpha,
+                                int32_t* status, void* stream);
+
+/* One product per head: C[t, h, n] = sum_k A[t, h, k] W[h, n, k], with A at A + t*lda + h*a_head, C at C + t*ldc + h*c_head and W
+ * [heads, N, K] dense.  dtype of all three.  For few tokens per head (decoding); fp32 sums.  No counterpart in the reference. */
+RD_API int rd_head_gemm(int dtype, const void* A, int64_t lda, int64_t a_head, const void* W, void* C, int64_t ldc, int64_t c_head,
+                 int m_max, const int32_t* m_dev, int heads, int N, int K, void* stream);
+
 /* A W^T whose output features [0, n_split) go to C as bf16 and [n_split, N) to C_hi as fp32 (column n - n_split):
  * projections some of whose outputs must not be rounded, such as the gates of a recurrence.  n_split a multiple of 32. */
 RD_API int rd_gemm_bf16_tc_split(const void* plan, void* C, int64_t ldc, float* C_hi, int64_t ld_hi, int n_split,
@@ -206,6 +219,14 @@ RD_API int rd_gemm_bf16_tc_qkvg_rope(const void* plan, const int32_t* m_dev, voi
                               void* gate_out, int64_t ld_gate, const int32_t* tok_row, const int32_t* tok_pos,
                               const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos, int nh, int nkv,
                               int hd, int rot_dims, int max_len, int32_t* status, void* stream);
+
+/* The same without v and gate rows ((nh + nkv) * 128 in all) for models whose values are the keys as projected and whose q
+ * and k heads are divided by their root mean square, sqrt(mean + eps), after the rotation; values and rotated, normed keys
+ * go to v_cache and k_cache.  The head stays fp32 from the product to the one rounding of each result. */
+RD_API int rd_gemm_bf16_tc_qk_rope_norm(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,
+                                 const int32_t* tok_row, const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_table,
+                                 const float* sin_table, int n_pos, int nh, int nkv, int hd, int rot_dims, int max_len, float eps,
+                                 int32_t* status, void* stream);
 
 /* LlamaRMSNorm (modeling_llama.py:21-34) folded into the two GEMMs around it, so that the norm between a residual
  * projection and the next projection needs no kernel of its own (bf16, tensor-core path).
@@ -296,12 +317,12 @@ RD_API int rd_attention_tc(const void* plan, void* out, const int32_t* row_start
                            const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
                            int32_t* status, void* stream);
 
-/* rd_attention_tc with the visibility and the gate of rd_attention_window (see there); scale > 0; in mode RD_ATTN_TREE the
- * window is at least RD_MAX_BEAM_LENGTH. */
-RD_API int rd_attention_tc_window(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
+/* rd_attention_tc with the visibility, the gate and the sink of rd_attention_masked (see there); scale > 0; mode
+ * RD_ATTN_TREE only with RD_MASK_WINDOW and a window of at least RD_MAX_BEAM_LENGTH. */
+RD_API int rd_attention_tc_masked(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
                            const int32_t* base_len, int max_new, int mode, const int32_t* tok_pos, const uint32_t* tree_mask,
-                           int mask_words, float scale, int window, int keep_first, const void* gate, int64_t ld_gate,
-                           int32_t* status, void* stream);
+                           int mask_words, float scale, int mask_kind, int window, int keep_first, const void* gate,
+                           int64_t ld_gate, const float* sink, int32_t* status, void* stream);
 
 /* rd_attention_tc with the key range of every (row, head) cut into n_split shares (1..RD_ATTN_MAX_SPLIT), one CTA
  * each, merged by a second kernel: for launches with fewer (row, head) pairs than the GPU has SMs and long caches
@@ -442,6 +463,66 @@ RD_API int rd_attention_window(int dtype, const void* q, int64_t ldq, const void
                         int64_t ld_gate, void* out, const int32_t* row_start, const int32_t* kv_begin, const int32_t* base_len,
                         int B, int nh, int nkv, int dim, int vdim, int max_len, int max_new, int mode, const int32_t* tok_pos,
                         const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first, int max_kv, void* stream);
+
+/* The general form of the above.  Key j of row b under key/value head g starts at k + b*k_batch + g*k_head + (kv_begin[b] + j)*k_row
+ * (strides in elements); its last tail_dim features may come from k_tail, one vector per key for all heads.  Values likewise.
+ * mask_kind RD_MASK_WINDOW: as above; RD_MASK_CHUNK: a query at position p sees s <= p iff p / window == s / window (or s <
+ * keep_first).  sink (optional, fp32 [nh]): a score per head that takes part in the softmax's sum without a value.  Where v
+ * is k (the values are the first vdim features of the one key all heads share) keys are read once for both. */
+#define RD_MASK_WINDOW 0
+#define RD_MASK_CHUNK 1
+typedef struct rd_attention_desc {
+  const void* q;
+  int64_t ldq;
+  const void* k;
+  int64_t k_batch, k_head, k_row;
+  const void* k_tail;
+  int64_t tail_batch, tail_row;
+  const void* v;
+  int64_t v_batch, v_head, v_row;
+  const void* gate;
+  int64_t ld_gate;
+  const float* sink;
+  void* out;
+  const int32_t* row_start;
+  const int32_t* kv_begin;
+  const int32_t* base_len;
+  const int32_t* tok_pos;
+  const uint32_t* tree_mask;
+  int32_t mask_words, dtype, B, nh, nkv, dim, tail_dim, vdim, max_new, max_kv, mode;
+  int32_t mask_kind, window, keep_first;
+  float scale;
+} rd_attention_desc;
+RD_API int rd_attention_masked(const rd_attention_desc* desc, void* stream);
+RD_API int rd_attention_desc_bytes(void); /* sizeof(rd_attention_desc), for bindings that restate it */
+
+/* Rotary embedding of the first rot_dims features of every q and k head, then (eps >= 0) each of these heads over its root
+ * mean square, and the cache append.  neighbours != 0 pairs features 2i and 2i+1, otherwise i and i + rot_dims/2; tables
+ * [n_pos, rot_dims/2].  proj row: q [nh*dim] | k [nkv*dim] | v [nkv*vdim] in `dtype`; vdim 0: the values are the keys as
+ * projected (the value cache then has rows of dim).  q is replaced in place. */
+RD_API int rd_rotary_norm_append(int dtype, void* proj, int64_t ld, void* k_cache, void* v_cache, const int32_t* tok_row,
+                          const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos,
+                          int m_max, const int32_t* m_dev, int nh, int nkv, int dim, int vdim, int rot_dims, int neighbours,
+                          float eps, int max_len, void* stream);
+
+/* Latent attention, the new tokens' part: the first `rank` values of a row of dkv (fp32) over their root mean square, times
+ * norm_weight, and the last rot_dim of them rotated go to cache [B, max_len, rank + rot_dim] at the token's slot.  The rot_dim
+ * features of every query head at q + t*ldq + h*(dim + rot_dim) + dim are rotated and written to q_rot + t*ld_rot + h*rot_head
+ * (which may be where they came from).  Rotation as in rd_rotary_norm_append, of the first rot_dims of the rot_dim features. */
+RD_API int rd_latent_append(int dtype, const void* q, int64_t ldq, void* q_rot, int64_t ld_rot, int64_t rot_head, const float* dkv,
+                     int64_t ld_dkv, const void* norm_weight, float eps, void* cache, const int32_t* tok_row, const int32_t* tok_pos,
+                     const int32_t* tok_slot, const float* cos_table, const float* sin_table, int n_pos, int m_max,
+                     const int32_t* m_dev, int nh, int dim, int rot_dim, int rot_dims, int neighbours, int rank, int max_len,
+                     void* stream);
+
+/* Latent attention, prompts: the cache rows that some new token of a row sees, from the first of them rounded down to a
+ * multiple of RD_GATHER_ALIGN, row after row into out [rows_max, width], followed by RD_GATHER_ALIGN - 1 rows of zeros.
+ * out_begin[b]: index of row b's key 0 in out (it may be negative: that key itself need not be there); n_out: rows written,
+ * zeros included. */
+#define RD_GATHER_ALIGN 64
+RD_API int rd_latent_gather(int dtype, const void* cache, int width, int max_len, const int32_t* row_start, const int32_t* kv_begin,
+                     const int32_t* base_len, int B, int mask_kind, int window, void* out, int rows_max, int32_t* out_begin,
+                     int32_t* n_out, void* stream);
 
 /* Matrix-memory recurrence with exponential gates over the new tokens of every row, token after token, continuing and
  * updating the row's fp32 state S [B, nh, dim, vdim], n [B, nh, dim], m [B, nh] (a row whose base_len is 0 starts from

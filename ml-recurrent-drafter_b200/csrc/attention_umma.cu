@@ -28,7 +28,7 @@
 // lets outstanding bulk copies land, frees its TMEM and returns.
 #include <cuda.h>
 
-#include "rd_common.cuh"
+#include "attention_window.cuh"
 
 namespace {
 
@@ -182,13 +182,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// WIN: sliding window with kept first tokens and an output gate per head.  Only the key tiles that hold a kept token or lie
-// in some query's window are visited.
+// WIN: sliding window or chunk with kept first tokens, an output gate and a sink per head.  Only the key tiles that hold a
+// kept token or that some query sees are visited.
 struct WindowArgs {
-  int window, keep_first;
+  int mask_kind, window, keep_first;
   const __nv_bfloat16* gate;  // optional [m, ld_gate]
   int64_t ld_gate;
   const int32_t* tok_pos;     // tree mode: positions of the new tokens
+  const float* sink;          // optional [nh]
 };
 
 template <bool WIN>
@@ -236,7 +237,7 @@ __global__ void __launch_bounds__(kThreads, 2)
   int all_tiles = (kv_end + BNK - 1) / BNK;
   int kept_tiles = 0, first_tile = 0;  // WIN: tiles of the kept tokens, then [first_tile, end)
   if (WIN) {
-    const int lo = base + (mode == RD_ATTN_CAUSAL ? q0 : 0) - win.window + 1;
+    const int lo = rd_win::first_visible(win.mask_kind, win.window, base + (mode == RD_ATTN_CAUSAL ? q0 : 0));
     first_tile = lo > 0 ? lo / BNK : 0;
     kept_tiles = min((min(win.keep_first, kv_end) + BNK - 1) / BNK, first_tile);
     all_tiles += kept_tiles - first_tile;
@@ -402,6 +403,11 @@ __global__ void __launch_bounds__(kThreads, 2)
       for (int w = 0; w < mask_words; ++w) sMask[r * mask_words + w] = live ? tree_mask[(int64_t)(rs + qi) * mask_words + w] : 0u;
     }
     const uint32_t* my_mask = sMask + r * mask_words;  // written and read by this thread only
+    int first_seen = 0;  // WIN: first position this row's query sees
+    if (WIN) {
+      const int p = mode == RD_ATTN_CAUSAL ? base + qi : (live ? win.tok_pos[rs + qi] : base);
+      first_seen = rd_win::first_visible(win.mask_kind, win.window, p);
+    }
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     int site = 0;  // which wait gave up (reported in the status word)
@@ -445,9 +451,8 @@ __global__ void __launch_bounds__(kThreads, 2)
         vis &= (n_in <= 0) ? 0ull : ((1ull << n_in) - 1ull);
       }
       if (WIN) {
-        // position of the query; keys before p - window + 1 are gone unless they are among the kept ones
-        const int p = mode == RD_ATTN_CAUSAL ? base + qi : (live ? win.tok_pos[rs + qi] : base);
-        const int gone = p - win.window + 1 - j0, kept = win.keep_first - j0;
+        // keys before the query's first visible one are gone unless they are among the kept ones
+        const int gone = first_seen - j0, kept = win.keep_first - j0;
         const uint64_t in_window = gone <= 0 ? ~0ull : (gone >= 64 ? 0ull : ~0ull << gone);
         const uint64_t among_kept = kept <= 0 ? 0ull : (kept >= 64 ? ~0ull : (1ull << kept) - 1ull);
         vis &= in_window | among_kept;
@@ -546,7 +551,7 @@ __global__ void __launch_bounds__(kThreads, 2)
       }
     } else if (ok) {
       tc_fence_after();
-      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      float inv = WIN ? rd_win::finish_softmax(m_run, l_run, win.sink, h) : (l_run > 0.f ? 1.0f / l_run : 0.f);
       if (WIN && win.gate != nullptr && live) inv /= 1.0f + __expf(-__bfloat162float(win.gate[(int64_t)(rs + qi) * win.ld_gate + h]));
       uint4* dst = reinterpret_cast<uint4*>(out + ((int64_t)(rs + qi) * nh + h) * HD);
 #pragma unroll 1
@@ -699,14 +704,16 @@ extern "C" int rd_attention_tc_split(const void* plan, void* out, const int32_t*
                              workspace_bytes, status, stream, nullptr, 1.0f / sqrtf((float)HD));
 }
 
-extern "C" int rd_attention_tc_window(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
+extern "C" int rd_attention_tc_masked(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,
                                       const int32_t* base_len, int max_new, int mode, const int32_t* tok_pos,
-                                      const uint32_t* tree_mask, int mask_words, float scale, int window, int keep_first,
-                                      const void* gate, int64_t ld_gate, int32_t* status, void* stream) {
-  // the kernel's running maximum is taken before the scale, and a tree's own tokens must lie inside every window
+                                      const uint32_t* tree_mask, int mask_words, float scale, int mask_kind, int window,
+                                      int keep_first, const void* gate, int64_t ld_gate, const float* sink, int32_t* status,
+                                      void* stream) {
+  // the kernel's running maximum is taken before the scale, and a tree's own tokens must all be visible by position
+  RD_REQUIRE(mask_kind == RD_MASK_WINDOW || (mask_kind == RD_MASK_CHUNK && mode == RD_ATTN_CAUSAL), RD_ERR_UNSUPPORTED);
   RD_REQUIRE(scale > 0.f && window >= (mode == RD_ATTN_TREE ? RD_MAX_BEAM_LENGTH : 1) && keep_first >= 0, RD_ERR_SIZE);
   RD_REQUIRE(mode != RD_ATTN_TREE || tok_pos, RD_ERR_ARG);
-  const WindowArgs win{window, keep_first, (const __nv_bfloat16*)gate, ld_gate, tok_pos};
+  const WindowArgs win{mask_kind, window, keep_first, (const __nv_bfloat16*)gate, ld_gate, tok_pos, sink};
   return attention_tc_launch(plan, out, row_start, kv_begin, base_len, max_new, mode, tree_mask, mask_words, 1, nullptr, 0, status,
                              stream, &win, scale);
 }

@@ -1,5 +1,6 @@
-// Sliding-window attention with kept first tokens, grouped key/value heads, different key and value sizes,
-// a free score scale and an output gate per head (see attention_window.cuh for the visibility rule).
+// Attention over a sliding window or a chunk with kept first tokens, grouped key/value heads, different key and value
+// sizes, a free score scale, an output gate and a sink per head, and key features that all heads share (see
+// attention_window.cuh for the visibility rule).
 //
 //   attention_window_rowwise_kernel  any dtype and size: one warp per (query, head), online softmax over 32 keys
 //                                    at a time, exact expf.  fp32 models and odd sizes.
@@ -10,9 +11,9 @@
 namespace {
 
 constexpr int kRowWarps = 8;
-constexpr int kMaxV = 16;  // value features per lane: vdim <= 512
 
-template <typename T>
+// kMaxV: value features per lane
+template <typename T, int kMaxV>
 __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kernel(const rd_win::Args a) {
   rd::pdl_launch_dependents();
   rd::pdl_wait();
@@ -29,9 +30,9 @@ __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kerne
   const T* qrow = (const T*)a.q + (int64_t)t * a.ldq + (int64_t)h * a.dim;
   for (int d = lane; d < a.dim; d += 32) qs[d] = rd::Num<T>::to_f(qrow[d]);
   __syncwarp();
-  const int64_t row0 = ((int64_t)b * a.nkv + hk) * a.max_len + a.kv_begin[b];
-  const T* kb = (const T*)a.k_cache + row0 * a.dim;
-  const T* vb = (const T*)a.v_cache + row0 * a.vdim;
+  rd_win::RowKeys<T> keys;
+  keys.init(a, b, hk);
+  const int own = a.dim - a.tail_dim;  // key features that belong to the head
   rd_win::Query qu;
   qu.init(a, a.base_len[b], rs, n_new, i);
   float m = -INFINITY, l = 0.f;
@@ -46,9 +47,13 @@ __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kerne
       const int j = j0 + lane;
       float s = -INFINITY;
       if (j < j_hi && qu.sees(a, j)) {
-        const T* kr = kb + (int64_t)j * a.dim;
+        const T* kr = keys.k + (int64_t)j * a.k_row;
         float dot = 0.f;
-        for (int d = 0; d < a.dim; ++d) dot = fmaf(qs[d], rd::Num<T>::to_f(kr[d]), dot);
+        for (int d = 0; d < own; ++d) dot = fmaf(qs[d], rd::Num<T>::to_f(kr[d]), dot);
+        if (a.tail_dim > 0) {
+          const T* tr = keys.tail + (int64_t)j * a.tail_row;
+          for (int d = own; d < a.dim; ++d) dot = fmaf(qs[d], rd::Num<T>::to_f(tr[d - own]), dot);
+        }
         s = dot * a.scale;
       }
       const float mt = rd::warp_max(s);
@@ -64,7 +69,7 @@ __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kerne
       for (int jj = 0; jj < n; ++jj) {
         const float pj = __shfl_sync(0xffffffffu, p, jj);
         if (pj == 0.f) continue;
-        const T* vr = vb + (int64_t)(j0 + jj) * a.vdim;
+        const T* vr = keys.v + (int64_t)(j0 + jj) * a.v_row;
 #pragma unroll
         for (int v = 0; v < kMaxV; ++v)
           if (v * 32 + lane < a.vdim) acc[v] = fmaf(pj, rd::Num<T>::to_f(vr[v * 32 + lane]), acc[v]);
@@ -72,6 +77,10 @@ __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kerne
     }
   }
   float f = l > 0.f ? 1.0f / l : 0.f;
+  if (a.sink != nullptr && l > 0.f) {
+    const float s = a.sink[h], top = fmaxf(m, s), w = expf(m - top);
+    f = w / (l * w + expf(s - top));
+  }
   if (a.gate != nullptr) f *= rd_win::sigmoid_exact(rd::Num<T>::to_f(((const T*)a.gate)[(int64_t)t * a.ld_gate + h]));
   T* orow = (T*)a.out + ((int64_t)t * a.nh + h) * a.vdim;
 #pragma unroll
@@ -79,46 +88,79 @@ __global__ void __launch_bounds__(kRowWarps * 32) attention_window_rowwise_kerne
     if (v * 32 + lane < a.vdim) orow[v * 32 + lane] = rd::Num<T>::from_f(acc[v] * f);
 }
 
-template <typename T>
-int launch_rowwise(const rd_win::Args& a, int B, int max_new, cudaStream_t s) {
+template <typename T, int kMaxV>
+int launch_rowwise_v(const rd_win::Args& a, cudaStream_t s) {
   const size_t smem = (size_t)kRowWarps * a.dim * sizeof(float);
-  RD_REQUIRE(smem <= 48 * 1024 && a.vdim <= kMaxV * 32, RD_ERR_SIZE);
-  dim3 grid((max_new + kRowWarps - 1) / kRowWarps, a.nh, B);
-  cudaError_t err = rd::launch_chained(attention_window_rowwise_kernel<T>, grid, dim3(kRowWarps * 32), smem, s, 1, a);
+  RD_REQUIRE(smem <= 48 * 1024, RD_ERR_SIZE);
+  dim3 grid((a.max_new + kRowWarps - 1) / kRowWarps, a.nh, a.B);
+  cudaError_t err = rd::launch_chained(attention_window_rowwise_kernel<T, kMaxV>, grid, dim3(kRowWarps * 32), smem, s, 1, a);
   RD_CHECK_CHAINED(err);
   return RD_OK;
 }
 
+template <typename T>
+int launch_rowwise(const rd_win::Args& a, cudaStream_t s) {
+  if (a.vdim <= 8 * 32) return launch_rowwise_v<T, 8>(a, s);
+  if (a.vdim <= 16 * 32) return launch_rowwise_v<T, 16>(a, s);
+  RD_REQUIRE(a.vdim <= 32 * 32, RD_ERR_SIZE);
+  return launch_rowwise_v<T, 32>(a, s);
+}
+
 }  // namespace
+
+int rd_attention_latent_launch(const rd_win::Args& a, cudaStream_t s);  // attention_latent.cu
+bool rd_attention_latent_ok(const rd_win::Args& a);
+
+extern "C" int rd_attention_masked(const rd_attention_desc* desc, void* stream) {
+  RD_REQUIRE(desc, RD_ERR_ARG);
+  const rd_win::Args& a = *desc;
+  RD_REQUIRE(a.q && a.k && a.v && a.out && a.row_start && a.kv_begin && a.base_len, RD_ERR_ARG);
+  RD_REQUIRE(a.mode == RD_ATTN_CAUSAL || (a.mode == RD_ATTN_TREE && a.tree_mask && a.tok_pos && a.mask_words >= 1), RD_ERR_ARG);
+  RD_REQUIRE(a.dtype == RD_F32 || a.dtype == RD_BF16, RD_ERR_DTYPE);
+  RD_REQUIRE(a.mask_kind == RD_MASK_WINDOW || a.mask_kind == RD_MASK_CHUNK, RD_ERR_ARG);
+  RD_REQUIRE(a.B >= 1 && a.B <= 65535 && a.nh >= 1 && a.nh <= 65535 && a.nkv >= 1 && a.nh % a.nkv == 0 && a.dim >= 1 && a.vdim >= 1 &&
+                 a.max_new >= 1 && a.window >= 1 && a.keep_first >= 0 && a.ldq >= (int64_t)a.nh * a.dim && a.tail_dim >= 0 &&
+                 a.tail_dim < a.dim && (a.tail_dim == 0 || a.k_tail),
+             RD_ERR_SIZE);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (a.dtype == RD_F32) return launch_rowwise<float>(a, s);
+  if (rd_attention_latent_ok(a)) return rd_attention_latent_launch(a, s);
+  const uintptr_t bits = (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.out | (uintptr_t)(a.tail_dim ? a.k_tail : nullptr);
+  const int64_t strides = a.ldq | a.k_batch | a.k_head | a.k_row | a.v_batch | a.v_head | a.v_row |
+                          (a.tail_dim ? a.tail_batch | a.tail_row | a.tail_dim : 0);
+  if (a.dim % 8 == 0 && a.vdim % 8 == 0 && strides % 8 == 0 && bits % 16 == 0 && a.dim <= 256 && a.vdim <= 256) {
+    // two row tiles of queries per key/value head are still cheaper to read K and V for than one 128-query tile per head
+    const bool decode = (a.nh / a.nkv) * a.max_new <= 2 * rd_win::kRows;
+    if (decode) {
+      if (a.dim <= 64 && a.vdim <= 64) return rd_win::launch_decode<64, 64>(a, s);
+      if (a.dim <= 128 && a.vdim <= 128) return rd_win::launch_decode<128, 128>(a, s);
+      return rd_win::launch_decode<256, 256>(a, s);
+    }
+    if (a.dim <= 64 && a.vdim <= 64) return rd_win::launch_prefill<64, 64>(a, s);
+    if (a.dim <= 64 && a.vdim <= 128) return rd_win::launch_prefill<64, 128>(a, s);
+    if (a.dim <= 128 && a.vdim <= 64) return rd_win::launch_prefill<128, 64>(a, s);
+    if (a.dim <= 128 && a.vdim <= 128) return rd_win::launch_prefill<128, 128>(a, s);
+  }
+  return launch_rowwise<__nv_bfloat16>(a, s);
+}
+
+extern "C" int rd_attention_desc_bytes(void) { return (int)sizeof(rd_attention_desc); }
 
 extern "C" int rd_attention_window(int dtype, const void* q, int64_t ldq, const void* k_cache, const void* v_cache,
                                    const void* gate, int64_t ld_gate, void* out, const int32_t* row_start,
                                    const int32_t* kv_begin, const int32_t* base_len, int B, int nh, int nkv, int dim, int vdim,
                                    int max_len, int max_new, int mode, const int32_t* tok_pos, const uint32_t* tree_mask,
                                    int mask_words, float scale, int window, int keep_first, int max_kv, void* stream) {
-  RD_REQUIRE(q && k_cache && v_cache && out && row_start && kv_begin && base_len, RD_ERR_ARG);
-  RD_REQUIRE(mode == RD_ATTN_CAUSAL || (mode == RD_ATTN_TREE && tree_mask && tok_pos && mask_words >= 1), RD_ERR_ARG);
-  RD_REQUIRE(dtype == RD_F32 || dtype == RD_BF16, RD_ERR_DTYPE);
-  RD_REQUIRE(B >= 1 && B <= 65535 && nh >= 1 && nh <= 65535 && nkv >= 1 && nh % nkv == 0 && dim >= 1 && vdim >= 1 && max_len >= 1 &&
-                 max_new >= 1 && window >= 1 && keep_first >= 0 && ldq >= (int64_t)nh * dim,
-             RD_ERR_SIZE);
-  rd_win::Args a{q,       ldq,     k_cache, v_cache,   gate,       ld_gate, out, row_start, kv_begin, base_len, tok_pos,
-                 tree_mask, mask_words, nh,   nkv, dim, vdim, max_len, mode, scale, window, keep_first};
-  cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == RD_F32) return launch_rowwise<float>(a, B, max_new, s);
-  const uintptr_t bits = (uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out;
-  if (dim % 8 == 0 && vdim % 8 == 0 && ldq % 8 == 0 && bits % 16 == 0 && dim <= 256 && vdim <= 256) {
-    // two row tiles of queries per key/value head are still cheaper to read K and V for than one 128-query tile per head
-    const bool decode = (nh / nkv) * max_new <= 2 * rd_win::kRows;
-    if (decode) {
-      if (dim <= 64 && vdim <= 64) return rd_win::launch_decode<64, 64>(a, B, max_new, max_kv, s);
-      if (dim <= 128 && vdim <= 128) return rd_win::launch_decode<128, 128>(a, B, max_new, max_kv, s);
-      return rd_win::launch_decode<256, 256>(a, B, max_new, max_kv, s);
-    }
-    if (dim <= 64 && vdim <= 64) return rd_win::launch_prefill<64, 64>(a, B, max_new, s);
-    if (dim <= 64 && vdim <= 128) return rd_win::launch_prefill<64, 128>(a, B, max_new, s);
-    if (dim <= 128 && vdim <= 64) return rd_win::launch_prefill<128, 64>(a, B, max_new, s);
-    if (dim <= 128 && vdim <= 128) return rd_win::launch_prefill<128, 128>(a, B, max_new, s);
-  }
-  return launch_rowwise<__nv_bfloat16>(a, B, max_new, s);
+  RD_REQUIRE(max_len >= 1, RD_ERR_SIZE);
+  rd_attention_desc a{};
+  a.q = q, a.ldq = ldq;
+  a.k = k_cache, a.k_row = dim, a.k_head = (int64_t)max_len * dim, a.k_batch = a.k_head * nkv;
+  a.v = v_cache, a.v_row = vdim, a.v_head = (int64_t)max_len * vdim, a.v_batch = a.v_head * nkv;
+  a.gate = gate, a.ld_gate = ld_gate;
+  a.out = out;
+  a.row_start = row_start, a.kv_begin = kv_begin, a.base_len = base_len, a.tok_pos = tok_pos;
+  a.tree_mask = tree_mask, a.mask_words = mask_words;
+  a.dtype = dtype, a.B = B, a.nh = nh, a.nkv = nkv, a.dim = dim, a.vdim = vdim, a.max_new = max_new, a.max_kv = max_kv, a.mode = mode;
+  a.mask_kind = RD_MASK_WINDOW, a.window = window, a.keep_first = keep_first, a.scale = scale;
+  return rd_attention_masked(&a, stream);
 }

@@ -1,4 +1,4 @@
-// Sliding-window attention on warp-level tensor cores (bf16; query/key size <= DQ, value size <= DV, multiples of 8).
+// Masked attention on warp-level tensor cores (bf16; query/key size <= DQ, value size <= DV, multiples of 8).
 //
 //   prefill  one CTA = 128 queries of one (row, head), 16 per warp; K/V tiles of 64 keys stream through a three-stage
 //            cp.async ring.  Only the tiles that hold a kept token or lie in some query's window are visited.
@@ -24,16 +24,21 @@ __device__ __forceinline__ int swz(int r, int c) {
   return r * (CH * 16) + ((c ^ (r & 7)) << 4);
 }
 
-// 64 rows [row0, row0 + 64) of a [*, dim] matrix into a tile of D features; rows >= row_end and features >= dim are zero
+// 64 rows [row0, row0 + 64) of a matrix with `dim` features and rows ld apart into a tile of D features, the features from
+// dim - tail_dim on from a second matrix; rows >= row_end and features >= dim are zero (row row_end - 1 stands in as address)
 template <int D, int THREADS>
-__device__ __forceinline__ void load_tile(uint8_t* dst, const __nv_bfloat16* src_base, int dim, int row0, int row_end, int tid) {
+__device__ __forceinline__ void load_tile(uint8_t* dst, const __nv_bfloat16* src_base, int64_t ld, int dim, int row0, int row_end, int tid,
+                                          const __nv_bfloat16* tail = nullptr, int64_t ld_tail = 0, int tail_dim = 0) {
   constexpr int CH = D / 8;
 #pragma unroll
   for (int i = 0; i < (kBN * CH) / THREADS; ++i) {
     const int idx = i * THREADS + tid;
     const int r = idx / CH, c = idx % CH;
     const bool in = row0 + r < row_end && c * 8 < dim;
-    cp_async16(dst + swz<CH>(r, c), src_base + (int64_t)(in ? row0 + r : 0) * dim + (in ? c * 8 : 0), in);
+    const int64_t row = in ? row0 + r : row_end - 1;
+    const int d = in ? c * 8 : 0;
+    const __nv_bfloat16* src = d < dim - tail_dim ? src_base + row * ld + d : tail + row * ld_tail + (d - (dim - tail_dim));
+    cp_async16(dst + swz<CH>(r, c), src, in);
   }
 }
 
@@ -83,12 +88,11 @@ __global__ void __launch_bounds__(kPrefillThreads) attention_window_prefill_kern
   const int p_last = tree ? base + RD_MAX_BEAM_LENGTH - 1 : base + min(n_new, q0 + kBM) - 1;
   const int kv_end = tree ? base + n_new : p_last + 1;
   TileRange tiles;
-  tiles.init(p_first - a.window + 1, a.keep_first, kv_end);
+  tiles.init(first_visible(a.mask_kind, a.window, p_first), a.keep_first, kv_end);
   const int n_tiles = tiles.count();
   const int hk = h / (a.nh / a.nkv);
-  const int64_t row0 = ((int64_t)b * a.nkv + hk) * a.max_len + a.kv_begin[b];
-  const __nv_bfloat16* kb = (const __nv_bfloat16*)a.k_cache + row0 * a.dim;
-  const __nv_bfloat16* vb = (const __nv_bfloat16*)a.v_cache + row0 * a.vdim;
+  RowKeys<__nv_bfloat16> keys;
+  keys.init(a, b, hk);
   constexpr int CQ = DQ / 8, CV = DV / 8;
   for (int idx = tid; idx < kBM * CQ; idx += kPrefillThreads) {
     const int r = idx / CQ, c = idx % CQ;
@@ -99,8 +103,8 @@ __global__ void __launch_bounds__(kPrefillThreads) attention_window_prefill_kern
   auto load = [&](int t) {
     if (t < n_tiles) {
       uint8_t* dst = sKV + (t % kStages) * (Y::kK + Y::kV);
-      load_tile<DQ, kPrefillThreads>(dst, kb, a.dim, tiles.tile(t) * kBN, kv_end, tid);
-      load_tile<DV, kPrefillThreads>(dst + Y::kK, vb, a.vdim, tiles.tile(t) * kBN, kv_end, tid);
+      load_tile<DQ, kPrefillThreads>(dst, keys.k, a.k_row, a.dim, tiles.tile(t) * kBN, kv_end, tid, keys.tail, a.tail_row, a.tail_dim);
+      load_tile<DV, kPrefillThreads>(dst + Y::kK, keys.v, a.v_row, a.vdim, tiles.tile(t) * kBN, kv_end, tid);
     }
     cp_async_commit();  // one group per tile, empty or not
   };
@@ -116,6 +120,7 @@ __global__ void __launch_bounds__(kPrefillThreads) attention_window_prefill_kern
 #pragma unroll
   for (int hh = 0; hh < 2; ++hh) qu[hh].init(a, base, rs, n_new, min(q0 + warp * 16 + g + hh * 8, n_new - 1));
   const float scale_log2 = a.scale * kLog2e;
+  const int first_last = first_visible(a.mask_kind, a.window, p_last);
 
   for (int it = 0; it < n_tiles; ++it) {
     cp_async_wait<1>();
@@ -145,7 +150,7 @@ __global__ void __launch_bounds__(kPrefillThreads) attention_window_prefill_kern
     const int j0 = tiles.tile(it) * kBN, j_last = j0 + kBN - 1;
     // a tile that every query of the CTA sees in full needs no mask
     const bool open = j_last <= p_first && j_last < kv_end && (!tree || j_last < base) &&
-                      (j0 > p_last - a.window || j_last < a.keep_first);
+                      (j0 >= first_last || j_last < a.keep_first);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nb = 0; nb < kBN / 8; ++nb)
@@ -204,7 +209,7 @@ __global__ void __launch_bounds__(kPrefillThreads) attention_window_prefill_kern
     l_run[hh] += __shfl_xor_sync(0xffffffffu, l_run[hh], 2);
     const int i = q0 + warp * 16 + g + hh * 8;
     if (i < n_new) {
-      float f = l_run[hh] > 0.f ? 1.0f / l_run[hh] : 0.f;
+      float f = finish_softmax(m_run[hh], l_run[hh], a.sink, h);
       if (a.gate != nullptr) f *= sigmoid_exact(__bfloat162float(((const __nv_bfloat16*)a.gate)[(int64_t)(rs + i) * a.ld_gate + h]));
       __nv_bfloat16* dst = (__nv_bfloat16*)a.out + ((int64_t)(rs + i) * a.nh + h) * a.vdim;
 #pragma unroll
@@ -260,13 +265,12 @@ __global__ void __launch_bounds__(kDecodeThreads) attention_window_decode_kernel
   auto tok_of = [&](int r) { return (row_tile * kRows + r) % n_new; };
   const int kv_end = base + n_new;
   TileRange tiles;
-  tiles.init(base - a.window + 1, a.keep_first, kv_end);  // no query sits before position base
+  tiles.init(first_visible(a.mask_kind, a.window, base), a.keep_first, kv_end);  // no query sits before position base
   const int n_all = tiles.count();
   const int per = (n_all + n_ranks - 1) / n_ranks;
   const int t_begin = min(rank * per, n_all), n_tiles = min(per, n_all - t_begin);
-  const int64_t row0 = ((int64_t)b * a.nkv + hk) * a.max_len + a.kv_begin[b];
-  const __nv_bfloat16* kb = (const __nv_bfloat16*)a.k_cache + row0 * a.dim;
-  const __nv_bfloat16* vb = (const __nv_bfloat16*)a.v_cache + row0 * a.vdim;
+  RowKeys<__nv_bfloat16> keys;
+  keys.init(a, b, hk);
   constexpr int CQ = DQ / 8, CV = DV / 8;
   for (int idx = tid; idx < kRows * CQ; idx += kDecodeThreads) {
     const int r = idx / CQ, c = idx % CQ;
@@ -279,8 +283,8 @@ __global__ void __launch_bounds__(kDecodeThreads) attention_window_decode_kernel
     if (t < n_tiles) {
       uint8_t* dst = ring + (t % kDecodeStages) * (Y::kK + Y::kV);
       const int j0 = tiles.tile(t_begin + t) * kBN;
-      load_tile<DQ, kDecodeThreads>(dst, kb, a.dim, j0, kv_end, tid);
-      load_tile<DV, kDecodeThreads>(dst + Y::kK, vb, a.vdim, j0, kv_end, tid);
+      load_tile<DQ, kDecodeThreads>(dst, keys.k, a.k_row, a.dim, j0, kv_end, tid, keys.tail, a.tail_row, a.tail_dim);
+      load_tile<DV, kDecodeThreads>(dst + Y::kK, keys.v, a.v_row, a.vdim, j0, kv_end, tid);
     }
     cp_async_commit();
   };
@@ -403,7 +407,7 @@ __global__ void __launch_bounds__(kDecodeThreads) attention_window_decode_kernel
       l = fmaf(f, ml[r * 2 + 1], l);
     }
     const int t = rs + tok_of(r), h = head_of(r);
-    float f = l > 0.f ? 1.0f / l : 0.f;
+    float f = finish_softmax(m, l, a.sink, h);
     if (a.gate != nullptr) f *= sigmoid_exact(__bfloat162float(((const __nv_bfloat16*)a.gate)[(int64_t)t * a.ld_gate + h]));
     ((__nv_bfloat16*)a.out)[((int64_t)t * a.nh + h) * a.vdim + d] = __float2bfloat16_rn(acc * f);
   }
@@ -411,7 +415,7 @@ __global__ void __launch_bounds__(kDecodeThreads) attention_window_decode_kernel
 }
 
 template <int DQ, int DV>
-int launch_prefill(const Args& a, int B, int max_new, cudaStream_t s) {
+int launch_prefill(const Args& a, cudaStream_t s) {
   auto kern = attention_window_prefill_kernel<DQ, DV>;
   constexpr int smem = PrefillSmem<DQ, DV>::kBytes;
   static bool set = false;
@@ -420,13 +424,13 @@ int launch_prefill(const Args& a, int B, int max_new, cudaStream_t s) {
     RD_CHECK_CHAINED(e);
     set = true;
   }
-  cudaError_t err = rd::launch_chained(kern, dim3((max_new + kBM - 1) / kBM, a.nh, B), dim3(kPrefillThreads), smem, s, 1, a);
+  cudaError_t err = rd::launch_chained(kern, dim3((a.max_new + kBM - 1) / kBM, a.nh, a.B), dim3(kPrefillThreads), smem, s, 1, a);
   RD_CHECK_CHAINED(err);
   return RD_OK;
 }
 
 template <int DQ, int DV>
-int launch_decode(const Args& a, int B, int max_new, int max_kv, cudaStream_t s) {
+int launch_decode(const Args& a, cudaStream_t s) {
   auto kern = attention_window_decode_kernel<DQ, DV>;
   constexpr int smem = DecodeSmem<DQ, DV>::kBytes;
   static bool set = false;
@@ -435,13 +439,13 @@ int launch_decode(const Args& a, int B, int max_new, int max_kv, cudaStream_t s)
     RD_CHECK_CHAINED(e);
     set = true;
   }
-  const int row_tiles = ((a.nh / a.nkv) * max_new + kRows - 1) / kRows;
+  const int row_tiles = ((a.nh / a.nkv) * a.max_new + kRows - 1) / kRows;
   // a cluster's CTAs share the key tiles of a row: enough of them to fill the GPU twice, at least two tiles each
-  const int64_t visible = (int64_t)a.window + max_new + a.keep_first + 2 * kBN;
-  const int tiles = (int)((visible < max_kv ? visible : max_kv) + kBN - 1) / kBN;
+  const int64_t visible = (int64_t)a.window + a.max_new + a.keep_first + 2 * kBN;
+  const int tiles = (int)((visible < a.max_kv ? visible : a.max_kv) + kBN - 1) / kBN;
   int ranks = 1;
-  while (ranks < 8 && (int64_t)B * a.nkv * row_tiles * ranks < 2 * 148 && tiles / (ranks * 2) >= 2) ranks *= 2;
-  cudaError_t err = rd::launch_chained(kern, dim3(ranks, a.nkv * row_tiles, B), dim3(kDecodeThreads), smem, s, ranks, a);
+  while (ranks < 8 && (int64_t)a.B * a.nkv * row_tiles * ranks < 2 * 148 && tiles / (ranks * 2) >= 2) ranks *= 2;
+  cudaError_t err = rd::launch_chained(kern, dim3(ranks, a.nkv * row_tiles, a.B), dim3(kDecodeThreads), smem, s, ranks, a);
   RD_CHECK_CHAINED(err);
   return RD_OK;
 }

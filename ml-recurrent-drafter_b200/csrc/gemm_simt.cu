@@ -60,11 +60,13 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= M) continue;
-    if (EPI == RD_EPI_SWIGLU) {
+    if (EPI == RD_EPI_SWIGLU || EPI == RD_EPI_CLAMPED_GLU) {
 #pragma unroll
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
-        if (n + 1 < N) store_out<OutT>(C + (int64_t)m * ldc + (n >> 1), rd::silu_exact(acc[i][j]) * acc[i][j + 1]);
+        if (n + 1 < N)
+          store_out<OutT>(C + (int64_t)m * ldc + (n >> 1), EPI == RD_EPI_SWIGLU ? rd::silu_exact(acc[i][j]) * acc[i][j + 1]
+                                                                                : rd::clamped_glu_exact(acc[i][j], acc[i][j + 1], act0, act1));
       }
     } else {
 #pragma unroll
@@ -99,6 +101,7 @@ int launch(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int6
     RD_LAUNCH_EPI(RD_EPI_RES)
     RD_LAUNCH_EPI(RD_EPI_SWIGLU)
     RD_LAUNCH_EPI(RD_EPI_XIELU)
+    RD_LAUNCH_EPI(RD_EPI_CLAMPED_GLU)
     default:
       return RD_ERR_ARG;
   }
@@ -118,8 +121,9 @@ static int gemm_checked(int dtype, int out_dtype, const void* A, int64_t lda, co
   const bool need_res = epilogue == RD_EPI_BIAS_SILU_RES || epilogue == RD_EPI_RES;
   RD_REQUIRE(!need_bias || bias, RD_ERR_ARG);
   RD_REQUIRE(!need_res || R, RD_ERR_ARG);
-  RD_REQUIRE(epilogue != RD_EPI_SWIGLU || N % 2 == 0, RD_ERR_SIZE);
-  RD_REQUIRE(ldc >= (epilogue == RD_EPI_SWIGLU ? N / 2 : N), RD_ERR_SIZE);
+  const bool glu = epilogue == RD_EPI_SWIGLU || epilogue == RD_EPI_CLAMPED_GLU;
+  RD_REQUIRE(!glu || N % 2 == 0, RD_ERR_SIZE);
+  RD_REQUIRE(ldc >= (glu ? N / 2 : N), RD_ERR_SIZE);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == RD_F32 && out_dtype == RD_F32)
     return launch<float, float>(A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, act0, act1, s);
@@ -133,12 +137,19 @@ static int gemm_checked(int dtype, int out_dtype, const void* A, int64_t lda, co
 extern "C" int rd_gemm(int dtype, int out_dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                        const void* bias, const void* R, int64_t ldr, int m_max, const int32_t* m_dev, int N,
                        int K, int epilogue, void* stream) {
-  RD_REQUIRE(epilogue != RD_EPI_XIELU, RD_ERR_ARG);  // it has parameters: rd_gemm_xielu
+  // these have parameters: rd_gemm_xielu, rd_gemm_clamped_glu
+  RD_REQUIRE(epilogue != RD_EPI_XIELU && epilogue != RD_EPI_CLAMPED_GLU, RD_ERR_ARG);
   return gemm_checked(dtype, out_dtype, A, lda, W, ldw, C, ldc, bias, R, ldr, m_max, m_dev, N, K, epilogue, 0.f, 0.f, stream);
 }
 
 extern "C" int rd_gemm_xielu(int dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int m_max,
                              const int32_t* m_dev, int N, int K, float pos, float neg, void* stream) {
   return gemm_checked(dtype, dtype, A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, m_max, m_dev, N, K, RD_EPI_XIELU, pos, neg,
+                      stream);
+}
+
+extern "C" int rd_gemm_clamped_glu(int dtype, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int m_max,
+                                   const int32_t* m_dev, int N, int K, float limit, float alpha, void* stream) {
+  return gemm_checked(dtype, dtype, A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, m_max, m_dev, N, K, RD_EPI_CLAMPED_GLU, limit, alpha,
                       stream);
 }

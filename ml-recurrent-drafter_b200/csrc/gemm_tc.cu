@@ -243,6 +243,8 @@ struct EpiArgs {
   const float* sin_t;
   int n_pos, nh, nkv, max_len;
   int rot_half;               // rotated pairs per head (64 = the whole head): feature i is paired with i + rot_half
+  int head_norm;              // q and k heads over sqrt(mean of squares + head_eps) after the rotation; the values are the raw k
+  float head_eps;
   __nv_bfloat16* gate_out;    // output features past the v heads (one per query head): [tok, ld_gate], plain
   int64_t ld_gate;
   // LlamaRMSNorm folded into the two GEMMs around it (optional; bf16 output, N a multiple of 32).
@@ -261,7 +263,7 @@ struct EpiArgs {
   int64_t ss_in_ld;
   int ss_slices;
   float norm_dim, norm_eps;
-  // RD_EPI_XIELU only: the activation's two coefficients
+  // RD_EPI_XIELU: the activation's two coefficients; RD_EPI_CLAMPED_GLU: its limit and alpha
   float act0, act1;
   // kEpiSplit only: output features >= n_split go to C_hi in fp32
   float* C_hi;
@@ -285,11 +287,15 @@ constexpr int kEpiSliceMax = 8;
 // [n_split, N) as fp32 in a second matrix; n_split is a multiple of 32, so a warp has one kind only
 constexpr int kEpiSplit = 10;
 
+// gated units: weight rows (2i, 2i+1) = (gate_i, up_i), half as many outputs as features
+template <int EPI>
+constexpr bool kGlu = EPI == RD_EPI_SWIGLU || EPI == RD_EPI_CLAMPED_GLU;
+
 constexpr int kScrLd = 36;  // floats per scratch row: 16-byte aligned rows, conflict-free float4 reads
 
 // Element-wise part of the epilogue in accumulator layout (lane = output feature n, i = token).
 template <int EPI>
-__device__ __forceinline__ void epilogue_math(float* v, const EpiArgs& e, int n, int N, bool swiglu_here, float bias) {
+__device__ __forceinline__ void epilogue_math(float* v, const EpiArgs& e, int n, int N, bool glu_here, float bias) {
   if (EPI == RD_EPI_BIAS || EPI == RD_EPI_BIAS_SILU || EPI == RD_EPI_BIAS_SILU_RES) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] += bias;
@@ -302,13 +308,13 @@ __device__ __forceinline__ void epilogue_math(float* v, const EpiArgs& e, int n,
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = rd::xielu_f(v[i], e.act0, e.act1);
   }
-  if (EPI == RD_EPI_SWIGLU && swiglu_here) {
+  if (kGlu<EPI> && glu_here) {
     // feature-per-lane stores only (the vector path forms the product after the transpose):
     // weight rows (2i, 2i+1) = (gate_i, up_i) sit in adjacent lanes; even lanes keep the product
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       const float up = __shfl_xor_sync(0xffffffffu, v[i], 1);
-      v[i] = rd::silu_f(v[i]) * up;
+      v[i] = EPI == RD_EPI_SWIGLU ? rd::silu_f(v[i]) * up : rd::clamped_glu_f(v[i], up, e.act0, e.act1);
     }
   }
 }
@@ -389,17 +395,17 @@ struct ResidualRegs {
 template <int EPI, bool OUT_F32>
 __device__ __forceinline__ void epilogue_block(float* v, const EpiArgs& e, float* scr, int lane, int n_warp0, int tok0,
                                                int tok_limit, int N, bool vec_ok,
-                                               const ResidualRegs<OUT_F32, (EPI == RD_EPI_SWIGLU ? 16 : 32)>& res,
+                                               const ResidualRegs<OUT_F32, (kGlu<EPI> ? 16 : 32)>& res,
                                                const float* s_scale, uint4 gamma8, float* ss_red_block) {
-  constexpr int kOut = (EPI == RD_EPI_SWIGLU) ? 16 : 32;  // output features per token of this warp
+  constexpr int kOut = kGlu<EPI> ? 16 : 32;  // output features per token of this warp
   constexpr bool kRes = (EPI == RD_EPI_BIAS_SILU_RES || EPI == RD_EPI_RES);
   using G = EpiLanes<OUT_F32, kOut>;
-  const int out0 = (EPI == RD_EPI_SWIGLU) ? (n_warp0 >> 1) : n_warp0;  // first output column of the warp
+  const int out0 = kGlu<EPI> ? (n_warp0 >> 1) : n_warp0;  // first output column of the warp
   if (!vec_ok) {
     // feature-per-lane fallback
     const int n = n_warp0 + lane;
-    const bool writer = (EPI == RD_EPI_SWIGLU) ? ((lane & 1) == 0 && n + 1 < N) : (n < N);
-    const int col = (EPI == RD_EPI_SWIGLU) ? (n >> 1) : n;
+    const bool writer = kGlu<EPI> ? ((lane & 1) == 0 && n + 1 < N) : (n < N);
+    const int col = kGlu<EPI> ? (n >> 1) : n;
     if (writer) {
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
@@ -425,7 +431,7 @@ __device__ __forceinline__ void epilogue_block(float* v, const EpiArgs& e, float
   const int sub = lane % G::kLanes, row0 = lane / G::kLanes;
   float* const ss_red = ss_red_block + ((n_warp0 >> 5) & 3) * 32;  // this warp's row of the reduction buffer
   float o[G::kPasses][G::kPer];
-  if (EPI == RD_EPI_SWIGLU) {
+  if (kGlu<EPI>) {
     // the token's 32 features are 16 (gate, up) pairs: one SiLU per output, no lane exchange.  The SiLUs of the
     // block are evaluated stage by stage (all exponentials, then all quotients) to keep the special-function
     // unit's latency off the critical path.
@@ -451,10 +457,20 @@ __device__ __forceinline__ void epilogue_block(float* v, const EpiArgs& e, float
         for (int j = 0; j < G::kPer; ++j) g[p][j] *= sc, u[p][j] *= sc;
       }
     }
+    if (EPI == RD_EPI_CLAMPED_GLU) {
+#pragma unroll
+      for (int p = 0; p < G::kPasses; ++p)
+#pragma unroll
+        for (int j = 0; j < G::kPer; ++j) {
+          g[p][j] = fminf(g[p][j], e.act0);
+          u[p][j] = fminf(fmaxf(u[p][j], -e.act0), e.act0) + 1.0f;
+        }
+    }
+    const float slope = EPI == RD_EPI_CLAMPED_GLU ? -e.act1 : -1.0f;
 #pragma unroll
     for (int p = 0; p < G::kPasses; ++p)
 #pragma unroll
-      for (int j = 0; j < G::kPer; ++j) o[p][j] = __expf(-g[p][j]);
+      for (int j = 0; j < G::kPer; ++j) o[p][j] = __expf(slope * g[p][j]);
 #pragma unroll
     for (int p = 0; p < G::kPasses; ++p)
 #pragma unroll
@@ -648,7 +664,7 @@ __device__ __forceinline__ void norm_scale_stage(const EpiArgs& e, float* s_scal
 // each), so the cos/sin reads and the stores of an instruction cover 8 rows, not 32.
 __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArgs& e, float* scr_all, int quarter, int lane,
                                                     int head, int tok0, int tok_limit, const int* s_pos, const int* s_dst,
-                                                    const float* s_scale) {
+                                                    const float* s_scale, float* ss_red) {
   float* scr = scr_all + quarter * 32 * kScrLd;
   const bool is_v = head >= e.nh + e.nkv;
   const int sub = lane & 3, row0 = lane >> 2;
@@ -670,9 +686,9 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
       }
     }
   }
-  if (s_scale != nullptr) {
+  if (s_scale != nullptr || e.head_norm) {
     // folded RMS norm: the projection of the normalised row is the projection of the row times its scale; scaled and
-    // rounded after the exchange, where a lane holds one token's values
+    // rounded after the exchange, where a lane holds one token's values.  Normed heads are rounded once, at the end.
 #pragma unroll
     for (int i = 0; i < 32; ++i) scr[i * kScrLd + lane] = v[i];
   } else {
@@ -688,6 +704,22 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
     const float4 a0 = *reinterpret_cast<const float4*>(own), a1 = *reinterpret_cast<const float4*>(own + 4);
     o[p][0] = a0.x, o[p][1] = a0.y, o[p][2] = a0.z, o[p][3] = a0.w;
     o[p][4] = a1.x, o[p][5] = a1.y, o[p][6] = a1.z, o[p][7] = a1.w;
+    if (e.head_norm) {
+      // this warp's share of the head's sum of squares (a rotation does not change it); raw keys are the values
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(o[p][j], o[p][j], ss);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (sub == 0) ss_red[quarter * 32 + r] = ss;
+      if (head >= e.nh && tok0 + r < tok_limit) {
+        uint4 pk;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&pk);
+#pragma unroll
+        for (int t = 0; t < 4; ++t) h[t] = __floats2bfloat162_rn(o[p][2 * t], o[p][2 * t + 1]);
+        *reinterpret_cast<uint4*>(e.v_cache + ((int64_t)s_dst[r] + (int64_t)(head - e.nh) * e.max_len) * 128 + d0) = pk;
+      }
+    }
     const float sc = s_scale != nullptr ? s_scale[r] : 1.0f;
     if (s_scale != nullptr) {
 #pragma unroll
@@ -722,6 +754,12 @@ __device__ __forceinline__ void epilogue_rope_block(const float* v, const EpiArg
 #pragma unroll
   for (int p = 0; p < 4; ++p) {
     const int tok = tok0 + row0 + 8 * p;
+    if (e.head_norm) {
+      const int r = row0 + 8 * p;
+      const float f = 1.0f / sqrtf((((ss_red[r] + ss_red[32 + r]) + ss_red[64 + r]) + ss_red[96 + r]) * (1.0f / 128.0f) + e.head_eps);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[p][j] *= f;
+    }
     if (tok < tok_limit) {
       __nv_bfloat16* dst = is_q ? e.q_out + ((int64_t)tok * e.nh + head) * 128 + d0
                                 : (is_v ? e.v_cache : e.k_cache) + ((int64_t)s_dst[row0 + 8 * p] + (int64_t)kvh * e.max_len) * 128 + d0;
@@ -890,7 +928,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     // ---------------- epilogue warps ----------------
     const int quarter = warp & 3;  // TMEM lanes [32*quarter, 32*quarter+32) belong to this warp
     float* scr = scratch + (warp - 2) * 32 * kScrLd;
-    constexpr int kOut = (EPI == RD_EPI_SWIGLU) ? 16 : 32;
+    constexpr int kOut = kGlu<EPI> ? 16 : 32;
     constexpr bool kRes = (EPI == RD_EPI_BIAS_SILU_RES || EPI == RD_EPI_RES);
     const int esz = OUT_F32 ? 4 : 2;
     const bool aligned = (((uintptr_t)epi.C | (uintptr_t)(kRes ? epi.R : epi.C)) % 16 == 0) && ((epi.ldc * esz) % 16 == 0) &&
@@ -905,7 +943,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       const int tok_limit = min(M, tok_base + ch.chunk);
       const int n_warp0 = w_tile * BM + quarter * 32;
       const bool vec_ok = aligned && (n_warp0 + 32 <= N);
-      const int out0 = (EPI == RD_EPI_SWIGLU) ? (n_warp0 >> 1) : n_warp0;
+      const int out0 = kGlu<EPI> ? (n_warp0 >> 1) : n_warp0;
       const int acc = local & 1;
       const uint32_t acc_phase = (local >> 1) & 1;
       // the first block's residual row is fetched while the main loop of this tile still runs
@@ -953,11 +991,13 @@ __global__ void __launch_bounds__(kThreads, 1)
         float v[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-        if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
+        if (EPI == kEpiQkvRope && rope_head * 128 >= N) {
+          // a pair's second tile past the last head
+        } else if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
           epilogue_gate_block(v, epi, lane, n_warp0 - (epi.nh + 2 * epi.nkv) * 128, tok_base + c, tok_limit);
         } else if (EPI == kEpiQkvRope) {
           epilogue_rope_block(v, epi, scratch, quarter, lane, rope_head, tok_base + c, tok_limit, s_pos + c, s_dst + c,
-                              norm_in ? s_scale + c : nullptr);
+                              norm_in ? s_scale + c : nullptr, ss_red + ((c >> 5) & 1) * 128);
         } else if (EPI == kEpiArgmax) {
           epilogue_argmax_block(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N);
         } else if (EPI == kEpiSplit && n_warp0 >= epi.n_split) {
@@ -1218,7 +1258,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     // ---------------- epilogue warps (both CTAs, own 128 weight rows) ----------------
     const int quarter = warp & 3;
     float* scr = scratch + (warp - 2) * 32 * kScrLd;
-    constexpr int kOut = (EPI == RD_EPI_SWIGLU) ? 16 : 32;
+    constexpr int kOut = kGlu<EPI> ? 16 : 32;
     constexpr bool kRes = (EPI == RD_EPI_BIAS_SILU_RES || EPI == RD_EPI_RES);
     const int esz = OUT_F32 ? 4 : 2;
     const bool aligned = (((uintptr_t)epi.C | (uintptr_t)(kRes ? epi.R : epi.C)) % 16 == 0) && ((epi.ldc * esz) % 16 == 0) &&
@@ -1232,7 +1272,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       const int tok_limit = min(M, tok_base + ch.chunk);
       const int n_warp0 = w_pair * 2 * BM + (int)rank * BM + quarter * 32;
       const bool vec_ok = aligned && (n_warp0 + 32 <= N);
-      const int out0 = (EPI == RD_EPI_SWIGLU) ? (n_warp0 >> 1) : n_warp0;
+      const int out0 = kGlu<EPI> ? (n_warp0 >> 1) : n_warp0;
       const int acc = local & 1;
       const uint32_t acc_phase = (local >> 1) & 1;
       ResidualRegs<OUT_F32, kOut> res_next;
@@ -1279,11 +1319,13 @@ __global__ void __launch_bounds__(kThreads, 1)
         float v[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-        if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
+        if (EPI == kEpiQkvRope && rope_head * 128 >= N) {
+          // a pair's second tile past the last head
+        } else if (EPI == kEpiQkvRope && rope_head >= epi.nh + 2 * epi.nkv) {
           epilogue_gate_block(v, epi, lane, n_warp0 - (epi.nh + 2 * epi.nkv) * 128, tok_base + c, tok_limit);
         } else if (EPI == kEpiQkvRope) {
           epilogue_rope_block(v, epi, scratch, quarter, lane, rope_head, tok_base + c, tok_limit, s_pos + c, s_dst + c,
-                              norm_in ? s_scale + c : nullptr);
+                              norm_in ? s_scale + c : nullptr, ss_red + ((c >> 5) & 1) * 128);
         } else if (EPI == kEpiArgmax) {
           epilogue_argmax_block(v, epi, scr, lane, n_warp0, tok_base + c, tok_limit, N);
         } else if (EPI == kEpiSplit && n_warp0 >= epi.n_split) {
@@ -1457,6 +1499,7 @@ int launch_epi(const GemmPlan* p, int out_dtype, const EpiArgs& e, const int32_t
     case RD_EPI_RES: return launch_out<RD_EPI_RES>(p, out_dtype, e, m_dev, status, s);
     case RD_EPI_SWIGLU: return launch_out<RD_EPI_SWIGLU>(p, out_dtype, e, m_dev, status, s);
     case RD_EPI_XIELU: return launch_out<RD_EPI_XIELU>(p, out_dtype, e, m_dev, status, s);
+    case RD_EPI_CLAMPED_GLU: return launch_out<RD_EPI_CLAMPED_GLU>(p, RD_BF16, e, m_dev, status, s);
     case kEpiSplit: return launch_out<kEpiSplit>(p, RD_BF16, e, m_dev, status, s);
     case kEpiQkvRope: return launch_out<kEpiQkvRope>(p, out_dtype, e, m_dev, status, s);
     case kEpiArgmax: return launch_out<kEpiArgmax>(p, out_dtype, e, m_dev, status, s);
@@ -1514,6 +1557,18 @@ extern "C" int rd_gemm_bf16_tc_xielu(const void* plan, void* C, int64_t ldc, con
   e.act0 = pos;
   e.act1 = neg;
   return launch_epi(static_cast<const GemmPlan*>(plan), RD_BF16, e, m_dev, RD_EPI_XIELU, status, (cudaStream_t)stream);
+}
+
+extern "C" int rd_gemm_bf16_tc_clamped_glu(const void* plan, void* C, int64_t ldc, const int32_t* m_dev, float limit, float alpha,
+                                           int32_t* status, void* stream) {
+  RD_REQUIRE(plan && C, RD_ERR_ARG);
+  RD_REQUIRE(static_cast<const GemmPlan*>(plan)->N % 2 == 0, RD_ERR_SIZE);
+  EpiArgs e{};
+  e.C = C;
+  e.ldc = ldc;
+  e.act0 = limit;
+  e.act1 = alpha;
+  return launch_epi(static_cast<const GemmPlan*>(plan), RD_BF16, e, m_dev, RD_EPI_CLAMPED_GLU, status, (cudaStream_t)stream);
 }
 
 extern "C" int rd_gemm_bf16_tc_split(const void* plan, void* C, int64_t ldc, float* C_hi, int64_t ld_hi, int n_split,
@@ -1579,11 +1634,12 @@ static int qkv_rope_launch(const void* plan, const int32_t* m_dev, void* q_out, 
                            const int32_t* tok_row, const int32_t* tok_pos, const int32_t* tok_slot, const float* cos_table,
                            const float* sin_table, int n_pos, int nh, int nkv, int hd, int max_len, const float* ss_in,
                            int64_t ss_ld, int ss_slices, int norm_dim, float eps, int32_t* status, void* stream,
-                           int rot_dims = 128, void* gate_out = nullptr, int64_t ld_gate = 0) {
+                           int rot_dims = 128, void* gate_out = nullptr, int64_t ld_gate = 0, bool head_norm = false,
+                           float head_eps = 0.f) {
   RD_REQUIRE(plan && q_out && k_cache && v_cache && tok_row && tok_pos && tok_slot && cos_table && sin_table, RD_ERR_ARG);
   const GemmPlan* p = static_cast<const GemmPlan*>(plan);
   RD_REQUIRE(hd == 128 && nh >= 1 && nkv >= 1 && n_pos >= 1 && max_len >= 1, RD_ERR_SIZE);
-  RD_REQUIRE(p->N == (nh + 2 * nkv) * hd + (gate_out ? nh : 0) && rot_dims % 16 == 0 && rot_dims >= 0 && rot_dims <= hd, RD_ERR_SIZE);
+  RD_REQUIRE(p->N == (nh + (head_norm ? 1 : 2) * nkv) * hd + (gate_out ? nh : 0) && rot_dims % 16 == 0 && rot_dims >= 0 && rot_dims <= hd, RD_ERR_SIZE);
   RD_REQUIRE((((uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)cos_table | (uintptr_t)sin_table) & 15) == 0,
              RD_ERR_ALIGN);
   EpiArgs e{};
@@ -1602,6 +1658,8 @@ static int qkv_rope_launch(const void* plan, const int32_t* m_dev, void* q_out, 
   e.nkv = nkv;
   e.max_len = max_len;
   e.rot_half = rot_dims / 2;
+  e.head_norm = head_norm;
+  e.head_eps = head_eps;
   e.gate_out = (__nv_bfloat16*)gate_out;
   e.ld_gate = ld_gate;
   if (ss_in) {
@@ -1630,6 +1688,15 @@ extern "C" int rd_gemm_bf16_tc_qkvg_rope(const void* plan, const int32_t* m_dev,
   RD_REQUIRE(gate_out && ld_gate >= nh, RD_ERR_ARG);
   return qkv_rope_launch(plan, m_dev, q_out, k_cache, v_cache, tok_row, tok_pos, tok_slot, cos_table, sin_table, n_pos, nh, nkv,
                          hd, max_len, nullptr, 0, 0, 0, 0.f, status, stream, rot_dims, gate_out, ld_gate);
+}
+
+extern "C" int rd_gemm_bf16_tc_qk_rope_norm(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,
+                                            const int32_t* tok_row, const int32_t* tok_pos, const int32_t* tok_slot,
+                                            const float* cos_table, const float* sin_table, int n_pos, int nh, int nkv, int hd,
+                                            int rot_dims, int max_len, float eps, int32_t* status, void* stream) {
+  RD_REQUIRE(eps >= 0.f, RD_ERR_ARG);
+  return qkv_rope_launch(plan, m_dev, q_out, k_cache, v_cache, tok_row, tok_pos, tok_slot, cos_table, sin_table, n_pos, nh, nkv,
+                         hd, max_len, nullptr, 0, 0, 0, 0.f, status, stream, rot_dims, nullptr, 0, true, eps);
 }
 
 extern "C" int rd_gemm_bf16_tc_qkv_rope_normed(const void* plan, const int32_t* m_dev, void* q_out, void* k_cache, void* v_cache,

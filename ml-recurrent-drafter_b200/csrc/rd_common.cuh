@@ -72,6 +72,17 @@ __device__ __forceinline__ float xielu_f(float z, float pos, float neg) {
   return fmaf(pos * p, p, fmaf(neg, __expf(m) - 1.0f - m, 0.5f * z));
 }
 
+// Gated unit with cut inputs: g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = up cut to [-limit, limit].
+__device__ __forceinline__ float clamped_glu_exact(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+// form for rounded (bf16) outputs
+__device__ __forceinline__ float clamped_glu_f(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
+
 __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));

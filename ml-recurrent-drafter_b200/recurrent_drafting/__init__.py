@@ -8,10 +8,12 @@ from . import (  # noqa: F401
     autoregressive,
     configuration_dilavik,
     configuration_drafter,
+    configuration_nulunex,
     kv_cache,
     modeling_dilavik,
     modeling_drafter,
     modeling_llama,
+    modeling_nulunex,
     recurrent_drafting,
     registry,
     replicas,

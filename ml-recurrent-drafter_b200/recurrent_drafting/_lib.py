@@ -16,6 +16,8 @@ LIB_PATH = os.path.join(_HERE, "libredrafter_b200.so")
 F32, BF16 = 0, 1
 EPI_NONE, EPI_BIAS, EPI_BIAS_SILU, EPI_BIAS_SILU_RES, EPI_RES, EPI_SWIGLU = range(6)
 ATTN_CAUSAL, ATTN_TREE, ATTN_DENSE = 0, 1, 2
+MASK_WINDOW, MASK_CHUNK = 0, 1
+GATHER_ALIGN = 64
 TOPK_MAX_KEPT = 64
 STATIC_SCRATCH_BYTES = 16 << 20
 MAX_BEAM_WIDTH = 64
@@ -37,12 +39,15 @@ SIGNATURES = {
     "rd_gemm": (_I, [_I, _I, _P, _L, _P, _L, _P, _L, _P, _P, _L, _I, _P, _I, _I, _I, _P]),
     "rd_gemm_xielu": (_I, [_I, _P, _L, _P, _L, _P, _L, _I, _P, _I, _I, _F, _F, _P]),
     "rd_gemm_bf16_tc_xielu": (_I, [_P, _P, _L, _P, _F, _F, _P, _P]),
+    "rd_gemm_clamped_glu": (_I, [_I, _P, _L, _P, _L, _P, _L, _I, _P, _I, _I, _F, _F, _P]),
+    "rd_gemm_bf16_tc_clamped_glu": (_I, [_P, _P, _L, _P, _F, _F, _P, _P]),
     "rd_gemm_bf16_tc_split": (_I, [_P, _P, _L, _P, _L, _I, _P, _P, _P]),
     "rd_gemm_plan_create": (_P, [_P, _L, _I, _P, _L, _I, _I]),
     "rd_gemm_plan_destroy": (None, [_P]),
     "rd_gemm_bf16_tc": (_I, [_P, _I, _P, _L, _P, _P, _L, _P, _I, _P, _P]),
     "rd_gemm_bf16_tc_qkv_rope": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P]),
     "rd_gemm_bf16_tc_qkvg_rope": (_I, [_P, _P, _P, _P, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P]),
+    "rd_gemm_bf16_tc_qk_rope_norm": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P]),
     "rd_gemm_bf16_tc_res_norm": (_I, [_P, _P, _L, _P, _L, _P, _P, _P, _L, _P, _L, _P, _P]),
     "rd_gemm_bf16_tc_swiglu_normed": (_I, [_P, _P, _L, _P, _P, _L, _I, _I, _F, _P, _P]),
     "rd_gemm_bf16_tc_qkv_rope_normed": (_I, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _L, _I, _I, _F,
@@ -58,7 +63,7 @@ SIGNATURES = {
     "rd_attention_plan_create": (_P, [_P, _I, _P, _P, _I, _I, _I, _I, _I]),
     "rd_attention_plan_destroy": (None, [_P]),
     "rd_attention_tc": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P]),
-    "rd_attention_tc_window": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _P, _L, _P, _P]),
+    "rd_attention_tc_masked": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _P, _P, _P]),
     "rd_attention_split_workspace_bytes": (_L, [_I, _I, _I]),
     "rd_attention_tc_split": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P, _L, _P, _P]),
     "rd_argmax_rows": (_I, [_P, _L, _I, _P, _I, _P, _P, _P]),
@@ -74,6 +79,12 @@ SIGNATURES = {
     "rd_stream_norm": (_I, [_I, _P, _P, _F, _P, _L, _P, _I, _P, _P, _P, _I, _P, _I, _I, _F, _P]),
     "rd_rotary_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
     "rd_attention_window": (_I, [_I, _P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P]),
+    "rd_attention_masked": (_I, [_P, _P]),
+    "rd_attention_desc_bytes": (_I, []),
+    "rd_rotary_norm_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P]),
+    "rd_latent_append": (_I, [_I, _P, _L, _P, _L, _L, _P, _L, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P]),
+    "rd_latent_gather": (_I, [_I, _P, _I, _I, _P, _P, _P, _I, _I, _I, _P, _I, _P, _P, _P]),
+    "rd_head_gemm": (_I, [_I, _P, _L, _L, _P, _P, _L, _L, _I, _P, _I, _I, _I, _P]),
     "rd_mlstm_chunk_workspace_bytes": (_L, [_I, _I, _I, _I, _I]),
     "rd_mlstm_chunk": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _L, _P, _P]),
     "rd_mlstm_tree": (_I, [_I, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _I, _P, _L, _P]),
@@ -82,6 +93,21 @@ SIGNATURES = {
     "rd_decode_advance": (_I, [_P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _P]),
     "rd_cache_unpack_static": (_I, [_I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P]),
 }
+
+
+class AttentionDesc(ctypes.Structure):
+    """rd_attention_desc of include/redrafter_b200.h."""
+
+    _fields_ = [
+        ("q", _P), ("ldq", _L),
+        ("k", _P), ("k_batch", _L), ("k_head", _L), ("k_row", _L),
+        ("k_tail", _P), ("tail_batch", _L), ("tail_row", _L),
+        ("v", _P), ("v_batch", _L), ("v_head", _L), ("v_row", _L),
+        ("gate", _P), ("ld_gate", _L), ("sink", _P), ("out", _P),
+        ("row_start", _P), ("kv_begin", _P), ("base_len", _P), ("tok_pos", _P), ("tree_mask", _P),
+    ] + [(n, ctypes.c_int32) for n in ("mask_words", "dtype", "B", "nh", "nkv", "dim", "tail_dim", "vdim", "max_new", "max_kv", "mode",
+                                       "mask_kind", "window", "keep_first")] + [("scale", _F)]
+
 
 _lib = None
 
@@ -147,6 +173,10 @@ def call(name: str, *args) -> None:
     global launches
     launches += KERNELS_PER_CALL.get(name, 1)
     check(getattr(load(), name)(*args), name)
+
+
+def attention_masked(desc: AttentionDesc) -> None:
+    call("rd_attention_masked", ctypes.byref(desc), stream())
 
 
 def count_replay(n_kernels: int) -> None:

@@ -1,9 +1,9 @@
 """Configuration of the Dilavik decoder: a list of layers, each with its own mixer (sliding-window attention or
 matrix-memory recurrence) and an optional dense feed-forward."""
-import json
-import os
 from dataclasses import dataclass
 from typing import Any, Dict, List, Optional, Union
+
+from .configuration_common import JsonConfig, rotation
 
 ARCHITECTURE = "Dilavik"
 
@@ -22,9 +22,8 @@ class AttentionConfig:
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "AttentionConfig":
-        rot = d.get("rot") or {"dims": 0, "base": 1.0}
-        c = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), int(rot["dims"]), float(rot["base"]),
-                float(d["scale"]), int(d["mask"]["size"]), int(d["mask"]["keep_first"]))
+        c = cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), *rotation(d), float(d["scale"]),
+                int(d["mask"]["size"]), int(d["mask"]["keep_first"]))
         if c.heads % c.kv_heads or c.rot_dims % 2 or c.rot_dims > c.dim or c.window < 1 or c.keep_first < 0:
             raise ValueError(f"inconsistent attention configuration {d}")
         return c
@@ -74,7 +73,7 @@ class LayerConfig:
 
 
 @dataclass(frozen=True)
-class DilavikConfig:
+class DilavikConfig(JsonConfig):
     vocab_size: int
     hidden_size: int
     layers: List[LayerConfig]
@@ -98,12 +97,3 @@ class DilavikConfig:
         return {"architecture": ARCHITECTURE, "vocab": self.vocab_size, "width": self.hidden_size,
                 "embedding": {"scale": self.embedding_scale}, "norm": {"eps": self.norm_eps, "groups": self.norm_groups},
                 "layers": [x.to_dict() for x in self.layers]}
-
-    @classmethod
-    def from_pretrained(cls, path: str) -> "DilavikConfig":
-        with open(os.path.join(path, "config.json")) as f:
-            return cls.from_dict(json.load(f))
-
-    def save_pretrained(self, path: str) -> None:
-        with open(os.path.join(path, "config.json"), "w") as f:
-            json.dump(self.to_dict(), f, indent=1)

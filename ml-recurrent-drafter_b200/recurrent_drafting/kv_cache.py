@@ -122,7 +122,14 @@ class MatrixStateSpec:
     vdim: int
 
 
-LayerSpec = Union[KeyValueSpec, MatrixStateSpec]
+@dataclass(frozen=True)
+class LatentSpec:
+    """A layer that keeps one vector of every token, from which all heads' keys and values are formed."""
+
+    width: int
+
+
+LayerSpec = Union[KeyValueSpec, MatrixStateSpec, LatentSpec]
 
 
 class LayerKeyValues:
@@ -144,10 +151,15 @@ class LayerMatrixState:
         self.draft_gates = torch.empty(draft_tokens, 2 * spec.heads, **f32) if draft_tokens else None
 
 
+class LayerLatents:
+    def __init__(self, spec: LatentSpec, batch: int, max_length: int, dtype: torch.dtype, device):
+        self.rows = torch.zeros(batch, 1, max_length, spec.width, dtype=dtype, device=device)
+
+
 class HybridCache:
     """State of a decoder whose layers differ in what they carry from token to token.  Attention layers keep keys
-    [batch, heads, max_length, dim] and values [batch, heads, max_length, vdim], slot = position in the row; recurrent
-    layers keep their state.  Rows are independent; a row whose length is 0 starts afresh whatever its memory holds (the
+    [batch, heads, max_length, dim] and values [batch, heads, max_length, vdim], or latents [batch, 1, max_length, width],
+    slot = position in the row; recurrent layers keep their state.  Rows are independent; a row whose length is 0 starts afresh whatever its memory holds (the
     recurrent kernels take the zero state then, and no key beyond a row's length is ever read), so giving a row back is
     setting its length to 0."""
 
@@ -156,12 +168,14 @@ class HybridCache:
         self.max_length = max_length
         self.batch_size = batch_size
         self.length = 0
-        self.layers: List[Union[LayerKeyValues, LayerMatrixState]] = []
+        self.layers: List[Union[LayerKeyValues, LayerMatrixState, LayerLatents]] = []
         for spec in layers:
             if isinstance(spec, KeyValueSpec):
                 self.layers.append(LayerKeyValues(spec, batch_size, max_length, dtype, device))
             elif isinstance(spec, MatrixStateSpec):
                 self.layers.append(LayerMatrixState(spec, batch_size, draft_tokens, dtype, device))
+            elif isinstance(spec, LatentSpec):
+                self.layers.append(LayerLatents(spec, batch_size, max_length, dtype, device))
             else:
                 raise TypeError(f"unknown layer spec {spec!r}")
 
@@ -174,5 +188,6 @@ class HybridCache:
 
     def bytes_per_token(self) -> int:
         """Memory that grows with the sequence."""
-        return sum((l.keys[0, :, 0].numel() + l.values[0, :, 0].numel()) * l.keys.element_size()
-                   for l in self.layers if isinstance(l, LayerKeyValues))
+        planes = [p for l in self.layers for p in ((l.keys, l.values) if isinstance(l, LayerKeyValues) else
+                                                   (l.rows,) if isinstance(l, LayerLatents) else ())]
+        return sum(p[0, :, 0].numel() * p.element_size() for p in planes)

@@ -86,6 +86,19 @@ class Linear:
                   _lib.ptr(gate_out), gate_out.stride(0), _lib.ptr(tok_row), _lib.ptr(tok_pos), _lib.ptr(tok_slot), _lib.ptr(cos),
                   _lib.ptr(sin), cos.shape[0], nh, nkv, 128, rot_dims, k_cache.shape[2], _lib.ptr(status), _lib.stream())
 
+    def qk_rope_norm(self, a: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, tok_row, tok_pos, tok_slot,
+                     cos: torch.Tensor, sin: torch.Tensor, nh: int, nkv: int, rot_dims: int, eps: float, m_dev, m_max: int,
+                     status: Optional[torch.Tensor]) -> None:
+        """This weight as the packed q and k projection of heads of 128 features whose values are the keys: rotary embedding
+        on rot_dims features, division by the head's root mean square and the append of keys and values in the epilogue
+        (rd_gemm_bf16_tc_qk_rope_norm); tensor-core path only."""
+        if not self._tc_ok(a, a.stride(0)):
+            raise _lib.RedrafterError("the fused QK projection needs the tensor-core GEMM path (bf16, aligned operands)")
+        plan = self._plan(a, a.stride(0), m_max)
+        _lib.call("rd_gemm_bf16_tc_qk_rope_norm", plan, _lib.ptr(m_dev), _lib.ptr(q_out), _lib.ptr(k_cache), _lib.ptr(v_cache),
+                  _lib.ptr(tok_row), _lib.ptr(tok_pos), _lib.ptr(tok_slot), _lib.ptr(cos), _lib.ptr(sin), cos.shape[0], nh, nkv, 128,
+                  rot_dims, k_cache.shape[2], eps, _lib.ptr(status), _lib.stream())
+
     def residual_with_norm(self, a: torch.Tensor, c: torch.Tensor, residual: torch.Tensor, gamma: torch.Tensor,
                            c2: torch.Tensor, ss: torch.Tensor, m_dev, m_max: int, status: Optional[torch.Tensor]) -> None:
         """c = a @ weight^T + residual, and the producer half of the RMS norm that follows: c2 = c * gamma and the
@@ -144,6 +157,20 @@ class Linear:
         else:
             _lib.call("rd_gemm_xielu", _lib.dtype_code(self.weight.dtype), _lib.ptr(a), a.stride(0), _lib.ptr(self.weight),
                       self.weight.stride(0), _lib.ptr(c), c.stride(0), m_max, _lib.ptr(m_dev), n, k, pos, neg, _lib.stream())
+
+    def clamped_glu(self, a: torch.Tensor, c: torch.Tensor, limit: float, alpha: float, m_dev=None, m_max: Optional[int] = None,
+                    status: Optional[torch.Tensor] = None) -> None:
+        """c = g sigmoid(alpha g) (u + 1) of the interleaved (gate, up) rows of this weight, g and u cut at limit, in the
+        epilogue."""
+        n, k = self.weight.shape
+        m_max = a.shape[0] if m_max is None else m_max
+        if self._tc_ok(a, a.stride(0)):
+            plan = self._plan(a, a.stride(0), m_max)
+            _lib.call("rd_gemm_bf16_tc_clamped_glu", plan, _lib.ptr(c), c.stride(0), _lib.ptr(m_dev), limit, alpha, _lib.ptr(status),
+                      _lib.stream())
+        else:
+            _lib.call("rd_gemm_clamped_glu", _lib.dtype_code(self.weight.dtype), _lib.ptr(a), a.stride(0), _lib.ptr(self.weight),
+                      self.weight.stride(0), _lib.ptr(c), c.stride(0), m_max, _lib.ptr(m_dev), n, k, limit, alpha, _lib.stream())
 
     def split(self, a: torch.Tensor, c: torch.Tensor, c_hi: torch.Tensor, n_split: int, m_dev=None,
               m_max: Optional[int] = None, status: Optional[torch.Tensor] = None) -> None:

@@ -132,6 +132,8 @@ class _StepGraphs:
         self.n_kernels = _lib.launches - before
         _lib.launches = before
         self.draft, self.verify, self.accept = graphs
+        # the captured kernels address these: they stay alive even if a larger request makes the model replace them
+        self.buffers = getattr(model.llm, "held_buffers", lambda: [])()
         self.ready = True
 
 

@@ -5,7 +5,7 @@ from typing import Any, Dict, List
 
 import torch
 
-from . import modeling_dilavik, modeling_llama
+from . import modeling_dilavik, modeling_llama, modeling_nulunex
 
 # architecture name -> class with from_pretrained(path, torch_dtype, device)
 _MODELS: Dict[str, Any] = {}
@@ -43,3 +43,4 @@ def load_model(path: str, torch_dtype: torch.dtype = torch.bfloat16, device="cud
 
 register("LlamaForCausalLM", modeling_llama.LlamaForCausalLM)
 register("Dilavik", modeling_dilavik.DilavikForCausalLM)
+register("Nulunex", modeling_nulunex.NulunexForCausalLM)

@@ -147,7 +147,8 @@ class DecodeGraphs:
         torch.cuda.current_stream().wait_stream(stream)
         self.n_forward = _lib.launches - before - self.n_pick
         # the captured kernels address these: they stay alive even if a larger request makes the model replace its set
-        self.buffers = (session.llm.workspace(session.batch, session.batch), session.llm._head_ws)
+        held = getattr(session.llm, "held_buffers", lambda: [])()
+        self.buffers = (session.llm.workspace(session.batch, session.batch), session.llm._head_ws, held)
         _lib.launches = before  # capturing enqueues nothing
 
 

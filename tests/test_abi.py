@@ -69,6 +69,7 @@ def test_host_only_calls():
     lib = _lib.load()
     assert lib.rd_abi_version() == 1
     assert lib.rd_strerror(0) == b"ok"
+    assert lib.rd_attention_desc_bytes() == ctypes.sizeof(_lib.AttentionDesc)
     assert b"dtype" in lib.rd_strerror(-2)
     # argument validation happens on the host before any launch
     assert lib.rd_tree_pack(None, 1, 1, 1, None, None, None, None, None, None, None, None, None, None, None, None, 1, None, None) == -1

@@ -100,7 +100,7 @@ def test_configuration_and_weights_round_trip(name, tmp_path):
 def test_registry_names_and_refusals(tmp_path):
     from recurrent_drafting import configuration_dilavik, modeling_llama, registry
 
-    assert registry.architectures() == ["Dilavik", "LlamaForCausalLM"]
+    assert {"Dilavik", "LlamaForCausalLM"} <= set(registry.architectures())
     (tmp_path / "config.json").write_text(json.dumps({"model_type": "llama"}))
     assert registry.model_class_of(str(tmp_path)) is modeling_llama.LlamaForCausalLM
     with pytest.raises(ValueError):
