@@ -23,7 +23,7 @@ reference: the reference's own PyTorch implementation (installed under baseline/
            timed beside it as a cross-check.  Without baseline/_ref, or without the host memory
            for the fp32 weights, the port alone is timed and the line says so.
 
---design dilavik [--size 2k|4k]: prefill and decode throughput of that base model beside Llama at equal width, with every
+--design dilavik|nulunex [--size 2k|4k]: prefill and decode throughput of that base model beside Llama at equal width, with every
 kernel's time against its roofline (a line of its own shape; not the workload above).
 
 One JSON line is printed by rank 0.
@@ -711,35 +711,49 @@ def run_cpu(args, as_reference_arm: bool):
 
 # ------------------------------------------------------------------------------------------------
 # Prefill and decode throughput of a base model of another design beside Llama at equal width (random weights).
-# name: width, query heads, key/value heads, matrix-memory heads and sizes, window, Llama feed-forward width, layers of each
+# width, query heads, key/value heads, window (and chunk), Llama feed-forward width, layers / 2; Dilavik: matrix-memory heads
+# and sizes; Nulunex: latent heads, own and shared key features, value features, rank
 DESIGN_SIZES = {
-    "2k": dict(width=2048, heads=16, kv=4, mem=(4, 256, 512), window=1024, ff=5632, blocks=2),
-    "4k": dict(width=4096, heads=32, kv=8, mem=(8, 256, 512), window=1024, ff=11008, blocks=2),
+    "2k": dict(width=2048, heads=16, kv=4, mem=(4, 256, 512), latent=(16, 128, 64, 128, 512), window=1024, ff=5632, blocks=2),
+    "4k": dict(width=4096, heads=32, kv=8, mem=(8, 256, 512), latent=(32, 128, 64, 128, 512), window=1024, ff=11008, blocks=2),
 }
 DESIGN_PREFILL = ((1, 8192), (8, 1024))
-DESIGN_DECODE = ((1, 2048), (8, 2048), (32, 2048))
+DESIGN_DECODE = ((1, 1984), (8, 1984), (32, 1984))  # the timed steps stay inside a chunk of 1024
 
 
-def design_models(size: str, device):
-    """(name, model) pairs: per block attention + feed-forward, two matrix-memory layers, attention + feed-forward; beside
-    it Llama with the same number of attention + feed-forward layers, heads and key/value heads, and as many feed-forward
-    weights (three matrices of ff there, two of 1.5 ff here)."""
+def design_config(design: str, size: str) -> dict:
+    """Dilavik: per block attention + feed-forward, two matrix-memory layers, attention + feed-forward, the feed-forward with
+    as many weights as Llama's (three matrices of ff there, two of 1.5 ff here).  Nulunex: chunked attention and latent
+    attention in turn, each with a feed-forward of Llama's size."""
+    z = DESIGN_SIZES[size]
+    common = {"vocab": 32000, "width": z["width"]}
+    rot = {"dims": 64, "base": 10000.0}
+    if design == "dilavik":
+        att = {"type": "attention", "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2},
+               "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "rot": rot, "scale": 128 ** -0.5,
+                         "mask": {"size": z["window"], "keep_first": 4}}}
+        mem = {"type": "mlstm", "mlp": None, "mixer": dict(zip(("heads", "dim", "vdim"), z["mem"]), gate_cap=15.0)}
+        return {"architecture": "Dilavik", "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6, "groups": 8},
+                "layers": [att, mem, mem, att] * z["blocks"], **common}
+    mlp = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "rot": {"dims": 128, "base": 10000.0},
+                     "scale": 128 ** -0.5, "mask": {"size": z["window"]}}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": dict(zip(("heads", "dim", "rot_dim", "vdim", "kv_rank"), z["latent"]), rot=rot, scale=192 ** -0.5, mask={"size": z["window"]})}
+    return {"architecture": "Nulunex", "norm": {"eps": 1e-6}, "layers": [att, lat] * z["blocks"], **common}
+
+
+def design_models(design: str, size: str, device):
+    """(name, model) pairs: the design, then Llama with as many attention + feed-forward layers, equal heads and key/value heads
+    and equal feed-forward weights."""
     import torch
     from transformers.models.llama.configuration_llama import LlamaConfig
 
     import recurrent_drafting as rd
 
     z = DESIGN_SIZES[size]
-    att = {"type": "attention", "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2},
-           "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "rot": {"dims": 64, "base": 10000.0},
-                     "scale": 128 ** -0.5, "mask": {"size": z["window"], "keep_first": 4}}}
-    mem = {"type": "mlstm", "mlp": None, "mixer": dict(zip(("heads", "dim", "vdim"), z["mem"]), gate_cap=15.0)}
-    cfg = {"architecture": "Dilavik", "vocab": 32000, "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6, "groups": 8},
-           "layers": [att, mem, mem, att] * z["blocks"]}
-    with torch.device(device):
-        m = rd.modeling_dilavik.DilavikForCausalLM(rd.configuration_dilavik.DilavikConfig.from_dict(cfg)).to(torch.bfloat16)
-    yield "dilavik", m.init_random(0.02, seed=1)
-    del m
+    yield design, rd.registry.new_model(design_config(design, size), torch.bfloat16, device).init_random(0.02, seed=1)
     torch.cuda.empty_cache()
     lc = LlamaConfig(hidden_size=z["width"], num_attention_heads=z["heads"], num_key_value_heads=z["kv"], num_hidden_layers=2 * z["blocks"],
                      intermediate_size=z["ff"], vocab_size=32000, rms_norm_eps=1e-6, hidden_act="silu", pad_token_id=0)
@@ -753,9 +767,9 @@ class KernelLog:
     """Event pairs around every C-ABI launch of a few steps, with each call's least time by the measured peaks: the larger of
     its FLOPs over the bf16 GEMM peak and its algorithmic bytes over the copy bandwidth."""
 
-    def __init__(self, model, size: str, batch: int, new: int, cached: int):
+    def __init__(self, design: str, size: str, batch: int, new: int, cached: int):
+        self.design = design
         self.z, self.B, self.new, self.cached, self.M = DESIGN_SIZES[size], batch, new, cached, batch * new
-        self.llama = type(model).__name__.startswith("Llama")
         self.peaks, self.calls, self.shape = _peaks(), [], None
 
     def least(self, name, args):
@@ -770,12 +784,16 @@ class KernelLog:
         elif name in ("rd_rmsnorm", "rd_embed_gather"):
             nbytes = 4.0 * M * H
         elif name.startswith("rd_attention"):
-            first, end = self.cached, self.cached + self.new
-            w = end if self.llama else z["window"]
-            pairs = sum(min(p + 1, w) for p in range(first, end)) if self.new > 1 else min(end, w + (0 if self.llama else 4))
-            keys = min(end, w + self.new)
-            flops = 4.0 * 128 * heads * B * pairs
-            nbytes = B * keys * kv * 256 * 2.0 + M * heads * 256 * 2.0
+            flops, nbytes = self.attention(name, args)
+        elif name == "rd_head_gemm":
+            nh, N, K = args[10:13]
+            flops, nbytes = 2.0 * M * nh * N * K, 2.0 * nh * (N * K + M * (N + K))
+        elif name == "rd_latent_append":
+            nh, _, rot, _, rank = z["latent"]
+            nbytes = M * (nh * rot * 4.0 + (rank + rot) * 6.0)
+        elif name == "rd_latent_gather":
+            nh, _, rot, _, rank = z["latent"]
+            nbytes = B * (self.new + min(self.cached, z["window"])) * (rank + rot) * 4.0
         elif name == "rd_mlstm_chunk":
             nh, d, v = z["mem"]
             flops = M * nh * (4.0 * d * v + 128.0 * (d + v))
@@ -787,6 +805,27 @@ class KernelLog:
             return None
         return max(flops / (self.peaks["tflops"] * 1e12), nbytes / (self.peaks["hbm_gbs"] * 1e9)) * 1e3
 
+    def chunked(self, name, args):
+        return self.design == "nulunex" and (args[0]._obj.mask_kind if name == "rd_attention_masked" else args[11]) == 1
+
+    def attention(self, name, args):
+        """(FLOPs, bytes) over the visible (query, key) pairs: every visible key read once, queries once, outputs written once."""
+        z, M, B = self.z, self.M, self.B
+        positions = range(self.cached, self.cached + self.new)
+        end = self.cached + self.new
+        chunk = self.chunked(name, args)
+        if chunk:
+            pairs, keys = sum(p % z["window"] + 1 for p in positions), end - self.cached // z["window"] * z["window"]
+        else:
+            w = end if self.design == "llama" else z["window"] + (4 if self.design == "dilavik" and self.new == 1 else 0)
+            pairs, keys = sum(min(p + 1, w) for p in positions), min(end, w + self.new)
+        if self.design == "nulunex" and not chunk:
+            nh, d, rot, v, rank = z["latent"]
+            if name == "rd_attention_masked":  # over the latents themselves
+                return 2.0 * nh * (2 * rank + rot) * B * pairs, 2.0 * (B * keys * (rank + rot) + M * nh * (2 * rank + rot))
+            return 2.0 * nh * (d + rot + v) * B * pairs, 2.0 * (B * keys * (nh * (d + v) + rot) + M * nh * (d + rot + v))
+        return 4.0 * 128 * z["heads"] * B * pairs, B * keys * z["kv"] * 256 * 2.0 + M * z["heads"] * 256 * 2.0
+
     def run(self, fn, repeat: int = 3):
         import torch
 
@@ -795,7 +834,7 @@ class KernelLog:
 
         real_call, saved = _lib.call, {}
         # bytes per output element: two, four with a fp32 result, eight where a fp32 residual is read as well; none for the arg-max
-        for method in ("__call__", "xielu", "split", "qkvg_rope", "qkv_rope", "argmax"):
+        for method in ("__call__", "xielu", "clamped_glu", "split", "qkvg_rope", "qkv_rope", "qk_rope_norm", "argmax"):
             saved[method] = getattr(Linear, method)
 
             def wrapped(lin, a, c, *pa, _real=saved[method], _m=method, **kw):
@@ -803,7 +842,8 @@ class KernelLog:
                 if _m == "__call__":
                     per = float(c.element_size()) * (2 if kw.get("residual") is not None else 1)
                 n = lin.weight.shape[0]
-                self.shape = (n // 2 * 2, lin.weight.shape[1], per * (0.5 if _m == "__call__" and pa and pa[0] == _lib.EPI_SWIGLU else 1.0))
+                glu = _m == "clamped_glu" or (_m == "__call__" and pa and pa[0] == _lib.EPI_SWIGLU)
+                self.shape = (n // 2 * 2, lin.weight.shape[1], per * (0.5 if glu else 1.0))
                 _real(lin, a, c, *pa, **kw)
                 self.shape = None
 
@@ -812,6 +852,8 @@ class KernelLog:
         def call(name, *a):
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             label = name if self.shape is None else f"{name} N={self.shape[0]} K={self.shape[1]}"
+            if name.startswith("rd_attention") and self.design == "nulunex":
+                label += " chunk" if self.chunked(name, a) else " latent"
             least = self.least(name, a)
             e0.record()
             real_call(name, *a)
@@ -871,7 +913,7 @@ def run_design(args):
     sampler.start()
     time.sleep(0.15)
     t_wall0, launches0 = datetime.datetime.now(), _lib.launches
-    for name, llm in design_models(args.size, dev):
+    for name, llm in design_models(args.design, args.size, dev):
         res = {"prefill": [], "decode": []}
         for B, T in DESIGN_PREFILL:
             s = Session(llm, B, T + 1)
@@ -884,7 +926,7 @@ def run_design(args):
 
             ms = timed(prefill, max(3, K // 4))
             res["prefill"].append({"batch": B, "tokens": T, "ms": round(ms, 3), "tokens_per_s": round(B * T / ms * 1e3),
-                                   "kernels": KernelLog(llm, args.size, B, T, 0).run(prefill)})
+                                   "kernels": KernelLog(name, args.size, B, T, 0).run(prefill)})
             s.check()
         for B, ctx in DESIGN_DECODE:
             s = Session(llm, B, ctx + K + Wm + 40)
@@ -897,7 +939,7 @@ def run_design(args):
                 s.forward(s.max_length)
 
             step()
-            kernels = KernelLog(llm, args.size, B, 1, ctx).run(step)
+            kernels = KernelLog(name, args.size, B, 1, ctx).run(step)
             graphs = DecodeGraphs(s, greedy, tokens, columns)
 
             def replay():
@@ -936,7 +978,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--config", default="c2", choices=sorted(CONFIGS))
-    ap.add_argument("--design", default=None, choices=["dilavik"],
+    ap.add_argument("--design", default=None, choices=["dilavik", "nulunex"],
                     help="instead of the workload: prefill and decode throughput of this base model beside Llama at equal size (one GPU)")
     ap.add_argument("--size", default="4k", choices=sorted(DESIGN_SIZES), help="layer width with --design")
     ap.add_argument("--no-cpu-baseline", action="store_true")

@@ -317,6 +317,12 @@ RD_API int rd_attention_tc(const void* plan, void* out, const int32_t* row_start
                            const int32_t* base_len, int max_new, int mode, const uint32_t* tree_mask, int mask_words,
                            int32_t* status, void* stream);
 
+/* A plan whose keys have 128 features of their own head and tail_dim (8 .. 64, a multiple of 8) that all heads share: q
+ * [m_max, nh * (128 + tail_dim)], k and v [rows, nh * 128], k_tail [rows, tail_dim], leading dimensions given; key j of row b
+ * is matrix row kv_begin[b] + j of all three.  rd_attention_tc_masked in mode RD_ATTN_CAUSAL takes it. */
+RD_API void* rd_attention_tail_plan_create(const void* q, int64_t ldq, int m_max, const void* k, int64_t ld_k, const void* k_tail,
+                                    int64_t ld_tail, const void* v, int64_t ld_v, int rows, int B, int nh, int tail_dim);
+
 /* rd_attention_tc with the visibility, the gate and the sink of rd_attention_masked (see there); scale > 0; mode
  * RD_ATTN_TREE only with RD_MASK_WINDOW and a window of at least RD_MAX_BEAM_LENGTH. */
 RD_API int rd_attention_tc_masked(const void* plan, void* out, const int32_t* row_start, const int32_t* kv_begin,

@@ -139,6 +139,67 @@ __global__ void __launch_bounds__(kLatentThreads) latent_append_kernel(const T* 
   for (int d = tid; d < a.rank; d += kLatentThreads) dst[d] = Num<T>::from_f(src[d] * f * Num<T>::to_f(norm_w[d]));
 }
 
+// The same for bf16, neighbouring pairs and sizes in multiples of 8, with every load 16 bytes wide: the latent stays in
+// registers between its sum of squares and its store (rank <= 4 * kLatentThreads).
+__global__ void __launch_bounds__(kLatentThreads) latent_append_vec_kernel(const __nv_bfloat16* q, __nv_bfloat16* q_rot, const __nv_bfloat16* norm_w,
+                                                                           __nv_bfloat16* cache, const LatentArgs a) {
+  __shared__ float part[kLatentThreads / 32];
+  rd::pdl_launch_dependents();
+  rd::pdl_wait();
+  const int t = blockIdx.x;
+  if (t >= rd::live_rows(a.m_dev, a.m_max)) return;
+  const int tid = threadIdx.x;
+  const int b = a.tok_row[t], slot = a.tok_slot[t], pos = clamp_pos(a.tok_pos[t], a.n_pos);
+  const float* src = a.dkv + (int64_t)t * a.ld_dkv;
+  const bool has = tid * 4 < a.rank;
+  const float4 x = has ? *reinterpret_cast<const float4*>(src + tid * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  const uint2 w = has ? *reinterpret_cast<const uint2*>(norm_w + tid * 4) : make_uint2(0u, 0u);
+  float ss = rd::warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+  if ((tid & 31) == 0) part[tid >> 5] = ss;
+  // four pairs of a query head, or of the key part (the last units)
+  const int per = a.rot / 8;
+  __nv_bfloat16* dst = cache + ((int64_t)b * a.max_len + slot) * (a.rank + a.rot_dim);
+  for (int u = tid; u < (a.nh + 1) * per; u += kLatentThreads) {
+    const int h = u / per, i = u % per;
+    const float4 c = *reinterpret_cast<const float4*>(a.cos_t + (int64_t)pos * (a.rot / 2) + i * 4);
+    const float4 s = *reinterpret_cast<const float4*>(a.sin_t + (int64_t)pos * (a.rot / 2) + i * 4);
+    float v[8];
+    __nv_bfloat16* to;
+    if (h < a.nh) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(q + (int64_t)t * a.ldq + (int64_t)h * (a.dim + a.rot_dim) + a.dim + i * 8);
+      const __nv_bfloat162* p2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(p2[e]);
+        v[2 * e] = f.x, v[2 * e + 1] = f.y;
+      }
+      to = q_rot + (int64_t)t * a.ld_rot + h * a.rot_head + i * 8;
+    } else {
+      *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(src + a.rank + i * 8);
+      *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(src + a.rank + i * 8 + 4);
+      to = dst + a.rank + i * 8;
+    }
+    const float cc[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
+    uint4 out;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      o2[e] = __floats2bfloat162_rn(v[2 * e] * cc[e] - v[2 * e + 1] * sn[e], v[2 * e + 1] * cc[e] + v[2 * e] * sn[e]);
+    *reinterpret_cast<uint4*>(to) = out;
+  }
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int k = 0; k < kLatentThreads / 32; ++k) tot += part[k];
+  const float f = 1.0f / sqrtf(tot / (float)a.rank + a.eps);
+  if (has) {
+    const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&w);
+    const float2 w0 = __bfloat1622float2(w2[0]), w1 = __bfloat1622float2(w2[1]);
+    __nv_bfloat162 o[2] = {__floats2bfloat162_rn(x.x * f * w0.x, x.y * f * w0.y), __floats2bfloat162_rn(x.z * f * w1.x, x.w * f * w1.y)};
+    *reinterpret_cast<uint2*>(dst + tid * 4) = *reinterpret_cast<uint2*>(o);
+  }
+}
+
 // One warp per gathered row; V: the widest word that divides a row.
 constexpr int kGatherWarps = 8;
 
@@ -150,17 +211,30 @@ __global__ void __launch_bounds__(kGatherWarps * 32) latent_gather_kernel(const 
   rd::pdl_launch_dependents();
   rd::pdl_wait();
   const int r = blockIdx.x * kGatherWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  // which batch row holds gathered row r
+  // which batch row holds gathered row r: the lanes take 32 batch rows at a time
   int at = 0, my_b = -1, my_j = 0;
-  for (int b = 0; b < B; ++b) {
-    const int base = base_len[b], n_new = row_start[b + 1] - row_start[b];
-    int lo = rd_win::first_visible(mask_kind, window, base);
-    lo = lo < 0 ? 0 : lo / RD_GATHER_ALIGN * RD_GATHER_ALIGN;
-    if (lo > base) lo = base / RD_GATHER_ALIGN * RD_GATHER_ALIGN;
-    const int n = n_new > 0 ? base + n_new - lo : 0;
-    if (blockIdx.x == 0 && threadIdx.x == 0) out_begin[b] = at - lo;
-    if (r >= at && r < at + n) my_b = b, my_j = lo + r - at;
-    at += n;
+  for (int b0 = 0; b0 < B; b0 += 32) {
+    const int b = b0 + lane;
+    int lo = 0, n = 0;
+    if (b < B) {
+      const int base = base_len[b], n_new = row_start[b + 1] - row_start[b];
+      lo = rd_win::first_visible(mask_kind, window, base);
+      lo = lo < 0 ? 0 : lo / RD_GATHER_ALIGN * RD_GATHER_ALIGN;
+      n = n_new > 0 ? base + n_new - lo : 0;
+    }
+    int end = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, end, o);
+      if (lane >= o) end += v;
+    }
+    const int begin = at + end - n;  // of this lane's batch row
+    if (b < B && blockIdx.x == 0 && threadIdx.x < 32) out_begin[b] = begin - lo;
+    const uint32_t hit = __ballot_sync(0xffffffffu, r >= begin && r < begin + n);
+    const int who = hit ? __ffs(hit) - 1 : 0;
+    const int j = __shfl_sync(0xffffffffu, lo + r - begin, who);
+    if (hit) my_b = b0 + who, my_j = j;
+    at += __shfl_sync(0xffffffffu, end, 31);
   }
   const int total = at + RD_GATHER_ALIGN - 1;
   if (blockIdx.x == 0 && threadIdx.x == 0) *n_out = total < rows_max ? total : rows_max;
@@ -226,10 +300,17 @@ extern "C" int rd_latent_append(int dtype, const void* q, int64_t ldq, void* q_r
   RD_REQUIRE(m_max >= 1 && nh >= 1 && dim >= 1 && rot_dim >= 0 && rank >= 1 && max_len >= 1 && ld_dkv >= rank + rot_dim &&
                  rotation_ok(rot_dims, rot_dim, cos_table, sin_table, n_pos) && ldq >= (int64_t)nh * (dim + rot_dim),
              RD_ERR_SIZE);
+  const uintptr_t bits = (uintptr_t)q | (uintptr_t)q_rot | (uintptr_t)norm_weight | (uintptr_t)cache | (uintptr_t)dkv | (uintptr_t)cos_table | (uintptr_t)sin_table;
+  const bool vec = dtype == RD_BF16 && neighbours && rot_dims == rot_dim && rot_dim > 0 && bits % 16 == 0 && ld_dkv % 4 == 0 &&
+                   (ldq | ld_rot | rot_head | dim | rot_dim | rank) % 8 == 0 && rank <= 4 * kLatentThreads;
   const LatentArgs a{ldq, ld_rot, rot_head, ld_dkv, dkv, eps, tok_row, tok_pos, tok_slot, cos_table, sin_table, n_pos, m_max, m_dev,
                      nh, dim, rot_dim, rot_dims, neighbours, rank, max_len};
   cudaError_t err = cudaSuccess;
-  RD_DISPATCH_T(dtype, (err = rd::launch_chained(latent_append_kernel<T>, dim3(m_max), dim3(kLatentThreads), 0, (cudaStream_t)stream, 1,
+  if (vec)
+    err = rd::launch_chained(latent_append_vec_kernel, dim3(m_max), dim3(kLatentThreads), 0, (cudaStream_t)stream, 1, (const __nv_bfloat16*)q,
+                             (__nv_bfloat16*)q_rot, (const __nv_bfloat16*)norm_weight, (__nv_bfloat16*)cache, a);
+  else
+    RD_DISPATCH_T(dtype, (err = rd::launch_chained(latent_append_kernel<T>, dim3(m_max), dim3(kLatentThreads), 0, (cudaStream_t)stream, 1,
                                                  (const T*)q, (T*)q_rot, (const T*)norm_weight, (T*)cache, a)));
   RD_CHECK_CHAINED(err);
   return RD_OK;

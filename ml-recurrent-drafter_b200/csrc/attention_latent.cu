@@ -13,6 +13,7 @@ using namespace rd_win;
 
 constexpr int kLatThreads = 256;
 constexpr int kLatWarps = kLatThreads / 32;
+constexpr int kMaxRanks = 8;
 
 template <int DK, int DV, int MT>
 struct LatentSmem {
@@ -25,7 +26,8 @@ struct LatentSmem {
   static constexpr int kP = kR * kBN * 2;
   static constexpr int kRed = 2 * kKG * kR * 4;        // row maxima and sums of every key group
   static constexpr int kMl = kR * 2 * 4;
-  static constexpr int kBytes = kQ + kRing + kP + kRed + kMl;
+  static constexpr int kWeights = kMaxRanks * kR * 4;  // what every rank's partial counts in the result
+  static constexpr int kBytes = kQ + kRing + kP + kRed + kMl + kWeights;
   static_assert(kR * kOld * 4 <= kRing, "the partial output lies over the key ring");
 };
 
@@ -52,6 +54,7 @@ __global__ void __launch_bounds__(kLatThreads) attention_latent_kernel(const Arg
   float* red_m = reinterpret_cast<float*>(sP + Y::kP);  // [KG][R]
   float* red_l = red_m + KG * R;                        // [KG][R]
   float* cta_ml = red_l + KG * R;                       // [R][2]
+  float* weight = cta_ml + R * 2;                       // [kMaxRanks][R]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3;
   const int mt_s = warp % MT, kg = warp / MT, k0 = kg * 8 * MT;  // this warp's rows and keys of a score tile
@@ -212,23 +215,53 @@ __global__ void __launch_bounds__(kLatThreads) attention_latent_kernel(const Arg
     cta_ml[tid * 2 + 1] = l;
   }
   cluster.sync();
-  // the ranks share the rows of the output
-  for (int idx = rank * kLatThreads + tid; idx < n_rows * DV; idx += n_ranks * kLatThreads) {
-    const int r = idx / DV, d = idx % DV;
-    if (d >= a.vdim) continue;
-    float m = -INFINITY;
-    for (int k = 0; k < n_ranks; ++k) m = fmaxf(m, cluster.map_shared_rank(cta_ml, k)[r * 2]);
-    float acc = 0.f, l = 0.f;
-    for (int k = 0; k < n_ranks; ++k) {
-      const float* ml = cluster.map_shared_rank(cta_ml, k);
-      const float f = ml[r * 2] == -INFINITY ? 0.f : exp2f(ml[r * 2] - m);
-      acc = fmaf(f, cluster.map_shared_rank(cta_o, k)[r * Y::kOld + d], acc);
-      l = fmaf(f, ml[r * 2 + 1], l);
+  // what each rank's partial counts in each row, the softmax's sum and the gate included
+  if (tid < n_rows) {
+    float mk[kMaxRanks], lk[kMaxRanks], m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k) {
+      const float2 ml = k < n_ranks ? *reinterpret_cast<const float2*>(cluster.map_shared_rank(cta_ml, k) + tid * 2) : make_float2(-INFINITY, 0.f);
+      mk[k] = ml.x, lk[k] = ml.y;
+      m = fmaxf(m, ml.x);
     }
-    const int t = rs + (row_first + r) / a.nh, h = (row_first + r) % a.nh;
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k) {
+      mk[k] = mk[k] == -INFINITY ? 0.f : exp2f(mk[k] - m);
+      l = fmaf(mk[k], lk[k], l);
+    }
+    const int t = rs + (row_first + tid) / a.nh, h = (row_first + tid) % a.nh;
     float f = finish_softmax(m, l, a.sink, h);
     if (a.gate != nullptr) f *= sigmoid_exact(__bfloat162float(((const __nv_bfloat16*)a.gate)[(int64_t)t * a.ld_gate + h]));
-    ((__nv_bfloat16*)a.out)[((int64_t)t * a.nh + h) * a.vdim + d] = __float2bfloat16_rn(acc * f);
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k) weight[k * R + tid] = mk[k] * f;
+  }
+  __syncthreads();
+  // the ranks share the rows of the output, four values per thread
+  for (int idx = rank * kLatThreads + tid; idx < n_rows * (DV / 4); idx += n_ranks * kLatThreads) {
+    const int r = idx / (DV / 4), d = idx % (DV / 4) * 4;
+    if (d >= a.vdim) continue;
+    float4 part[kMaxRanks];
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k)
+      if (k < n_ranks) part[k] = *reinterpret_cast<const float4*>(cluster.map_shared_rank(cta_o, k) + r * Y::kOld + d);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < kMaxRanks; ++k)
+      if (k < n_ranks) {
+        const float w = weight[k * R + r];
+        acc[0] = fmaf(w, part[k].x, acc[0]);
+        acc[1] = fmaf(w, part[k].y, acc[1]);
+        acc[2] = fmaf(w, part[k].z, acc[2]);
+        acc[3] = fmaf(w, part[k].w, acc[3]);
+      }
+    __nv_bfloat16* dst = (__nv_bfloat16*)a.out + ((int64_t)(rs + (row_first + r) / a.nh) * a.nh + (row_first + r) % a.nh) * a.vdim + d;
+    if (a.vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(a.out) & 7) == 0) {
+      *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc[0], acc[1]), pack_bf16(acc[2], acc[3]));
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (d + e < a.vdim) dst[e] = __float2bfloat16_rn(acc[e]);
+    }
   }
   cluster.sync();  // peers have read this CTA's partial
 }
@@ -249,7 +282,7 @@ int launch(const Args& a, cudaStream_t s) {
   const int64_t visible = (int64_t)a.window + a.max_new + a.keep_first + 2 * kBN;
   const int tiles = (int)((visible < a.max_kv ? visible : a.max_kv) + kBN - 1) / kBN;
   int ranks = 1;
-  while (ranks < 8 && a.B * row_tiles * ranks < 148 && tiles / (ranks * 2) >= 2) ranks *= 2;
+  while (ranks < kMaxRanks && a.B * row_tiles * ranks < 148 && tiles / (ranks * 2) >= 2) ranks *= 2;
   cudaError_t err = rd::launch_chained(kern, dim3(ranks, (int)row_tiles, a.B), dim3(kLatThreads), Y::kBytes, s, ranks, a);
   RD_CHECK_CHAINED(err);
   return RD_OK;

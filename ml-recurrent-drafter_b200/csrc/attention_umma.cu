@@ -1,4 +1,5 @@
-// Tree-masked flash attention on the 5th-generation tensor cores (head_dim 128, bf16).
+// Tree-masked flash attention on the 5th-generation tensor cores (head_dim 128, bf16), and its form for heads of 128 own
+// key features plus up to 64 that all heads share (latent attention's prompts).
 //
 // One CTA serves 128 queries of one (batch row, head): normally every packed tree token of the row.
 //   warps 0, 6  TMA producers (one elected lane each): warp 0 loads the K tiles of 64 keys, warp 6 the V
@@ -20,7 +21,8 @@
 //               one of its rows' running max moved.
 // QK of tile t+1 overlaps the softmax and PV of tile t; P is double-buffered in TMEM so that the
 // softmax of tile t does not wait for PV of tile t-1 before writing P; two CTAs fit on an SM (105 KB
-// of shared memory, 256 TMEM columns each) and overlap each other's latencies.  With n_split > 1
+// of shared memory, 256 TMEM columns each) and overlap each other's latencies.  With the shared key features a CTA holds
+// three boxes of Q and of every K tile and only one V stage, so that two CTAs still fit.  With n_split > 1
 // a CTA walks only its share of the key tiles and leaves an unnormalised partial for the merge
 // kernel at the end of this file.
 //
@@ -37,12 +39,18 @@ constexpr int BMQ = 128;  // queries per CTA
 constexpr int BNK = 64;   // keys per tile
 constexpr int kThreads = 224;
 constexpr int kSubTile = 64 * 128;            // bytes of a [64 rows x 64 bf16] box = 8 KB
-constexpr int kQBytes = BMQ * HD * 2;         // 32 KB: two [128 x 64] boxes
-constexpr int kKVStage = 2 * BNK * HD * 2;    // 32 KB: K (2 boxes) then V (2 boxes)
-constexpr int kStages = 2;
 constexpr int kMaxMaskWords = 16;
-constexpr int kMaskBytes = BMQ * kMaxMaskWords * 4;  // the tile's bitmask rows
-constexpr int kSmemBytes = kQBytes + kStages * kKVStage + kMaskBytes + 1024 + 256;
+// QB: boxes of 64 features of a query and of a key (3: the last box is the shared part)
+template <int QB>
+struct Layout {
+  static constexpr int kQBytes = QB * BMQ * 128;       // QB boxes of [128 x 64]
+  static constexpr int kKStage = QB * kSubTile;
+  static constexpr int kVStage = 2 * kSubTile;
+  static constexpr int kKStages = 2;
+  static constexpr int kVStages = QB == 2 ? 2 : 1;
+  static constexpr int kMaskBytes = QB == 2 ? BMQ * kMaxMaskWords * 4 : 0;  // the tile's bitmask rows (tree mode)
+  static constexpr int kBytes = kQBytes + kKStages * kKStage + kVStages * kVStage + kMaskBytes + 256;
+};
 // TMEM columns
 constexpr float kMaxSlack = 6.0f;  // log2 units the tile max may exceed the running max without moving it
 constexpr uint32_t kColS = 0;     // S: 64 fp32 columns
@@ -50,11 +58,20 @@ constexpr uint32_t kColP = 64;    // P: two buffers of 64 bf16 = 32 columns each
 constexpr uint32_t kColO = 128;   // O: 128 fp32 columns, accumulated over the tiles
 constexpr uint32_t kTmemCols = 256;
 
+// Where a tile's boxes lie: key j of batch row b and key/value head g is row b * row_b + g * row_h + kv_begin[b] + j of the
+// K and V matrices, its own features start at column g * k_col, its value at g * v_col; query head h at column h * q_col.
+struct Places {
+  int row_b, row_h, k_col, v_col, q_col;
+};
+
 struct AttnPlan {
-  CUtensorMap map_q;  // [m_max, nh*128] box 64 x 128
-  CUtensorMap map_k;  // [B*nkv*max_len, 128] box 64 x 64
+  CUtensorMap map_q;  // [m_max, nh * q_col] box 64 x 128
+  CUtensorMap map_k;  // box 64 x 64
   CUtensorMap map_v;
-  int nh, nkv, max_len, B, m_max;
+  CUtensorMap map_t;  // shared key features (tail plans)
+  Places at;
+  bool tail;
+  int nh, nkv, B, m_max;
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -192,17 +209,20 @@ struct WindowArgs {
   const float* sink;          // optional [nh]
 };
 
-template <bool WIN>
+template <bool WIN, int QB>
 __global__ void __launch_bounds__(kThreads, 2)
     attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                          const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* out,
+                          const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_t,
+                          const Places at, __nv_bfloat16* out,
                           const int32_t* row_start, const int32_t* kv_begin,
-                          const int32_t* base_len, int nh, int nkv, int max_len, int mode,
+                          const int32_t* base_len, int nh, int nkv, int mode,
                           const uint32_t* tree_mask, int mask_words, float scale_log2, int32_t* status,
                           int n_split, float* partial, const WindowArgs win) {
+  using L = Layout<QB>;
   const int b = blockIdx.z, h = blockIdx.y;
   rd::pdl_launch_dependents();
   if (threadIdx.x == 0) {
+    if (QB == 3) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_t) : "memory");
     // the descriptors are kernel parameters: their fetch may start before the dependency wait
     asm volatile("prefetch.tensormap [%0];" ::"l"(&map_q) : "memory");
     asm volatile("prefetch.tensormap [%0];" ::"l"(&map_k) : "memory");
@@ -214,12 +234,16 @@ __global__ void __launch_bounds__(kThreads, 2)
   const int q0 = ((int)blockIdx.x / n_split) * BMQ;
   const int split = (int)blockIdx.x % n_split;  // this CTA's share of the key tiles (1 share = the whole row)
   if (q0 >= n_new) return;
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  extern __shared__ __align__(1024) uint8_t smem[];  // the swizzled boxes start at multiples of 1024
+  if ((smem_u32(smem) & 1023) != 0) {
+    if (status && threadIdx.x == 0) atomicExch(status, 24);
+    return;
+  }
   uint8_t* sQ = smem;
-  uint8_t* sKV = smem + kQBytes;
-  uint32_t* sMask = reinterpret_cast<uint32_t*>(smem + kQBytes + kStages * kKVStage);  // [128][mask_words]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kQBytes + kStages * kKVStage + kMaskBytes);
+  uint8_t* sK = smem + L::kQBytes;
+  uint8_t* sV = sK + L::kKStages * L::kKStage;
+  uint32_t* sMask = reinterpret_cast<uint32_t*>(sV + L::kVStages * L::kVStage);  // [128][mask_words]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + L::kVStages * L::kVStage + L::kMaskBytes);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;    // [2]
   uint64_t* v_full = bars + 3;    // [2]
@@ -260,11 +284,26 @@ __global__ void __launch_bounds__(kThreads, 2)
     const int u = t_begin + t;
     return (WIN && u >= kept_tiles) ? u - kept_tiles + first_tile : u;
   };
-  const int kv_row0 = (b * nkv + hk) * max_len + kv_begin[b];  // row of key 0 in the [B*nkv*max_len, 128] view
+  const int kv_row0 = b * at.row_b + hk * at.row_h + kv_begin[b];  // matrix row of key 0
+  auto load_k = [&](int t, uint64_t* bar) {
+    const int row = kv_row0 + tile_of(t) * BNK;
+    uint8_t* dst = sK + (t & 1) * L::kKStage;
+    mbar_expect_tx(bar, L::kKStage);
+    tma_load_2d(dst, &map_k, bar, hk * at.k_col, row);
+    tma_load_2d(dst + kSubTile, &map_k, bar, hk * at.k_col + 64, row);
+    if (QB == 3) tma_load_2d(dst + 2 * kSubTile, &map_t, bar, 0, row);
+  };
+  auto load_v = [&](int t, uint64_t* bar) {
+    const int row = kv_row0 + tile_of(t) * BNK;
+    uint8_t* dst = sV + (t % L::kVStages) * L::kVStage;
+    mbar_expect_tx(bar, L::kVStage);
+    tma_load_2d(dst, &map_v, bar, hk * at.v_col, row);
+    tma_load_2d(dst + kSubTile, &map_v, bar, hk * at.v_col + 64, row);
+  };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < kStages; ++s) {
+    for (int s = 0; s < 2; ++s) {
       mbar_init(&k_full[s], 1);
       mbar_init(&v_full[s], 1);
       mbar_init(&s_full[s], 1);
@@ -277,23 +316,11 @@ __global__ void __launch_bounds__(kThreads, 2)
     // The first loads (Q and the first ring's worth of K and V tiles) go out here, before the TMEM
     // allocation and the block-wide barrier below: a short chain of key tiles spends a large part of its
     // life waiting for this first data.
-    mbar_expect_tx(q_full, kQBytes);
-    tma_load_2d(sQ, &map_q, q_full, h * HD, rs + q0);
-    tma_load_2d(sQ + BMQ * 128, &map_q, q_full, h * HD + 64, rs + q0);
-    for (int t = 0; t < kStages && t < n_tiles; ++t) {
-      const int row = kv_row0 + tile_of(t) * BNK;
-      uint8_t* dk = sKV + t * kKVStage;
-      mbar_expect_tx(&k_full[t], 2 * kSubTile);
-      tma_load_2d(dk, &map_k, &k_full[t], 0, row);
-      tma_load_2d(dk + kSubTile, &map_k, &k_full[t], 64, row);
-    }
-    for (int t = 0; t < kStages && t < n_tiles; ++t) {
-      const int row = kv_row0 + tile_of(t) * BNK;
-      uint8_t* dv = sKV + t * kKVStage + 2 * kSubTile;
-      mbar_expect_tx(&v_full[t], 2 * kSubTile);
-      tma_load_2d(dv, &map_v, &v_full[t], 0, row);
-      tma_load_2d(dv + kSubTile, &map_v, &v_full[t], 64, row);
-    }
+    mbar_expect_tx(q_full, L::kQBytes);
+#pragma unroll
+    for (int i = 0; i < QB; ++i) tma_load_2d(sQ + i * BMQ * 128, &map_q, q_full, h * at.q_col + 64 * i, rs + q0);
+    for (int t = 0; t < L::kKStages && t < n_tiles; ++t) load_k(t, &k_full[t]);
+    for (int t = 0; t < L::kVStages && t < n_tiles; ++t) load_v(t, &v_full[t]);
   }
   if (warp == 1) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(kTmemCols)
@@ -308,24 +335,20 @@ __global__ void __launch_bounds__(kThreads, 2)
   if (warp == 0 || warp == 6) {
     // ---------------- TMA producers: warp 0 = Q and the K ring, warp 6 = the V ring ----------------
     if (lane == 0) {
-      const bool is_k = warp == 0;
-      uint64_t* full = is_k ? k_full : v_full;
-      // a stage is free when the product that read it is done: QK^T of tile t-2 for K, PV of tile t-2
-      // for V.  Each of these barriers completes once per two tiles, so a parity wait is unambiguous.
-      uint64_t* done = is_k ? s_full : o_full;
-      const CUtensorMap* map = is_k ? &map_k : &map_v;
+      // a stage is free when the product that read it is done: QK^T of the tile kKStages before for K, PV of the tile
+      // kVStages before for V.  Each of these barriers completes once per two tiles, so a parity wait is unambiguous.
       bool ok = true;
-      for (int t = kStages; ok && t < n_tiles; ++t) {  // tiles 0 .. kStages-1 were requested at set-up
-        const int s = t & 1;
-        if (!mbar_wait(&done[s], ((t - 2) >> 1) & 1, abort_flag)) {
-          ok = false;
-          break;
+      if (warp == 0) {
+        for (int t = L::kKStages; ok && t < n_tiles; ++t) {  // the tiles before were requested at set-up
+          ok = mbar_wait(&s_full[t & 1], ((t - 2) >> 1) & 1, abort_flag);
+          if (ok) load_k(t, &k_full[t & 1]);
         }
-        uint8_t* dst = sKV + s * kKVStage + (is_k ? 0 : 2 * kSubTile);
-        mbar_expect_tx(&full[s], 2 * kSubTile);
-        const int row = kv_row0 + tile_of(t) * BNK;
-        tma_load_2d(dst, map, &full[s], 0, row);
-        tma_load_2d(dst + kSubTile, map, &full[s], 64, row);
+      } else {
+        for (int t = L::kVStages; ok && t < n_tiles; ++t) {
+          const int u = t - L::kVStages;
+          ok = mbar_wait(&o_full[u & 1], (u >> 1) & 1, abort_flag);
+          if (ok) load_v(t, &v_full[t % L::kVStages]);
+        }
       }
       if (!ok) {
         if (atomicCAS((int*)abort_flag, 0, 1) == 0 && status) atomicExch(status, 21);
@@ -340,11 +363,11 @@ __global__ void __launch_bounds__(kThreads, 2)
       const uint32_t tS = tmem_base + kColS, tP = tmem_base + kColP, tO = tmem_base + kColO;
       bool ok = mbar_wait(q_full, 0, abort_flag);
       auto issue_qk = [&](int t) {
-        const uint8_t* sK = sKV + (t & 1) * kKVStage;
+        const uint8_t* k = sK + (t & 1) * L::kKStage;
 #pragma unroll
-        for (int kd = 0; kd < HD / 16; ++kd) {
+        for (int kd = 0; kd < QB * 4; ++kd) {
           const uint64_t da = desc_k_major(smem_u32(sQ + (kd >> 2) * (BMQ * 128) + (kd & 3) * 32));
-          const uint64_t db = desc_k_major(smem_u32(sK + (kd >> 2) * kSubTile + (kd & 3) * 32));
+          const uint64_t db = desc_k_major(smem_u32(k + (kd >> 2) * kSubTile + (kd & 3) * 32));
           umma_ss(tS, da, db, idesc_qk, kd != 0);
         }
         umma_commit(&s_full[t & 1]);  // S is ready; the K stage is free once this product is done
@@ -375,17 +398,17 @@ __global__ void __launch_bounds__(kThreads, 2)
           ok = false;
           break;
         }
-        if (!mbar_wait(&v_full[t & 1], (t >> 1) & 1, abort_flag)) {
+        if (!mbar_wait(&v_full[t % L::kVStages], (t / L::kVStages) & 1, abort_flag)) {
           ok = false;
           break;
         }
         tc_fence_after();
-        const uint8_t* sV = sKV + (t & 1) * kKVStage + 2 * kSubTile;
+        const uint8_t* v = sV + (t % L::kVStages) * L::kVStage;
 #pragma unroll
         for (int ks = 0; ks < BNK / 16; ++ks) {
           // V: keys are the K dimension (rows of 128 bytes), head_dim the MN dimension: two 64-wide
           // halves kSubTile bytes apart, 8-key groups 1024 bytes apart; 16 keys per MMA = 2048 bytes
-          const uint64_t dv = desc_mn_major(smem_u32(sV + ks * 2048), kSubTile, 1024);
+          const uint64_t dv = desc_mn_major(smem_u32(v + ks * 2048), kSubTile, 1024);
           umma_ts(tO, tP + (t & 1) * 32 + ks * 8, dv, idesc_pv, (t | ks) != 0);
         }
         umma_commit(&o_full[t & 1]);  // O holds tile t; its P buffer and V stage are free
@@ -399,7 +422,7 @@ __global__ void __launch_bounds__(kThreads, 2)
     const int qi = q0 + r;              // query index within the batch row
     const bool live = qi < n_new;
     const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    if (mode == RD_ATTN_TREE) {
+    if (QB == 2 && mode == RD_ATTN_TREE) {
       for (int w = 0; w < mask_words; ++w) sMask[r * mask_words + w] = live ? tree_mask[(int64_t)(rs + qi) * mask_words + w] : 0u;
     }
     const uint32_t* my_mask = sMask + r * mask_words;  // written and read by this thread only
@@ -635,12 +658,34 @@ extern "C" void* rd_attention_plan_create(const void* q, int m_max, const void* 
   AttnPlan* p = new AttnPlan();
   p->nh = nh;
   p->nkv = nkv;
-  p->max_len = max_len;
   p->B = B;
   p->m_max = m_max;
+  p->tail = false;
+  p->at = Places{nkv * max_len, max_len, 0, 0, HD};
   const int64_t kv_rows = (int64_t)B * nkv * max_len;
   if (!make_map(&p->map_q, q, m_max, (int64_t)nh * HD, (int64_t)nh * HD, BMQ) ||
       !make_map(&p->map_k, k_cache, kv_rows, HD, HD, BNK) || !make_map(&p->map_v, v_cache, kv_rows, HD, HD, BNK)) {
+    delete p;
+    return nullptr;
+  }
+  p->map_t = p->map_k;  // not read
+  return p;
+}
+
+extern "C" void* rd_attention_tail_plan_create(const void* q, int64_t ldq, int m_max, const void* k, int64_t ld_k, const void* k_tail,
+                                               int64_t ld_tail, const void* v, int64_t ld_v, int rows, int B, int nh, int tail_dim) {
+  if (!q || !k || !k_tail || !v || m_max < 1 || rows < 1 || B < 1 || nh < 1 || tail_dim < 8 || tail_dim > 64 || tail_dim % 8) return nullptr;
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)k_tail | (uintptr_t)v) & 15) return nullptr;
+  if (ldq % 8 || ld_k % 8 || ld_tail % 8 || ld_v % 8 || ldq < (int64_t)nh * (HD + tail_dim)) return nullptr;
+  AttnPlan* p = new AttnPlan();
+  p->nh = p->nkv = nh;
+  p->B = B;
+  p->m_max = m_max;
+  p->tail = true;
+  p->at = Places{0, 0, HD, HD, HD + tail_dim};
+  // the third box of a query reaches past a tail shorter than 64, into features that meet zeros of the key's box
+  if (!make_map(&p->map_q, q, m_max, (int64_t)nh * (HD + tail_dim), ldq, BMQ) || !make_map(&p->map_k, k, rows, (int64_t)nh * HD, ld_k, BNK) ||
+      !make_map(&p->map_t, k_tail, rows, tail_dim, ld_tail, BNK) || !make_map(&p->map_v, v, rows, (int64_t)nh * HD, ld_v, BNK)) {
     delete p;
     return nullptr;
   }
@@ -666,17 +711,21 @@ static int attention_tc_launch(const void* plan, void* out, const int32_t* row_s
     RD_REQUIRE(workspace && ((uintptr_t)workspace & 15) == 0, RD_ERR_ARG);
     RD_REQUIRE(workspace_bytes >= rd_attention_split_workspace_bytes(p->m_max, p->nh, n_split), RD_ERR_CAPACITY);
   }
-  auto kern = win ? attention_umma_kernel<true> : attention_umma_kernel<false>;
-  static bool smem_set[2] = {false, false};  // set once each, so that steady-state launches are pure launches
-  if (!smem_set[win != nullptr]) {
-    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
-    smem_set[win != nullptr] = true;
+  RD_REQUIRE(!p->tail || (win && n_split == 1 && mode == RD_ATTN_CAUSAL), RD_ERR_UNSUPPORTED);
+  const int which = p->tail ? 2 : (win ? 1 : 0);
+  auto kern = p->tail ? attention_umma_kernel<true, 3> : (win ? attention_umma_kernel<true, 2> : attention_umma_kernel<false, 2>);
+  const int smem = p->tail ? Layout<3>::kBytes : Layout<2>::kBytes;
+  static bool smem_set[3] = {false, false, false};  // set once each, so that steady-state launches are pure launches
+  if (!smem_set[which]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    RD_CHECK_CHAINED(e);
+    smem_set[which] = true;
   }
   dim3 grid(((max_new + BMQ - 1) / BMQ) * n_split, p->nh, p->B);
   const float scale_log2 = 1.4426950408889634f * scale;
-  cudaError_t err = rd::launch_chained(kern, grid, dim3(kThreads), kSmemBytes, (cudaStream_t)stream, 1, p->map_q, p->map_k, p->map_v,
-                                       (__nv_bfloat16*)out, row_start, kv_begin, base_len, p->nh, p->nkv, p->max_len, mode,
-                                       tree_mask, mask_words, scale_log2, status, n_split, (float*)workspace, win ? *win : WindowArgs{});
+  cudaError_t err = rd::launch_chained(kern, grid, dim3(kThreads), smem, (cudaStream_t)stream, 1, p->map_q, p->map_k, p->map_v, p->map_t,
+                                       p->at, (__nv_bfloat16*)out, row_start, kv_begin, base_len, p->nh, p->nkv, mode, tree_mask,
+                                       mask_words, scale_log2, status, n_split, (float*)workspace, win ? *win : WindowArgs{});
   RD_CHECK_CHAINED(err);
   if (n_split > 1) {
     attention_merge_kernel<<<dim3(p->m_max, p->nh), HD, 0, (cudaStream_t)stream>>>((const float*)workspace, (__nv_bfloat16*)out,

@@ -61,6 +61,7 @@ SIGNATURES = {
     "rd_rope_kv_write": (_I, [_I, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _P]),
     "rd_attention": (_I, [_I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _L, _L, _P]),
     "rd_attention_plan_create": (_P, [_P, _I, _P, _P, _I, _I, _I, _I, _I]),
+    "rd_attention_tail_plan_create": (_P, [_P, _L, _I, _P, _L, _P, _L, _P, _L, _I, _I, _I, _I]),
     "rd_attention_plan_destroy": (None, [_P]),
     "rd_attention_tc": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P]),
     "rd_attention_tc_masked": (_I, [_P, _P, _P, _P, _P, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P, _L, _P, _P, _P]),

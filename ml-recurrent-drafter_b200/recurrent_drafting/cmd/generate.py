@@ -9,8 +9,8 @@ of tokens per step:" and "Tokens/second" lines).
 Differences that the missing network and datasets impose: prompts are token ids, either read from
 --prompt_token_ids (a text file, one request per line, ids separated by blanks or commas) or drawn
 uniformly at random (--synthetic_prompts N, the stand-in for --eval_mt_bench); --hf_llm and
---hf_drafter are checkpoint directories, or `random:NAME` (NAME in tiny, vicuna-7b, vicuna-13b, dilavik-tiny) for
-random-init weights of that architecture; the base model's class follows the architecture its config.json
+--hf_drafter are checkpoint directories, or `random:NAME` (NAME in tiny, vicuna-7b, vicuna-13b, dilavik-tiny,
+nulunex-tiny) for random-init weights of that architecture; the base model's class follows the architecture its config.json
 names (registry.py).  A tokenizer directory is optional and only used to print
 text.  There is no CPU path: --use_gpu must name a CUDA device.
 """
@@ -29,15 +29,28 @@ ARCHITECTURES = {
 }
 
 
-# a decoder with window attention and matrix-memory layers, small enough for a smoke run
-DILAVIK_TINY = {
-    "architecture": "Dilavik", "vocab": 1024, "width": 384, "embedding": {"scale": 1.5}, "norm": {"eps": 1e-6, "groups": 3},
-    "layers": [
-        {"type": "mlstm", "mixer": {"heads": 3, "dim": 64, "vdim": 128, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": 1024}},
-        {"type": "attention", "mixer": {"heads": 6, "kv_heads": 3, "dim": 64, "vdim": 64, "rot": {"dims": 64, "base": 10000.0},
-                                        "scale": 0.125, "mask": {"size": 128, "keep_first": 4}},
-         "mlp": {"kind": "dense", "ff": 1024}},
-    ],
+# decoders with layers of different kinds, small enough for a smoke run
+DECODERS = {
+    "dilavik-tiny": {
+        "architecture": "Dilavik", "vocab": 1024, "width": 384, "embedding": {"scale": 1.5}, "norm": {"eps": 1e-6, "groups": 3},
+        "layers": [
+            {"type": "mlstm", "mixer": {"heads": 3, "dim": 64, "vdim": 128, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": 1024}},
+            {"type": "attention", "mixer": {"heads": 6, "kv_heads": 3, "dim": 64, "vdim": 64, "rot": {"dims": 64, "base": 10000.0},
+                                            "scale": 0.125, "mask": {"size": 128, "keep_first": 4}},
+             "mlp": {"kind": "dense", "ff": 1024}},
+        ],
+    },
+    "nulunex-tiny": {
+        "architecture": "Nulunex", "vocab": 1024, "width": 384, "norm": {"eps": 1e-6},
+        "layers": [
+            {"type": "attention", "mixer": {"heads": 6, "kv_heads": 3, "dim": 64, "vdim": 64, "rot": {"dims": 64, "base": 10000.0},
+                                            "scale": 0.125, "mask": {"size": 128}},
+             "mlp": {"ff": 1024, "kind": "dense", "limit": 7.0}},
+            {"type": "latent_attention", "mixer": {"heads": 6, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 128,
+                                                   "rot": {"dims": 32, "base": 10000.0}, "scale": 96 ** -0.5, "mask": {"size": 192}},
+             "mlp": {"ff": 1024, "kind": "dense", "limit": 7.0}},
+        ],
+    },
 }
 
 
@@ -106,15 +119,14 @@ def left_pad(rows: Sequence[List[int]], pad_id: int) -> torch.Tensor:
 def load_models(args, device):
     from transformers.models.llama.configuration_llama import LlamaConfig
 
-    from .. import configuration_dilavik, configuration_drafter, modeling_dilavik, modeling_drafter, modeling_llama, registry
+    from .. import configuration_drafter, modeling_drafter, modeling_llama, registry
 
     dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}[args.dtype]
-    if args.hf_llm == "random:dilavik-tiny":
-        with torch.device(device):
-            llm = modeling_dilavik.DilavikForCausalLM(configuration_dilavik.DilavikConfig.from_dict(DILAVIK_TINY)).to(dtype)
-        llm.init_random(0.02, seed=args.rng_seed)
-    elif args.hf_llm.startswith("random:"):
-        cfg = LlamaConfig(rms_norm_eps=1e-6, hidden_act="silu", pad_token_id=args.pad_token_id, **ARCHITECTURES[args.hf_llm.split(":", 1)[1]])
+    name = args.hf_llm.split(":", 1)[1] if args.hf_llm.startswith("random:") else None
+    if name in DECODERS:
+        llm = registry.new_model(DECODERS[name], dtype, device).init_random(0.02, seed=args.rng_seed)
+    elif name is not None:
+        cfg = LlamaConfig(rms_norm_eps=1e-6, hidden_act="silu", pad_token_id=args.pad_token_id, **ARCHITECTURES[name])
         cfg.rope_theta = 10000.0
         with torch.device(device):
             llm = modeling_llama.LlamaForCausalLM(cfg).to(dtype)

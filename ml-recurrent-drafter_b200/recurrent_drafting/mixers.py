@@ -415,7 +415,7 @@ class LatentAttention(_Mixer):
         c = self.cfg
         if self.w_in.dtype != torch.bfloat16 or ctx.mode != _lib.ATTN_CAUSAL or ctx.max_new <= self.FEW:
             return False
-        if c.dim % 8 or c.rot_dim % 8 or c.vdim % 8 or c.kv_rank % 8:
+        if c.dim % 8 or c.rot_dim % 8 or c.vdim % 8 or c.kv_rank % 8 or self.visible.keep_first:
             return False
         return self._tensor_core_sizes() or (c.dim + c.rot_dim <= 128 and c.vdim <= 128)
 
@@ -440,9 +440,17 @@ class LatentAttention(_Mixer):
                   _lib.ptr(ctx.kv_begin), _lib.ptr(ctx.base_len), ctx.batch, self.visible.kind, self.visible.size, _lib.ptr(rows), n,
                   _lib.ptr(begin), _lib.ptr(n_out), st)
         self.lin[2](rows, kv, m_dev=n_out, m_max=n, status=ctx.status)
-        values = kv[:, H * c.dim :]
+        values, tail = kv[:, H * c.dim :], rows[:, c.kv_rank :]
+        if self._tensor_core_sizes():
+            key = (q.data_ptr(), q.stride(0), ctx.m_max, rows.data_ptr(), n, ctx.batch)
+            plan = self._plans.get(key, "rd_attention_tail_plan_create", _lib.ptr(q), q.stride(0), ctx.m_max, _lib.ptr(kv), up, _lib.ptr(tail),
+                                   self.width, _lib.ptr(values), up, n, ctx.batch, H, c.rot_dim)
+            v = self.visible
+            _lib.call("rd_attention_tc_masked", plan, _lib.ptr(mixed), _lib.ptr(ctx.row_start), _lib.ptr(begin), _lib.ptr(ctx.base_len), ctx.max_new,
+                      ctx.mode, None, None, 0, c.scale, v.kind, v.size, v.keep_first, None, 0, _lib.ptr(self.sink), _lib.ptr(ctx.status), st)
+            return
         _lib.attention_masked(attention_desc(
-            ctx, self.visible, c.scale, q.dtype, q=q, ldq=q.stride(0), k=kv, k_head=c.dim, k_row=up, k_tail=rows[:, c.kv_rank :],
+            ctx, self.visible, c.scale, q.dtype, q=q, ldq=q.stride(0), k=kv, k_head=c.dim, k_row=up, k_tail=tail,
             tail_row=self.width, tail_dim=c.rot_dim, v=values, v_head=c.vdim, v_row=up, sink=self.sink, out=mixed, nh=H, nkv=H,
             dim=c.dim + c.rot_dim, vdim=c.vdim, kv_begin=begin))
 

@@ -41,6 +41,13 @@ def load_model(path: str, torch_dtype: torch.dtype = torch.bfloat16, device="cud
     return model_class_of(path).from_pretrained(path, torch_dtype=torch_dtype, device=device)
 
 
+def new_model(config: Dict[str, Any], torch_dtype: torch.dtype = torch.bfloat16, device="cuda"):
+    """A base model without weights, from the contents of a nested config.json (the classes that name their config_class)."""
+    cls = _MODELS[architecture_of(config)]
+    with torch.device(device):
+        return cls(cls.config_class.from_dict(config)).to(torch_dtype)
+
+
 register("LlamaForCausalLM", modeling_llama.LlamaForCausalLM)
 register("Dilavik", modeling_dilavik.DilavikForCausalLM)
 register("Nulunex", modeling_nulunex.NulunexForCausalLM)
