@@ -718,7 +718,8 @@ DESIGN_SIZES = {
     "4k": dict(width=4096, heads=32, kv=8, mem=(8, 256, 512), latent=(32, 128, 64, 128, 512), window=1024, ff=11008, blocks=2),
 }
 DESIGN_PREFILL = ((1, 8192), (8, 1024))
-DESIGN_DECODE = ((1, 1984), (8, 1984), (32, 1984))  # the timed steps stay inside a chunk of 1024
+DESIGN_DECODE = (1, 8, 32)
+DESIGN_CONTEXT = {"dilavik": 2048, "nulunex": 1984}  # the steps after 1984 tokens stay inside a chunk of 1024 positions
 
 
 def design_config(design: str, size: str) -> dict:
@@ -806,7 +807,9 @@ class KernelLog:
         return max(flops / (self.peaks["tflops"] * 1e12), nbytes / (self.peaks["hbm_gbs"] * 1e9)) * 1e3
 
     def chunked(self, name, args):
-        return self.design == "nulunex" and (args[0]._obj.mask_kind if name == "rd_attention_masked" else args[11]) == 1
+        if self.design != "nulunex" or name == "rd_attention_latent":
+            return False
+        return (args[0]._obj.mask_kind if name == "rd_attention_masked" else args[11]) == 1
 
     def attention(self, name, args):
         """(FLOPs, bytes) over the visible (query, key) pairs: every visible key read once, queries once, outputs written once."""
@@ -821,7 +824,7 @@ class KernelLog:
             pairs, keys = sum(min(p + 1, w) for p in positions), min(end, w + self.new)
         if self.design == "nulunex" and not chunk:
             nh, d, rot, v, rank = z["latent"]
-            if name == "rd_attention_masked":  # over the latents themselves
+            if name in ("rd_attention_masked", "rd_attention_latent"):  # over the latents themselves
                 return 2.0 * nh * (2 * rank + rot) * B * pairs, 2.0 * (B * keys * (rank + rot) + M * nh * (2 * rank + rot))
             return 2.0 * nh * (d + rot + v) * B * pairs, 2.0 * (B * keys * (nh * (d + v) + rot) + M * nh * (d + rot + v))
         return 4.0 * 128 * z["heads"] * B * pairs, B * keys * z["kv"] * 256 * 2.0 + M * z["heads"] * 256 * 2.0
@@ -852,7 +855,7 @@ class KernelLog:
         def call(name, *a):
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             label = name if self.shape is None else f"{name} N={self.shape[0]} K={self.shape[1]}"
-            if name.startswith("rd_attention") and self.design == "nulunex":
+            if name in ("rd_attention_masked", "rd_attention_tc_masked") and self.design == "nulunex":
                 label += " chunk" if self.chunked(name, a) else " latent"
             least = self.least(name, a)
             e0.record()
@@ -928,7 +931,8 @@ def run_design(args):
             res["prefill"].append({"batch": B, "tokens": T, "ms": round(ms, 3), "tokens_per_s": round(B * T / ms * 1e3),
                                    "kernels": KernelLog(name, args.size, B, T, 0).run(prefill)})
             s.check()
-        for B, ctx in DESIGN_DECODE:
+        ctx = DESIGN_CONTEXT[args.design]
+        for B in DESIGN_DECODE:
             s = Session(llm, B, ctx + K + Wm + 40)
             s.extend(torch.randint(3, 32000, (B * ctx,), device=dev), [ctx] * B)
             tokens = torch.zeros(B, s.max_length, dtype=torch.int64, device=dev)

@@ -473,8 +473,7 @@ RD_API int rd_attention_window(int dtype, const void* q, int64_t ldq, const void
 /* The general form of the above.  Key j of row b under key/value head g starts at k + b*k_batch + g*k_head + (kv_begin[b] + j)*k_row
  * (strides in elements); its last tail_dim features may come from k_tail, one vector per key for all heads.  Values likewise.
  * mask_kind RD_MASK_WINDOW: as above; RD_MASK_CHUNK: a query at position p sees s <= p iff p / window == s / window (or s <
- * keep_first).  sink (optional, fp32 [nh]): a score per head that takes part in the softmax's sum without a value.  Where v
- * is k (the values are the first vdim features of the one key all heads share) keys are read once for both. */
+ * keep_first).  sink (optional, fp32 [nh]): a score per head that takes part in the softmax's sum without a value. */
 #define RD_MASK_WINDOW 0
 #define RD_MASK_CHUNK 1
 typedef struct rd_attention_desc {
@@ -500,6 +499,13 @@ typedef struct rd_attention_desc {
   float scale;
 } rd_attention_desc;
 RD_API int rd_attention_masked(const rd_attention_desc* desc, void* stream);
+/* The same for bf16 where all heads share one key of dim <= 576 features (a multiple of 8) whose first vdim <= 512 are the
+ * value: keys are read once for both.  `plan` (host memory; NULL on failure) holds the TMA descriptors of these exact buffers:
+ * q [q_rows = tokens * nh, dim] and cache [cache_rows, dim]; the descriptor's ldq is nh * dim, k_row dim, nkv 1; its pointers
+ * q, k and v are not read.  `status` (optional) receives a non-zero code if a bounded device-side wait gave up. */
+RD_API void* rd_attention_latent_plan_create(const void* q, int64_t q_rows, const void* cache, int64_t cache_rows, int dim);
+RD_API void rd_attention_latent_plan_destroy(void* plan);
+RD_API int rd_attention_latent(const void* plan, const rd_attention_desc* desc, int32_t* status, void* stream);
 RD_API int rd_attention_desc_bytes(void); /* sizeof(rd_attention_desc), for bindings that restate it */
 
 /* Rotary embedding of the first rot_dims features of every q and k head, then (eps >= 0) each of these heads over its root

@@ -108,9 +108,6 @@ int launch_rowwise(const rd_win::Args& a, cudaStream_t s) {
 
 }  // namespace
 
-int rd_attention_latent_launch(const rd_win::Args& a, cudaStream_t s);  // attention_latent.cu
-bool rd_attention_latent_ok(const rd_win::Args& a);
-
 extern "C" int rd_attention_masked(const rd_attention_desc* desc, void* stream) {
   RD_REQUIRE(desc, RD_ERR_ARG);
   const rd_win::Args& a = *desc;
@@ -124,7 +121,6 @@ extern "C" int rd_attention_masked(const rd_attention_desc* desc, void* stream) 
              RD_ERR_SIZE);
   cudaStream_t s = (cudaStream_t)stream;
   if (a.dtype == RD_F32) return launch_rowwise<float>(a, s);
-  if (rd_attention_latent_ok(a)) return rd_attention_latent_launch(a, s);
   const uintptr_t bits = (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.out | (uintptr_t)(a.tail_dim ? a.k_tail : nullptr);
   const int64_t strides = a.ldq | a.k_batch | a.k_head | a.k_row | a.v_batch | a.v_head | a.v_row |
                           (a.tail_dim ? a.tail_batch | a.tail_row | a.tail_dim : 0);

@@ -81,6 +81,9 @@ SIGNATURES = {
     "rd_rotary_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
     "rd_attention_window": (_I, [_I, _P, _L, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _I, _I, _I, _P]),
     "rd_attention_masked": (_I, [_P, _P]),
+    "rd_attention_latent_plan_create": (_P, [_P, _L, _P, _L, _I]),
+    "rd_attention_latent_plan_destroy": (None, [_P]),
+    "rd_attention_latent": (_I, [_P, _P, _P, _P]),
     "rd_attention_desc_bytes": (_I, []),
     "rd_rotary_norm_append": (_I, [_I, _P, _L, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P]),
     "rd_latent_append": (_I, [_I, _P, _L, _P, _L, _L, _P, _L, _P, _F, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P]),

@@ -1,6 +1,7 @@
 """Building blocks of decoders with a 32-bit residual stream: grouped attention over a window or a chunk, latent attention,
 the matrix-memory recurrence, dense feed-forwards.  A block owns its weights in the layouts the kernels consume and runs
 packed tokens (see StepContext); every constant is a parameter of the block."""
+import ctypes
 import math
 import os
 from dataclasses import dataclass
@@ -141,7 +142,8 @@ class AttentionPlans:
 
     MAX_PLANS = 8
 
-    def __init__(self):
+    def __init__(self, destroy: str = "rd_attention_plan_destroy"):
+        self._destroy = destroy
         self._plans: Dict[Tuple, int] = {}
 
     def get(self, key: Tuple, entry: str, *args) -> int:
@@ -158,9 +160,9 @@ class AttentionPlans:
     def drop(self) -> None:
         plans, self._plans = self._plans, {}
         if plans:
-            lib = _lib.load()
+            destroy = getattr(_lib.load(), self._destroy)
             for p in plans.values():
-                lib.rd_attention_plan_destroy(p)
+                destroy(p)
 
     def __del__(self):
         try:
@@ -341,9 +343,11 @@ class LatentAttention(_Mixer):
         self.up_k: Optional[torch.Tensor] = None  # [heads, rank, dim]
         self.up_v: Optional[torch.Tensor] = None  # [heads, vdim, rank]
         self._plans = AttentionPlans()
+        self._latent_plans = AttentionPlans("rd_attention_latent_plan_destroy")
 
     def drop_plans(self) -> None:
         self._plans.drop()
+        self._latent_plans.drop()
 
     def cache_spec(self) -> kv_cache.LayerSpec:
         return kv_cache.LatentSpec(self.width)
@@ -404,9 +408,15 @@ class LatentAttention(_Mixer):
         _lib.call("rd_head_gemm", code, _lib.ptr(q), q.stride(0), c.dim + c.rot_dim, _lib.ptr(self.up_k), _lib.ptr(wide), wide.stride(0),
                   self.width, m, _lib.ptr(ctx.m_dev), H, r, c.dim, st)
         rows = state.rows
-        _lib.attention_masked(attention_desc(
-            ctx, self.visible, c.scale, q.dtype, q=wide, ldq=wide.stride(0), k=rows, v=rows, sink=self.sink, out=latent, nh=H, nkv=1,
-            dim=self.width, vdim=r, **cache_strides(rows, "k"), **cache_strides(rows, "v")))
+        desc = attention_desc(ctx, self.visible, c.scale, q.dtype, q=wide, ldq=wide.stride(0), k=rows, v=rows, sink=self.sink, out=latent, nh=H,
+                              nkv=1, dim=self.width, vdim=r, **cache_strides(rows, "k"), **cache_strides(rows, "v"))
+        if q.dtype == torch.bfloat16 and self.width % 8 == 0 and self.width <= 576 and r <= 512:
+            key = (wide.data_ptr(), m, rows.data_ptr(), rows.shape)
+            plan = self._latent_plans.get(key, "rd_attention_latent_plan_create", _lib.ptr(wide), m * H, _lib.ptr(rows), rows.shape[0] * rows.shape[2],
+                                          self.width)
+            _lib.call("rd_attention_latent", plan, ctypes.byref(desc), _lib.ptr(ctx.status), st)
+        else:
+            _lib.attention_masked(desc)
         _lib.call("rd_head_gemm", code, _lib.ptr(latent), latent.stride(0), r, _lib.ptr(self.up_v), _lib.ptr(mixed), mixed.stride(0), c.vdim,
                   m, _lib.ptr(ctx.m_dev), H, c.vdim, r, st)
 

@@ -1,4 +1,6 @@
 """Each mechanism of the Nulunex decoder alone: the CUDA kernels against the plain implementation."""
+import ctypes
+
 import numpy as np
 import pytest
 import torch
@@ -325,7 +327,16 @@ def run_attention(form, kind, size, rows, dtype, H, G, d, dv, tail=0, scale=None
         else:
             desc.k, desc.k_batch, desc.k_head, desc.k_row = ptr(kc), *kc.stride()[:3]
             desc.v, desc.v_batch, desc.v_head, desc.v_row = ptr(vc), *vc.stride()[:3]
-        _lib.attention_masked(desc)
+        if form == "latent" and dtype == torch.bfloat16 and d % 8 == 0:
+            lib = _lib.load()
+            plan = lib.rd_attention_latent_plan_create(ptr(tq), M * H, ptr(kc), B * max_len, d)
+            assert plan
+            _lib.call("rd_attention_latent", plan, ctypes.byref(desc), ptr(status), _lib.stream())
+            torch.cuda.synchronize()
+            lib.rd_attention_latent_plan_destroy(plan)
+            assert int(status) == 0
+        else:
+            _lib.attention_masked(desc)
         torch.cuda.synchronize()
     got = out.double().cpu().numpy().reshape(M, H, dv)
     visible = (nulunex.window_visible, nulunex.chunk_visible)[kind]
@@ -389,15 +400,13 @@ def test_attention_whose_values_are_a_part_of_the_shared_key(dt, kind, size, H, 
         check_attention(run_attention("latent", kind, size, rows, DTYPES[dt], H, 1, d, dv, sink=sink), DTYPES[dt])
 
 
-@pytest.mark.parametrize("dt", ["fp32", "bf16"])
 @pytest.mark.parametrize("kind,size", [(0, 50), (0, 64), (1, 50), (1, 64), (1, 40)])
-@pytest.mark.parametrize("form,H,G,d,dv,tail", [("cache", 4, 2, 64, 56, 0), ("umma", 4, 2, 128, 128, 0), ("latent", 4, 1, 72, 64, 0), ("tail", 2, 2, 40, 32, 8),
-                                               ("umma-tail", 2, 2, 192, 128, 64)])
+@pytest.mark.parametrize("dt,form,H,G,d,dv,tail", [
+    ("fp32", "cache", 4, 2, 64, 56, 0), ("bf16", "cache", 4, 2, 64, 56, 0), ("bf16", "umma", 4, 2, 128, 128, 0), ("fp32", "latent", 4, 1, 72, 64, 0),
+    ("bf16", "latent", 4, 1, 72, 64, 0), ("bf16", "tail", 2, 2, 40, 32, 8), ("bf16", "umma-tail", 2, 2, 192, 128, 64)])
 def test_one_key_at_every_edge_stands_out(dt, kind, size, form, H, G, d, dv, tail):
     """A key that outweighs all others sits just inside or just outside the window or the chunk, or at a tile's border: the
     output is its value, or is not moved by it."""
-    if dt == "fp32" and form != "cache" and form != "latent":
-        pytest.skip("a bf16 kernel")
     q = 199
     first = q - size + 1 if kind == 0 else q // size * size
     for cached, new in ((0, 200), (140, 60), (199, 1), (196, 4)):
