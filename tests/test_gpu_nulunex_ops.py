@@ -5,7 +5,6 @@ import numpy as np
 import pytest
 import torch
 
-import nulunex_builders as nb
 from oracle import nulunex
 
 pytestmark = pytest.mark.gpu
